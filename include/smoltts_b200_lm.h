@@ -23,7 +23,7 @@
 extern "C" {
 #endif
 
-#define SMOL_LM_ABI_VERSION 4
+#define SMOL_LM_ABI_VERSION 5
 
 enum { SMOL_LM_BF16 = 0, SMOL_LM_F32 = 1 };
 /* token mixers */
@@ -40,8 +40,10 @@ enum {
                                           norm-divided queries and keys, the values being the key projection; one gate per head */
     SMOL_LM_MIX_LIGHTNING = 6,         /* linear attention with one constant decay per head over silu'd q, k, v; state [dim, vdim]
                                           per head; RMS norm over all heads together and a sigmoid gate per channel */
-    SMOL_LM_MIX_HGRN2 = 7              /* linear attention whose forget gate f (bounded below per channel) also writes: key = 1 - f;
+    SMOL_LM_MIX_HGRN2 = 7,             /* linear attention whose forget gate f (bounded below per channel) also writes: key = 1 - f;
                                           state [dim, vdim] per head; RMS norm per head */
+    SMOL_LM_MIX_RETENTION = 8          /* linear attention with one constant decay per head and rotated queries and keys; state
+                                          [dim, vdim] per head; weightless RMS division per head and a silu gate per channel */
 };
 /* feed-forward kinds */
 enum {
@@ -58,22 +60,37 @@ enum {
     SMOL_LM_ACT_RELU_SQUARED = 3       /* max(z, 0)^2 */
 };
 /* how a router turns its logits into scores */
-enum { SMOL_LM_ROUTE_SOFTMAX = 0, SMOL_LM_ROUTE_SIGMOID = 1 };
+enum {
+    SMOL_LM_ROUTE_SOFTMAX = 0,
+    SMOL_LM_ROUTE_SIGMOID = 1,
+    SMOL_LM_ROUTE_CHOSEN = 2           /* the largest logits are chosen, the weights are the softmax over the chosen logits alone */
+};
 /* how a layer wraps its sublayers */
 enum {
     SMOL_LM_BLOCK_SANDWICH = 0,        /* x += ls * norm_b(sublayer(norm_a(x))): norms with one-plus weight vectors, layer scales */
     SMOL_LM_BLOCK_POSTNORM = 1,        /* x = g * rms_divide(alpha * x + sublayer(x)): one gain per norm; after each layer the
                                           stream becomes a weighted sum of the embedding output and every layer's result */
-    SMOL_LM_BLOCK_PRENORM = 2          /* x += sublayer(norm(x)) with the norm SmolLmConfig.norm_kind names; a run flagged
+    SMOL_LM_BLOCK_PRENORM = 2,         /* x += sublayer(norm(x)) with the norm SmolLmConfig.norm_kind names; a run flagged
                                           SMOL_LM_RUN_ADD_EMBED starts from x + the embedding output */
+    SMOL_LM_BLOCK_PARALLEL = 3         /* x += residual_mult * (mixer(h) + feed-forward(h)), h = norm1(x) read by both (norms as in the
+                                          pre-norm block).  Feed-forwards: none or routed.  w_in holds, after the mixer's rows, what
+                                          the feed-forward needs of the same input: the shared expert's gate and up rows [shared_ff
+                                          each], the router's rows [n_experts], with shared_gate one gate row, then zero rows up to a
+                                          multiple of 8; w_out is [width, mixer columns + shared_ff], its last columns the shared
+                                          expert's down matrix.  A run flagged SMOL_LM_RUN_MERGE_EMBED starts from
+                                          w_merge [x; embedding output] */
 };
-/* the norm of the pre-norm block */
+/* the norm of the pre-norm and the parallel block */
 enum {
     SMOL_LM_NORM_RMS = 0,              /* x / rms(x) * weight */
-    SMOL_LM_NORM_DYT = 1               /* tanh(alpha * x) * weight + shift: no mean, no variance */
+    SMOL_LM_NORM_DYT = 1,              /* tanh(alpha * x) * weight + shift: no mean, no variance */
+    SMOL_LM_NORM_LAYER = 2             /* (x - mean) / sqrt(variance + eps) * weight + shift */
 };
 /* per-run flags (SmolLmConfig.run_flags) */
-enum { SMOL_LM_RUN_ADD_EMBED = 1 };    /* the embedding output is added to the stream before this run */
+enum {
+    SMOL_LM_RUN_ADD_EMBED = 1,         /* the embedding output is added to the stream before this run (pre-norm block) */
+    SMOL_LM_RUN_MERGE_EMBED = 2        /* the stream becomes w_merge [stream; embedding output] before this run (parallel block) */
+};
 
 /* One layer: sizes, constants and weights.  Matrices (`const void*`) have the engine's element type and are [out, in]
  * row-major; vectors (`const float*`) are always fp32. */
@@ -183,6 +200,15 @@ typedef struct SmolLmLayer {
     int32_t shared_ff;        /* routed: size of an expert every token uses, added with weight 1 (0: none) */
     const void* w_shared_in;  /* [2 * shared_ff (gate rows, up rows) or shared_ff (ff_plain)][width] */
     const void* w_shared_out; /* [width][shared_ff] */
+    /* --- options of the softmax attention: q_norm = k_norm = NULL leaves queries and keys as projected; q_temp_every > 0: the query at
+     *     position p is multiplied by 1 + q_temp_coef * ln(floor((p + 1) / q_temp_every) + 1) --- */
+    float q_temp_coef, q_temp_every;
+    /* --- retention (w_in rows: q | k [heads*dim each] | v | gate [heads*vdim each]): q and k rotated on their leading rot_dims coordinates
+     *     (rot_half 1: coordinate i with i + rot_dims/2, 0: 2i with 2i + 1), k then multiplied by score_scale; head_decay [heads] --- */
+    int32_t rot_half;
+    /* --- feed-forward options --- */
+    const float* router_bias; /* added to the router's logits themselves [n_experts + n_identity] (NULL: none) */
+    int32_t shared_gate;      /* 1: the shared expert's result is multiplied by sigmoid of one gate row's product with the input (parallel block) */
 } SmolLmLayer;
 
 typedef struct SmolLmConfig {
@@ -201,8 +227,10 @@ typedef struct SmolLmConfig {
     float residual_alpha;     /* post-norm block: multiplies the stream before the sublayer's output is added */
     float logit_scale;        /* multiplies the logits */
     int32_t norm_plain;       /* sandwich block: 1 = the norms' weight vectors are used as they are, 0 = one is added to them */
-    int32_t norm_kind;        /* pre-norm block: SMOL_LM_NORM_* */
+    int32_t norm_kind;        /* pre-norm and parallel block: SMOL_LM_NORM_* */
     const int32_t* run_flags; /* HOST array [n_runs] of SMOL_LM_RUN_* bits, copied by create (NULL: none set) */
+    float residual_mult;      /* parallel block */
+    float logit_softcap;      /* logits <- logit_softcap * tanh(logits / logit_softcap) after logit_scale (0: none) */
 } SmolLmConfig;
 
 typedef struct SmolLmGlobals {
@@ -210,7 +238,8 @@ typedef struct SmolLmGlobals {
     const void* head;         /* [vocab, width] */
     const float* final_norm;  /* sandwich block: [width] one-plus weight; post-norm block: one gain */
     const float* embed_norm;  /* post-norm block: one gain of the norm after the embedding */
-    const float *final_norm_shift, *final_norm_alpha;   /* Dynamic-Tanh final norm: shift [width], alpha (one number) */
+    const float *final_norm_shift, *final_norm_alpha;   /* Dynamic-Tanh final norm: shift [width], alpha (one number); layer norm: shift */
+    const void* w_merge;      /* [width, 2 * width]: runs flagged SMOL_LM_RUN_MERGE_EMBED */
 } SmolLmGlobals;
 
 /* A ragged batch.  All arrays live on the device. */

@@ -11,7 +11,7 @@ import os
 from . import build as _build
 from ._errors import SMOL_OK, SmolError
 
-SMOL_LM_ABI_VERSION = 4
+SMOL_LM_ABI_VERSION = 5
 SMOL_LM_BF16, SMOL_LM_F32 = 0, 1
 
 
@@ -38,18 +38,20 @@ SmolLmLayer._fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "kv_heads", "
     (n, C.c_void_p) for n in ("norm1_shift", "norm1_alpha", "norm2_shift", "norm2_alpha")] + [("chunk", C.c_int32)] + [
     (n, C.c_void_p) for n in ("head_bias", "talk")] + [(n, C.c_float) for n in ("rot_stretch", "rot_low", "rot_high", "rot_original")] + [
     (n, C.c_void_p) for n in ("head_decay", "forget_lower", "proj_norm")] + [
-    (n, C.c_int32) for n in ("ff_plain", "group_rank_top", "shared_ff")] + [(n, C.c_void_p) for n in ("w_shared_in", "w_shared_out")]
+    (n, C.c_int32) for n in ("ff_plain", "group_rank_top", "shared_ff")] + [(n, C.c_void_p) for n in ("w_shared_in", "w_shared_out")] + [
+    ("q_temp_coef", C.c_float), ("q_temp_every", C.c_float), ("rot_half", C.c_int32), ("router_bias", C.c_void_p), ("shared_gate", C.c_int32)]
 
 
 class SmolLmConfig(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("dtype", "vocab", "width", "n_layers", "n_runs", "page_size", "max_step_tokens",
                                          "max_step_seqs", "max_want", "max_context", "use_graph")] + [
         ("embed_scale", C.c_float), ("norm_eps", C.c_float), ("block", C.c_int32), ("residual_alpha", C.c_float), ("logit_scale", C.c_float),
-        ("norm_plain", C.c_int32), ("norm_kind", C.c_int32), ("run_flags", C.POINTER(C.c_int32))]
+        ("norm_plain", C.c_int32), ("norm_kind", C.c_int32), ("run_flags", C.POINTER(C.c_int32)),
+        ("residual_mult", C.c_float), ("logit_softcap", C.c_float)]
 
 
 class SmolLmGlobals(C.Structure):
-    _fields_ = [(n, C.c_void_p) for n in ("embed", "head", "final_norm", "embed_norm", "final_norm_shift", "final_norm_alpha")]
+    _fields_ = [(n, C.c_void_p) for n in ("embed", "head", "final_norm", "embed_norm", "final_norm_shift", "final_norm_alpha", "w_merge")]
 
 
 class SmolLmStep(C.Structure):

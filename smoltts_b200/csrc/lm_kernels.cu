@@ -618,7 +618,13 @@ struct AttnArgs {
     const float *bias, *slope;
     int window, has_gate, out_ld;
     float softcap, two_over_cap, out_scale;      // two_over_cap = 2 / softcap (0 without a cap)
+    float temp_coef = 0.0f, temp_every = 0.0f;   // query temperature (temp_every 0: none), see attn_temperature
 };
+
+// what a query at `pos` is multiplied by: 1 + coef * ln(floor((pos + 1) / every) + 1)
+__device__ __forceinline__ float attn_temperature(const AttnArgs& A, int pos) {
+    return A.temp_every > 0.0f ? 1.0f + A.temp_coef * logf(floorf((float)(pos + 1) / A.temp_every) + 1.0f) : 1.0f;
+}
 
 // first key a query at `pos` sees
 __device__ __forceinline__ int attn_first_key(const AttnArgs& A, int pos) { return A.window > 0 ? max(0, pos - A.window + 1) : 0; }
@@ -637,8 +643,8 @@ __device__ __forceinline__ float attn_score(const AttnArgs& A, float dot, int di
     return s;
 }
 
-// One warp per (token, slot): slots 0..H-1 norm a query head into qbuf, H..H+G-1 norm a key head into the pool,
-// H+G..H+2G-1 copy a value head into the pool.
+// One warp per (token, slot): slots 0..H-1 norm a query head into qbuf (times the query temperature), H..H+G-1 norm a key head
+// into the pool, H+G..H+2G-1 copy a value head into the pool.  q_norm / k_norm == nullptr: no norm.
 template <class T>
 __global__ void attn_prep_kernel(const AttnArgs A, T* __restrict__ qbuf, T* __restrict__ pool) {
     const int lane = threadIdx.x & 31;
@@ -653,8 +659,9 @@ __global__ void attn_prep_kernel(const AttnArgs A, T* __restrict__ qbuf, T* __re
         float ss = 0.0f;
         for (int c = lane; c < A.d; c += 32) { const float v = q[c] + (qb ? qb[c] : 0.0f); ss += v * v; }
         ss = warp_sum(ss);
-        const float r = 1.0f / sqrtf(ss / (float)A.d + A.eps);
-        for (int c = lane; c < A.d; c += 32) qbuf[((size_t)t * A.H + s) * A.d + c] = from_f<T>((q[c] + (qb ? qb[c] : 0.0f)) * r * A.q_norm[c]);
+        const float r = (A.q_norm ? 1.0f / sqrtf(ss / (float)A.d + A.eps) : 1.0f) * attn_temperature(A, A.tok_pos[t]);
+        for (int c = lane; c < A.d; c += 32)
+            qbuf[((size_t)t * A.H + s) * A.d + c] = from_f<T>((q[c] + (qb ? qb[c] : 0.0f)) * r * (A.q_norm ? A.q_norm[c] : 1.0f));
         return;
     }
     const int pos = A.tok_pos[t];
@@ -672,9 +679,9 @@ __global__ void attn_prep_kernel(const AttnArgs A, T* __restrict__ qbuf, T* __re
         float ss = 0.0f;
         for (int c = lane; c < A.d; c += 32) { const float v = k[c] + (kb ? kb[c] : 0.0f); ss += v * v; }
         ss = warp_sum(ss);
-        const float r = 1.0f / sqrtf(ss / (float)A.d + A.eps);
+        const float r = A.k_norm ? 1.0f / sqrtf(ss / (float)A.d + A.eps) : 1.0f;
         T* dst = base + A.k_off + ((size_t)gk * A.page_size + in_pg) * A.d;
-        for (int c = lane; c < A.d; c += 32) dst[c] = from_f<T>((k[c] + (kb ? kb[c] : 0.0f)) * r * A.k_norm[c]);
+        for (int c = lane; c < A.d; c += 32) dst[c] = from_f<T>((k[c] + (kb ? kb[c] : 0.0f)) * r * (A.k_norm ? A.k_norm[c] : 1.0f));
     } else {
         const int gv = s - A.H - A.G;
         const float* v = row + (A.H + A.G) * A.d + gv * A.dv;
@@ -740,7 +747,7 @@ __global__ void __launch_bounds__(256) attn_prep_whole_kernel(const AttnArgs A, 
             }
         }
     };
-    emit(0, nq, rq, A.q_norm, [&](int c, float v) { qbuf[(size_t)t * nq + c] = from_f<T>(v); });
+    emit(0, nq, rq * attn_temperature(A, pos), A.q_norm, [&](int c, float v) { qbuf[(size_t)t * nq + c] = from_f<T>(v); });
     if (page < 0 || page >= A.n_pages) {
         if (threadIdx.x == 0) atomicExch(A.err, 1);
         return;
@@ -1513,13 +1520,13 @@ struct SmolLm {
     SmolLmGlobals g{};
     size_t page_elems = 0, slot_floats = 0, esize = 2;
     int max_in = 0, max_mix = 0, max_ff = 0, max_hd = 0, max_q = 0;
-    bool any_restart = false, any_own_proj = false;
+    bool any_restart = false, any_own_proj = false, any_merge = false;
     // workspace carving (byte offsets)
     size_t o_x, o_hn, o_proj, o_mix, o_y, o_z, o_act, o_dec, o_u, o_au, o_oraw, o_q, o_hw, o_err, o_part, total;
     // post-norm block: every layer result of the step; latent attention: query latent (T), full query (fp32 and T), query in
     // latent space (fp32), rotation frequencies; routed feed-forward: choices, sorted order, tile table, per-pair buffers
     size_t o_hist = 0, o_cq = 0, o_qf = 0, o_freq = 0;
-    size_t o_x0 = 0, o_mix2 = 0, o_y2 = 0, o_spart = 0;
+    size_t o_x0 = 0, o_mix2 = 0, o_y2 = 0, o_spart = 0, o_cat = 0;
     int max_sig_cols = 0;                     // sigmoid attention: widest heads * vdim (partial sums of the tiled kernel's key ranges)    // pre-norm block: the embedding output; mixers with their own output projections: the second result
     size_t o_rlogits = 0, o_rdone = 0, o_ap = 0, o_sel_id = 0, o_sel_w = 0, o_perm = 0, o_slot_of = 0, o_seg = 0, o_tile_g = 0, o_tile_r = 0, o_ntiles = 0, o_zp = 0, o_actp = 0, o_yp = 0;
     int max_routed = 0, max_cq = 0, max_qf = 0, max_top = 0, max_experts = 0, max_pair_ff = 0;
@@ -1537,7 +1544,13 @@ struct SmolLm {
     struct Captured { SmolLmStep key; cudaGraphExec_t exec; int64_t launches; };
     std::vector<Captured> graphs;
     cudaStream_t cap_stream = nullptr;
+    // parallel block: the feed-forward runs on its own stream beside the mixer, between these two events
+    cudaStream_t ff_stream = nullptr;
+    cudaEvent_t ff_start = nullptr, ff_done = nullptr;
     ~SmolLm() {
+        if (ff_start) cudaEventDestroy(ff_start);
+        if (ff_done) cudaEventDestroy(ff_done);
+        if (ff_stream) cudaStreamDestroy(ff_stream);
         for (auto& g : graphs) cudaGraphExecDestroy(g.exec);
         if (cap_stream) cudaStreamDestroy(cap_stream);
     }
@@ -1551,7 +1564,7 @@ static int n_in_of(const SmolLmLayer& L) {
     if (L.mixer == SMOL_LM_MIX_LATENT_ATTENTION) return L.q_rank + L.kv_rank + L.rot_dim + L.heads;
     if (L.mixer == SMOL_LM_MIX_GATED_LINEAR) return 2 * L.heads * L.dim + 2 * L.heads * L.vdim + L.rank;
     if (L.mixer == SMOL_LM_MIX_SIGMOID_ATTENTION) return L.heads * L.dim + L.kv_heads * L.dim + L.heads;
-    if (L.mixer == SMOL_LM_MIX_LIGHTNING) return 2 * L.heads * L.dim + 2 * L.heads * L.vdim;
+    if (L.mixer == SMOL_LM_MIX_LIGHTNING || L.mixer == SMOL_LM_MIX_RETENTION) return 2 * L.heads * L.dim + 2 * L.heads * L.vdim;
     if (L.mixer == SMOL_LM_MIX_HGRN2) return 2 * L.heads * L.dim + L.heads * L.vdim;
     return 5 * L.heads * L.dim + L.rank;
 }
@@ -1560,8 +1573,14 @@ static int n_in_of(const SmolLmLayer& L) {
 static int mix_cols_of(const SmolLmLayer& L) { return L.mixer == SMOL_LM_MIX_GENERAL_DELTA ? L.heads * L.dim : L.heads * L.vdim; }
 static bool pairable(const SmolLmLayer& L) {
     return L.mixer == SMOL_LM_MIX_SINK_ATTENTION || L.mixer == SMOL_LM_MIX_STATE_SPACE || L.mixer == SMOL_LM_MIX_SIGMOID_ATTENTION ||
-           L.mixer == SMOL_LM_MIX_LIGHTNING;
+           L.mixer == SMOL_LM_MIX_LIGHTNING || L.mixer == SMOL_LM_MIX_RETENTION;
 }
+// Parallel block: the rows of the fused input projection that serve the feed-forward (shared expert's gate and up, router, shared
+// gate), and the projection's whole height (a multiple of 8).
+static int ff_rows_of(const SmolLmLayer& L) {
+    return L.mlp == SMOL_LM_MLP_EXPERTS ? (L.ff_plain ? 1 : 2) * L.shared_ff + L.n_experts + L.n_identity + (L.shared_gate ? 1 : 0) : 0;
+}
+static int parallel_n_in_of(const SmolLmLayer& L) { return (n_in_of(L) + ff_rows_of(L) + 7) / 8 * 8; }
 // base^(-2i/dims) for the dims/2 rotated pairs of a latent or sigmoid attention, stretched band by band when L.rot_stretch
 // is set (see the header)
 static void push_frequencies(std::vector<float>& table, const SmolLmLayer& L, bool stretch) {
@@ -1612,7 +1631,8 @@ extern "C" int smol_lm_create(const SmolLmConfig* cfg, const SmolLmLayer* layers
         if (L.mixer == SMOL_LM_MIX_SINK_ATTENTION) {
             if (L.kv_heads < 1 || L.heads % L.kv_heads != 0 || L.vdim < 1) return fail(SMOL_ERR_INVALID, "attention: heads must be a multiple of kv_heads");
             if (L.vdim > 32 * kAttnMaxV) return fail(SMOL_ERR_UNSUPPORTED, "attention: value size above 256");
-            if (L.window < 0 || L.softcap < 0.0f) return fail(SMOL_ERR_INVALID, "attention: window and softcap must not be negative");
+            if (L.window < 0 || L.softcap < 0.0f || L.q_temp_every < 0.0f) return fail(SMOL_ERR_INVALID, "attention: window, softcap and q_temp_every must not be negative");
+            if (!L.q_norm != !L.k_norm || (L.norm_whole && !L.q_norm)) return fail(SMOL_ERR_INVALID, "attention: q_norm and k_norm come together, norm_whole needs them");
             r.k_off = m->page_elems;
             r.v_off = r.k_off + (size_t)L.kv_heads * cfg->page_size * L.dim;
             m->page_elems = r.v_off + (size_t)L.kv_heads * cfg->page_size * L.vdim;
@@ -1673,6 +1693,18 @@ extern "C" int smol_lm_create(const SmolLmConfig* cfg, const SmolLmLayer* layers
             m->max_heads = std::max(m->max_heads, L.heads);
             m->max_vdim = std::max(m->max_vdim, L.vdim);
             m->max_mix = std::max(m->max_mix, L.heads * L.vdim);
+        } else if (L.mixer == SMOL_LM_MIX_RETENTION) {
+            if (L.dim > 256) return fail(SMOL_ERR_UNSUPPORTED, "recurrent mixer: key size above 256");
+            if (L.vdim < 1 || !L.head_decay || L.rot_dims < 0 || L.rot_dims > L.dim || L.rot_dims % 2)
+                return fail(SMOL_ERR_INVALID, "retention: vdim must be positive, head_decay set, rot_dims even and at most dim");
+            r.state_off = m->slot_floats;
+            m->slot_floats += (size_t)L.heads * L.dim * L.vdim;
+            m->slot_floats = (m->slot_floats + 3) / 4 * 4;
+            r.freq_off = m->freq_table.size();
+            push_frequencies(m->freq_table, L, true);
+            m->max_hd = std::max(m->max_hd, L.heads * std::max(L.dim, L.vdim));
+            m->max_mix = std::max(m->max_mix, L.heads * L.vdim);
+            m->max_conv = std::max(m->max_conv, 2 * L.heads * L.dim);
         } else if (L.mixer == SMOL_LM_MIX_LIGHTNING || L.mixer == SMOL_LM_MIX_HGRN2) {
             if (L.dim > 256) return fail(SMOL_ERR_UNSUPPORTED, "recurrent mixer: key size above 256");
             if (L.vdim < 1 || !L.out_norm) return fail(SMOL_ERR_INVALID, "linear attention: vdim must be positive and out_norm set");
@@ -1707,28 +1739,34 @@ extern "C" int smol_lm_create(const SmolLmConfig* cfg, const SmolLmLayer* layers
         r.layer = rs.layer = li;
         r.flags = cfg->run_flags ? cfg->run_flags[n] : 0;
         if (r.flags & SMOL_LM_RUN_ADD_EMBED) m->any_restart = true;
+        if (r.flags & SMOL_LM_RUN_MERGE_EMBED) m->any_merge = true;
         int rc = place(L, r);
-        const bool prenorm = cfg->block == SMOL_LM_BLOCK_PRENORM;
+        const bool prenorm = cfg->block == SMOL_LM_BLOCK_PRENORM, parallel = cfg->block == SMOL_LM_BLOCK_PARALLEL;
         if (rc == SMOL_OK && L.side) {
             if (!pairable(L) || !pairable(*L.side)) rc = fail(SMOL_ERR_UNSUPPORTED, "mixers side by side: softmax or sigmoid attention, the state-space recurrence, lightning attention");
-            else if (cfg->block == SMOL_LM_BLOCK_POSTNORM) rc = fail(SMOL_ERR_UNSUPPORTED, "mixers side by side need the sandwich or the pre-norm block");
+            else if (cfg->block == SMOL_LM_BLOCK_POSTNORM || parallel) rc = fail(SMOL_ERR_UNSUPPORTED, "mixers side by side need the sandwich or the pre-norm block");
             else if (L.proj_norm && (!prenorm || !L.side->proj_norm || !L.side->w_out)) rc = fail(SMOL_ERR_INVALID, "proj_norm: the pre-norm block, and set on both mixers with their own w_out");
             else rc = place(*L.side, rs);
             if (rc == SMOL_OK) m->max_mix = std::max(m->max_mix, mix_cols_of(L) + mix_cols_of(*L.side));
             if (rc == SMOL_OK && L.proj_norm) m->any_own_proj = true;
         }
-        if (rc == SMOL_OK && prenorm) {
-            if (cfg->norm_kind != SMOL_LM_NORM_RMS && cfg->norm_kind != SMOL_LM_NORM_DYT) rc = fail(SMOL_ERR_INVALID, "pre-norm block: unknown norm kind");
-            else if (!L.norm1 || (L.mlp != SMOL_LM_MLP_NONE && !L.norm2)) rc = fail(SMOL_ERR_INVALID, "pre-norm block: norm weights");
-            else if (cfg->norm_kind == SMOL_LM_NORM_DYT && (!L.norm1_shift || !L.norm1_alpha || (L.mlp != SMOL_LM_MLP_NONE && (!L.norm2_shift || !L.norm2_alpha))))
-                rc = fail(SMOL_ERR_INVALID, "pre-norm block: the Dynamic-Tanh norms need shifts and alphas");
+        const bool norm2 = prenorm && L.mlp != SMOL_LM_MLP_NONE;
+        if (rc == SMOL_OK && (prenorm || parallel)) {
+            if (cfg->norm_kind < SMOL_LM_NORM_RMS || cfg->norm_kind > SMOL_LM_NORM_LAYER) rc = fail(SMOL_ERR_INVALID, "unknown norm kind");
+            else if (!L.norm1 || (norm2 && !L.norm2)) rc = fail(SMOL_ERR_INVALID, "pre-norm and parallel block: norm weights");
+            else if (cfg->norm_kind == SMOL_LM_NORM_DYT && (!L.norm1_alpha || (norm2 && !L.norm2_alpha))) rc = fail(SMOL_ERR_INVALID, "the Dynamic-Tanh norms need alphas");
+            else if (cfg->norm_kind != SMOL_LM_NORM_RMS && (!L.norm1_shift || (norm2 && !L.norm2_shift))) rc = fail(SMOL_ERR_INVALID, "Dynamic-Tanh and layer norms need shifts");
+            else if (parallel && ((L.mlp != SMOL_LM_MLP_NONE && L.mlp != SMOL_LM_MLP_EXPERTS) || !pairable(L) || L.in_bias))
+                rc = fail(SMOL_ERR_UNSUPPORTED, "parallel block: routed feed-forwards or none, softmax / sigmoid attention, state-space, lightning or retention mixers without biases");
             else if (L.mlp == SMOL_LM_MLP_POLYNORM || L.route_input || L.out_bias || L.n_identity > 0)
-                rc = fail(SMOL_ERR_UNSUPPORTED, "pre-norm block: PolyNorm feed-forwards, input-weighted routing, identity outputs and out_bias are not built");
+                rc = fail(SMOL_ERR_UNSUPPORTED, "pre-norm and parallel block: PolyNorm feed-forwards, input-weighted routing, identity outputs and out_bias are not built");
         }
-        if (rc == SMOL_OK && !prenorm && (L.shared_ff > 0 || L.proj_norm || (r.flags & SMOL_LM_RUN_ADD_EMBED) || L.mixer >= SMOL_LM_MIX_SIGMOID_ATTENTION ||
+        if (rc == SMOL_OK && ((r.flags & SMOL_LM_RUN_ADD_EMBED) && !prenorm)) rc = fail(SMOL_ERR_UNSUPPORTED, "runs that add the embedding output need the pre-norm block");
+        if (rc == SMOL_OK && ((r.flags & SMOL_LM_RUN_MERGE_EMBED) || L.shared_gate) && !parallel) rc = fail(SMOL_ERR_UNSUPPORTED, "merging runs and gated shared experts need the parallel block");
+        if (rc == SMOL_OK && !prenorm && !parallel && (L.shared_ff > 0 || L.proj_norm || L.mixer >= SMOL_LM_MIX_SIGMOID_ATTENTION ||
                                          (L.side && L.side->mixer >= SMOL_LM_MIX_SIGMOID_ATTENTION)))
-            rc = fail(SMOL_ERR_UNSUPPORTED, "shared experts, proj_norm, restarting runs, sigmoid / lightning attention and HGRN2 need the pre-norm block");
-        if (rc == SMOL_OK && L.shared_ff > 0 && (L.mlp != SMOL_LM_MLP_EXPERTS || !L.w_shared_in || !L.w_shared_out)) rc = fail(SMOL_ERR_INVALID, "shared expert: routed feed-forwards only, with both matrices");
+            rc = fail(SMOL_ERR_UNSUPPORTED, "shared experts, proj_norm, sigmoid / lightning attention, HGRN2 and retention need the pre-norm or the parallel block");
+        if (rc == SMOL_OK && L.shared_ff > 0 && (L.mlp != SMOL_LM_MLP_EXPERTS || (!parallel && (!L.w_shared_in || !L.w_shared_out)))) rc = fail(SMOL_ERR_INVALID, "shared expert: routed feed-forwards only, with both matrices");
         if (rc == SMOL_OK && cfg->block == SMOL_LM_BLOCK_POSTNORM && (L.out_bias || L.route_input))
             rc = fail(SMOL_ERR_UNSUPPORTED, "out_bias and route_input need the sandwich block");
         if (rc != SMOL_OK) { delete m; return rc; }
@@ -1749,9 +1787,10 @@ extern "C" int smol_lm_create(const SmolLmConfig* cfg, const SmolLmLayer* layers
             m->max_routed = std::max(m->max_routed, E);
             m->max_experts = std::max(m->max_experts, L.n_experts);
             m->max_pair_ff = std::max(m->max_pair_ff, L.top_k * L.ff);
-            if (L.shared_ff > 0) m->max_ff = std::max(m->max_ff, (L.ff_plain ? 1 : 2) * L.shared_ff);
+            if (L.shared_ff > 0 && !parallel) m->max_ff = std::max(m->max_ff, (L.ff_plain ? 1 : 2) * L.shared_ff);
+            if (parallel) m->max_mix = std::max(m->max_mix, mix_cols_of(L) + L.shared_ff);
         }
-        m->max_in = std::max(m->max_in, n_in_of(L) + (L.side ? n_in_of(*L.side) : 0));
+        m->max_in = std::max(m->max_in, parallel ? parallel_n_in_of(L) : n_in_of(L) + (L.side ? n_in_of(*L.side) : 0));
         m->runs.push_back(r);
         m->side_runs.push_back(rs);
     }
@@ -1787,6 +1826,7 @@ extern "C" int smol_lm_create(const SmolLmConfig* cfg, const SmolLmLayer* layers
     }
     if (!m->freq_table.empty()) m->o_freq = carve(m->freq_table.size() * 4 + 4);
     if (m->any_restart) m->o_x0 = carve(T * D * 4);
+    if (m->any_merge) m->o_cat = carve(2 * T * D * E);
     if (m->max_sig_cols > 0 && cfg->dtype == SMOL_LM_BF16) m->o_spart = carve((size_t)kSigmoidRanges * T * m->max_sig_cols * 4);
     if (m->any_own_proj) {
         m->o_mix2 = carve(T * (size_t)std::max(m->max_mix, 1) * E);
@@ -1899,6 +1939,14 @@ extern "C" int smol_lm_bind(SmolLm* m, const SmolLmGlobals* g, void* d_workspace
     if (m->cfg.block == SMOL_LM_BLOCK_POSTNORM && !g->embed_norm) return fail(SMOL_ERR_INVALID, "smol_lm_bind: the post-norm block needs embed_norm");
     if (m->cfg.block == SMOL_LM_BLOCK_PRENORM && m->cfg.norm_kind == SMOL_LM_NORM_DYT && (!g->final_norm_shift || !g->final_norm_alpha))
         return fail(SMOL_ERR_INVALID, "smol_lm_bind: the Dynamic-Tanh final norm needs its shift and alpha");
+    if ((m->cfg.block == SMOL_LM_BLOCK_PRENORM || m->cfg.block == SMOL_LM_BLOCK_PARALLEL) && m->cfg.norm_kind == SMOL_LM_NORM_LAYER && !g->final_norm_shift)
+        return fail(SMOL_ERR_INVALID, "smol_lm_bind: the final layer norm needs its shift");
+    if (m->any_merge && !g->w_merge) return fail(SMOL_ERR_INVALID, "smol_lm_bind: merging runs need w_merge");
+    if (m->cfg.block == SMOL_LM_BLOCK_PARALLEL && !m->ff_stream) {
+        CU(cudaStreamCreateWithFlags(&m->ff_stream, cudaStreamNonBlocking));
+        CU(cudaEventCreateWithFlags(&m->ff_start, cudaEventDisableTiming));
+        CU(cudaEventCreateWithFlags(&m->ff_done, cudaEventDisableTiming));
+    }
     if ((size_t)m->cfg.width * 4 > 48 * 1024) {
         CU(cudaFuncSetAttribute(residual_norm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, m->cfg.width * 4));
         CU(cudaFuncSetAttribute(residual_norm_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, m->cfg.width * 4));
@@ -2170,8 +2218,10 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
     float* hist = reinterpret_cast<float*>(m->ws + m->o_hist);
     T* pool = static_cast<T*>(m->pages);
     const int nthr = D >= 1024 ? 256 : 128;
-    const bool postnorm = c.block == SMOL_LM_BLOCK_POSTNORM, prenorm = c.block == SMOL_LM_BLOCK_PRENORM;
+    const bool postnorm = c.block == SMOL_LM_BLOCK_POSTNORM, parallel = c.block == SMOL_LM_BLOCK_PARALLEL;
+    const bool prenorm = c.block == SMOL_LM_BLOCK_PRENORM;
     float* x0 = m->any_restart ? reinterpret_cast<float*>(m->ws + m->o_x0) : nullptr;
+    T* cat = m->any_merge ? reinterpret_cast<T*>(m->ws + m->o_cat) : nullptr;
     T* mix2 = reinterpret_cast<T*>(m->ws + m->o_mix2);
     float* y2 = reinterpret_cast<float*>(m->ws + m->o_y2);
     auto norm_of = [&](const float* w, const float* shift, const float* alpha) { return NormSpec{c.norm_kind, w, shift, alpha, c.norm_eps}; };
@@ -2185,10 +2235,11 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
 
     if (postnorm) {
         embed_gain_norm_kernel<T><<<Tn, nthr, 0, st>>>(s->tokens, static_cast<const T*>(m->g.embed), D, c.vocab, m->g.embed_norm, c.norm_eps, x, hist, hn);
-    } else if (prenorm) {
+    } else if (prenorm || parallel) {
         const SmolLmLayer& L0 = m->layers[m->runs[0].layer];
+        const bool merge = m->runs[0].flags & SMOL_LM_RUN_MERGE_EMBED;
         embed_prenorm_kernel<T><<<Tn, nthr, 0, st>>>(s->tokens, static_cast<const T*>(m->g.embed), c.embed_scale, D, c.vocab,
-                                                     norm_of(L0.norm1, L0.norm1_shift, L0.norm1_alpha), x, x0, hn);
+                                                     merge ? no_norm : norm_of(L0.norm1, L0.norm1_shift, L0.norm1_alpha), x, x0, hn, cat);
     } else {
         embed_norm_kernel<T><<<Tn, nthr, 0, st>>>(s->tokens, static_cast<const T*>(m->g.embed), c.embed_scale, D, c.vocab,
                                                   m->layers[m->runs[0].layer].norm1, c.norm_eps, x, hn, woff);
@@ -2197,9 +2248,16 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
     for (size_t n = 0; n < m->runs.size(); ++n) {
         const RunInfo& R = m->runs[n];
         const SmolLmLayer& L = m->layers[R.layer];
-        const int n_in_main = n_in_of(L), n_in = n_in_main + (L.side ? n_in_of(*L.side) : 0);
+        const int n_in_main = n_in_of(L), n_in = parallel ? parallel_n_in_of(L) : n_in_main + (L.side ? n_in_of(*L.side) : 0);
+        if (R.flags & SMOL_LM_RUN_MERGE_EMBED) {
+            // the stream starts anew from the merged rows, which the previous run's last kernel (or the embedding) has left in cat
+            CU(linear<T>(m, cat, static_cast<const T*>(m->g.w_merge), x, Tn, D, 2 * D, st));
+            prenorm_rows_kernel<T><<<Tn, nthr, 0, st>>>(x, nullptr, norm_of(L.norm1, L.norm1_shift, L.norm1_alpha), D, hn);
+            m->launches++;
+        }
         CU(linear<T>(m, hn, static_cast<const T*>(L.w_in), proj, Tn, n_in, D, st));
-        const int mix_ld = mix_cols_of(L) + (L.side ? mix_cols_of(*L.side) : 0);      // row stride of the mixers' shared result
+        // row stride of the mixers' shared result (parallel block: the shared expert's unit stands behind the mixer's columns)
+        const int mix_ld = mix_cols_of(L) + (L.side ? mix_cols_of(*L.side) : 0) + (parallel && L.mlp == SMOL_LM_MLP_EXPERTS ? L.shared_ff : 0);
         int mix_cols;
         int out_ld_now = mix_ld;        // row stride of the buffer the current mixer writes
         const T* mix_in = mix;          // what the output projection reads
@@ -2219,6 +2277,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             A.q_norm = M.q_norm; A.k_norm = M.k_norm; A.r1 = M.dist_r1; A.r2 = M.dist_r2; A.sink = M.sink;
             A.slope = M.dist_slope; A.window = M.window; A.softcap = M.softcap; A.two_over_cap = M.softcap > 0.0f ? 2.0f / M.softcap : 0.0f;
             A.out_ld = out_ld_now; A.out_scale = M.mix_scale;
+            A.temp_coef = M.q_temp_coef; A.temp_every = M.q_temp_every;
             if (M.norm_whole) {
                 attn_prep_whole_kernel<T><<<Tn, Tn > 64 ? 128 : 256, 0, st>>>(A, qbuf, pool);      // few tokens: more loads in flight per token
             } else {
@@ -2253,7 +2312,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             A.q_src = conv + inner + gn; A.k_src = conv + inner; A.v_src = conv;
             A.q_ld = A.k_ld = A.v_ld = ch;
             A.qk_share = M.heads / M.bc_groups;
-            A.head_decay = head; A.head_step = head + (size_t)Tn * M.heads;
+            A.head_decay = head; A.head_step = head + (size_t)Tn * M.heads; A.head_ld = M.heads;
             A.out_ld = out_ld_now; A.out_scale = 1.0f;
             CU(launch_gla_scan_any(A, s->n_seqs, nullptr, m->slots, oraw, st));
             ssd_out_kernel<T><<<dim3(Tn, M.norm_parts), 256, 0, st>>>(P, oraw, conv, mix_at, m->slots);
@@ -2324,7 +2383,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             A.decay_w2 = A.decay_bias = A.out_norm = nullptr;
             A.seq_start = s->seq_start; A.seq_pos0 = s->seq_pos0; A.seq_slot = s->seq_slot;
             A.slot_floats = m->slot_floats; A.state_off = Ri.state_off; A.n_slots = m->n_slots; A.err = err;
-            A.qk_share = 1; A.head_decay = A.head_step = nullptr;
+            A.qk_share = 1; A.head_decay = A.head_step = nullptr; A.head_ld = M.heads;
             A.out_ld = M.heads * M.vdim; A.out_scale = 1.0f;
             return A;
         };
@@ -2343,13 +2402,163 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             m->launches += 3;
             return SMOL_OK;
         };
+        // Retention: rotated q and k, the scan with one constant decay per head, RMS division per head and silu gate.
+        auto retention = [&](const SmolLmLayer& M, const RunInfo& Ri, const float* pj, T* mix_at, int ld) -> int {
+            const int hd = M.heads * M.dim, pairs = M.rot_dims / 2, per = M.heads * (M.dim - pairs);
+            RetentionArgs P{pj, n_in, M.heads, M.dim, pairs, M.rot_half, M.score_scale, reinterpret_cast<const float*>(m->ws + m->o_freq) + Ri.freq_off, s->tok_pos};
+            retention_prep_kernel<<<dim3(Tn, (per + 511) / 512), 128, 0, st>>>(P, conv);
+            GlaArgs A = scan_args(M, Ri, pj);
+            A.q_src = conv; A.k_src = conv + hd; A.v_src = pj + 2 * hd;
+            A.q_ld = A.k_ld = 2 * hd; A.v_ld = n_in;
+            A.head_decay = M.head_decay; A.head_ld = 0;
+            CU(launch_gla_scan_any(A, s->n_seqs, nullptr, m->slots, oraw, st));
+            A.out_ld = ld; A.out_scale = M.mix_scale;
+            gla_out_kernel<T><<<(Tn * M.heads + 3) / 4, 128, 0, st>>>(A, oraw, mix_at);
+            m->launches += 3;
+            return SMOL_OK;
+        };
         auto run_mixer = [&](const SmolLmLayer& M, const RunInfo& Ri, const float* pj, const float* bias, T* mix_at, int ld) -> int {
             out_ld_now = ld;
             if (M.mixer == SMOL_LM_MIX_SINK_ATTENTION) return attention(M, Ri, pj, bias, mix_at);
             if (M.mixer == SMOL_LM_MIX_STATE_SPACE) return state_space(M, Ri, pj, bias, mix_at);
             if (M.mixer == SMOL_LM_MIX_SIGMOID_ATTENTION) return sigmoid_attention(M, Ri, pj, bias, mix_at, ld);
+            if (M.mixer == SMOL_LM_MIX_RETENTION) return retention(M, Ri, pj, mix_at, ld);
             return lightning(M, Ri, pj, mix_at, ld);
         };
+        // the feed-forward reads hn and leaves its output in y, routed experts theirs in `routed` for the kernel that follows
+        RoutedSum routed;
+        routed.yp = nullptr; routed.slot_of = nullptr; routed.sel_w = nullptr; routed.top = 0;
+        const RoutedSum no_sum = routed;
+        auto actp_of = [](const SmolLmLayer& M) { return ActParams{M.mlp_act, M.act_limit, M.act_alpha, 0}; };
+        // the experts (and a shared expert) of a routed feed-forward may lack gate rows
+        auto expert_actp = [](const SmolLmLayer& M) { return ActParams{M.mlp_act, M.act_limit, M.act_alpha, M.ff_plain ? 1 : 0}; };
+        auto feed_forward = [&](cudaStream_t st) -> int {
+            if (L.mlp == SMOL_LM_MLP_POLYNORM) {
+                CU(linear<T>(m, hn, static_cast<const T*>(L.w_up), z, Tn, L.ff, D, st));
+                polynorm_kernel<T><<<Tn, 256, 0, st>>>(z, L.act, c.norm_eps, L.ff, act);
+                CU(linear<T>(m, act, static_cast<const T*>(L.w_down), y, Tn, D, L.ff, st));
+                m->launches += 1;
+            } else if (L.mlp == SMOL_LM_MLP_GATED) {
+                CU(linear<T>(m, hn, static_cast<const T*>(L.w_up), z, Tn, 2 * L.ff, D, st));
+                gated_act_kernel<T><<<cast_grid((size_t)Tn * L.ff / 4), 256, 0, st>>>(z, L.ff, actp_of(L), (size_t)Tn, act);
+                CU(linear<T>(m, act, static_cast<const T*>(L.w_down), y, Tn, D, L.ff, st));
+                m->launches += 1;
+            } else if (L.mlp == SMOL_LM_MLP_EXPERTS) {
+                int32_t* sel_id = reinterpret_cast<int32_t*>(m->ws + m->o_sel_id);
+                float* sel_w = reinterpret_cast<float*>(m->ws + m->o_sel_w);
+                int32_t* perm = reinterpret_cast<int32_t*>(m->ws + m->o_perm);
+                int32_t* slot_of = reinterpret_cast<int32_t*>(m->ws + m->o_slot_of);
+                int32_t* seg = reinterpret_cast<int32_t*>(m->ws + m->o_seg);
+                int32_t* tile_g = reinterpret_cast<int32_t*>(m->ws + m->o_tile_g);
+                int32_t* tile_r = reinterpret_cast<int32_t*>(m->ws + m->o_tile_r);
+                int32_t* n_tiles = reinterpret_cast<int32_t*>(m->ws + m->o_ntiles);
+                float* zp = reinterpret_cast<float*>(m->ws + m->o_zp);
+                T* actp = reinterpret_cast<T*>(m->ws + m->o_actp);
+                float* yp = reinterpret_cast<float*>(m->ws + m->o_yp);
+                RouteArgs Rt;
+                Rt.w_router = L.w_router; Rt.bias = L.route_bias; Rt.D = D; Rt.E = L.n_experts + L.n_identity; Rt.E_real = L.n_experts;
+                Rt.top = L.top_k; Rt.n_groups = L.n_groups; Rt.keep = L.keep_groups; Rt.scale = L.router_scale; Rt.n_tokens = Tn;
+                Rt.score = L.router_score; Rt.plain = L.router_plain; Rt.group_top = L.group_rank_top; Rt.logit_bias = L.router_bias;
+                Rt.given = nullptr; Rt.given_ld = n_in; Rt.perm = Rt.slot_of = Rt.n_sorted = nullptr;
+                Rt.unit_in = Rt.unit_gate = nullptr; Rt.unit_out = nullptr; Rt.unit_ff = Rt.unit_ld = 0; Rt.unit_act = expert_actp(L);
+                const int pairs = Tn * L.top_k;
+                const bool few = !kIsF32 && L.n_experts > 0 && pairs <= kMoeGemvPairs && D % 8 == 0 && L.ff % 8 == 0;
+                const bool direct = few && L.n_identity == 0;      // the pairs stay in their order: nothing to sort
+                if (direct) { Rt.perm = perm; Rt.slot_of = slot_of; Rt.n_sorted = seg + L.n_experts; }
+                // the router reads the sublayer's input in fp32 where the block keeps it (post-norm), else its T form
+                float* r_logits = reinterpret_cast<float*>(m->ws + m->o_rlogits);
+                int32_t* r_done = reinterpret_cast<int32_t*>(m->ws + m->o_rdone);
+                if (parallel) {
+                    // the fused input product has left the shared expert's gate and up, the router's logits and the shared gate
+                    // behind the mixer's columns
+                    const int SF = (L.ff_plain ? 1 : 2) * L.shared_ff;
+                    Rt.given = proj + n_in_main + SF;
+                    Rt.unit_in = proj + n_in_main; Rt.unit_gate = L.shared_gate ? Rt.given + Rt.E : nullptr;
+                    Rt.unit_out = mix + mix_cols_of(L); Rt.unit_ff = L.shared_ff; Rt.unit_ld = mix_ld;
+                }
+                const dim3 rgrid(Tn, parallel ? 1 : (Rt.E + 3) / 4);
+                if (postnorm) moe_route_kernel<float><<<rgrid, 128, 0, st>>>(Rt, x, r_logits, r_done, sel_id, sel_w);
+                else moe_route_kernel<T><<<rgrid, 128, 0, st>>>(Rt, hn, r_logits, r_done, sel_id, sel_w);
+                m->launches += 1;
+                if (L.n_experts > 0) {
+                    // three forms of the two grouped products, by how many rows an expert gets: a warp per output column for
+                    // a handful of pairs (decoding), 32-row mma.sync tiles, 128-row tcgen05 tiles over rows copied into sorted order
+                    const int NF = L.ff_plain ? L.ff : 2 * L.ff;          // rows of an expert's first matrix
+                    const bool big = !kIsF32 && !few && m->tc_ready && pairs / L.n_experts >= 64 && D % 8 == 0 && L.ff % 8 == 0 &&
+                                     NF >= kTcTileN && D >= kTcTileN && D >= smol::umma::kBK && L.ff >= smol::umma::kBK;
+                    const int tile_rows = big ? smol::umma::kM : kGroupTile;
+                    if (!direct) {
+                        moe_index_kernel<<<1, 256, 0, st>>>(sel_id, pairs, L.n_experts, tile_rows, seg, perm, slot_of, tile_g, tile_r, n_tiles);
+                        m->launches++;
+                    }
+                    const int tiles = pairs / kGroupTile + L.n_experts;
+                    GemmIo io = plain_io(D, NF);
+                    io.sw = (long long)NF * D;
+                    io.tile_group = tile_g; io.tile_row0 = tile_r; io.seg = seg; io.n_tiles = n_tiles;
+                    GemmIo io2 = plain_io(L.ff, D);
+                    io2.sw = (long long)D * L.ff;
+                    io2.tile_group = tile_g; io2.tile_row0 = tile_r; io2.seg = seg; io2.n_tiles = n_tiles;
+                    const size_t act_n = (size_t)pairs * L.ff;
+                    // a router whose weight multiplies the expert's input: the rows are copied into sorted order, each times
+                    // its weight, and the products read that copy
+                    T* ap = reinterpret_cast<T*>(m->ws + m->o_ap);
+                    if (L.route_input) {
+                        moe_gather_scaled_kernel<T><<<pairs, 128, 0, st>>>(hn, perm, L.top_k, sel_w, seg + L.n_experts, D, ap);
+                        m->launches++;
+                    }
+                    if (few) {
+                        moe_gemv_kernel<false><<<dim3((NF + 7) / 8, pairs), 256, 0, st>>>(L.route_input ? ap : hn, perm, L.route_input ? 0 : L.top_k, sel_id,
+                                                                                         seg + L.n_experts, reinterpret_cast<const bf16*>(L.w_experts_in), io.sw,
+                                                                                         zp, NF, D, expert_actp(L));
+                        // the second product applies the activation as it reads the first one's result
+                        moe_gemv_kernel<true><<<dim3((D + 7) / 8, pairs), 256, 0, st>>>(zp, perm, 0, sel_id, seg + L.n_experts,
+                                                                                        reinterpret_cast<const bf16*>(L.w_experts_out), io2.sw, yp, D, L.ff, expert_actp(L));
+                        m->launches += 1;
+                    } else {
+                        bool done = false;
+                        if (big) {
+                            if (!L.route_input) {
+                                moe_gather_kernel<<<pairs, 128, 0, st>>>(reinterpret_cast<const bf16*>(hn), perm, L.top_k, seg + L.n_experts, D,
+                                                                         reinterpret_cast<bf16*>(ap));
+                                m->launches++;
+                            }
+                            done = linear_grouped_tc(m, reinterpret_cast<const bf16*>(ap), reinterpret_cast<const bf16*>(L.w_experts_in), zp, pairs, L.n_experts,
+                                                     NF, D, io, st);
+                        }
+                        if (!done) {
+                            if (!L.route_input) { io.gather = perm; io.gather_div = L.top_k; }
+                            CU(linear_ex<T>(m, L.route_input ? ap : hn, static_cast<const T*>(L.w_experts_in), zp, pairs, NF, D, io, 1, tiles, st));
+                        }
+                        gated_act_kernel<T><<<cast_grid(act_n / 4), 256, 0, st>>>(zp, L.ff, expert_actp(L), (size_t)pairs, actp);
+                        if (!(big && linear_grouped_tc(m, reinterpret_cast<const bf16*>(actp), reinterpret_cast<const bf16*>(L.w_experts_out), yp, pairs,
+                                                       L.n_experts, D, L.ff, io2, st)))
+                            CU(linear_ex<T>(m, actp, static_cast<const T*>(L.w_experts_out), yp, pairs, D, L.ff, io2, 1, tiles, st));
+                    }
+                    m->launches += 1;
+                } else {
+                    CU(cudaMemsetAsync(slot_of, 0xff, (size_t)pairs * 4, st));
+                }
+                if (L.shared_ff > 0 && !parallel) {
+                    // the expert every token uses: its result lands in y and joins the routed sum in the kernel that follows
+                    const int SF = L.ff_plain ? L.shared_ff : 2 * L.shared_ff;
+                    CU(linear<T>(m, hn, static_cast<const T*>(L.w_shared_in), z, Tn, SF, D, st));
+                    gated_act_kernel<T><<<cast_grid((size_t)Tn * L.shared_ff / 4), 256, 0, st>>>(z, L.shared_ff, expert_actp(L), (size_t)Tn, act);
+                    CU(linear<T>(m, act, static_cast<const T*>(L.w_shared_out), y, Tn, D, L.shared_ff, st));
+                    m->launches += 1;
+                }
+                // summed by the norm that follows
+                routed.yp = yp; routed.slot_of = slot_of; routed.sel_w = L.route_input ? nullptr : sel_w; routed.top = L.top_k;
+            }
+            return SMOL_OK;
+        };
+        if (parallel && L.mlp != SMOL_LM_MLP_NONE) {
+            // both sublayers read the same projection: the feed-forward runs on its own stream beside the mixer
+            CU(cudaEventRecord(m->ff_start, st));
+            CU(cudaStreamWaitEvent(m->ff_stream, m->ff_start, 0));
+            const int rc = feed_forward(m->ff_stream);
+            if (rc != SMOL_OK) return rc;
+            CU(cudaEventRecord(m->ff_done, m->ff_stream));
+        }
         if (pairable(L)) {
             int rc = run_mixer(L, R, proj, L.in_bias, mix, own_proj ? mix_cols_of(L) : mix_ld);
             if (rc == SMOL_OK && L.side) {
@@ -2453,122 +2662,25 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             m->launches += 3;
             mix_cols = L.heads * L.dim;
         }
+        if (parallel && L.mlp != SMOL_LM_MLP_NONE) CU(cudaStreamWaitEvent(st, m->ff_done, 0));      // also: w_out covers the shared expert's unit
         CU(linear<T>(m, mix_in, static_cast<const T*>(L.w_out), y, Tn, D, mix_cols, st));
         if (own_proj) CU(linear<T>(m, mix2, static_cast<const T*>(L.side->w_out), y2, Tn, D, mix_cols_of(*L.side), st));
         const bool last = n + 1 == m->runs.size();
         const float* next_norm1 = last ? nullptr : m->layers[m->runs[n + 1].layer].norm1;
-        // the feed-forward reads hn and leaves its output in y (routed experts under the post-norm block: in `routed`)
-        RoutedSum routed;
-        routed.yp = nullptr; routed.slot_of = nullptr; routed.sel_w = nullptr; routed.top = 0;
-        const RoutedSum no_sum = routed;
-        auto actp_of = [](const SmolLmLayer& M) { return ActParams{M.mlp_act, M.act_limit, M.act_alpha, 0}; };
-        // the experts (and a shared expert) of a routed feed-forward may lack gate rows
-        auto expert_actp = [](const SmolLmLayer& M) { return ActParams{M.mlp_act, M.act_limit, M.act_alpha, M.ff_plain ? 1 : 0}; };
-        auto feed_forward = [&]() -> int {
-            if (L.mlp == SMOL_LM_MLP_POLYNORM) {
-                CU(linear<T>(m, hn, static_cast<const T*>(L.w_up), z, Tn, L.ff, D, st));
-                polynorm_kernel<T><<<Tn, 256, 0, st>>>(z, L.act, c.norm_eps, L.ff, act);
-                CU(linear<T>(m, act, static_cast<const T*>(L.w_down), y, Tn, D, L.ff, st));
-                m->launches += 1;
-            } else if (L.mlp == SMOL_LM_MLP_GATED) {
-                CU(linear<T>(m, hn, static_cast<const T*>(L.w_up), z, Tn, 2 * L.ff, D, st));
-                gated_act_kernel<T><<<cast_grid((size_t)Tn * L.ff / 4), 256, 0, st>>>(z, L.ff, actp_of(L), (size_t)Tn, act);
-                CU(linear<T>(m, act, static_cast<const T*>(L.w_down), y, Tn, D, L.ff, st));
-                m->launches += 1;
-            } else if (L.mlp == SMOL_LM_MLP_EXPERTS) {
-                int32_t* sel_id = reinterpret_cast<int32_t*>(m->ws + m->o_sel_id);
-                float* sel_w = reinterpret_cast<float*>(m->ws + m->o_sel_w);
-                int32_t* perm = reinterpret_cast<int32_t*>(m->ws + m->o_perm);
-                int32_t* slot_of = reinterpret_cast<int32_t*>(m->ws + m->o_slot_of);
-                int32_t* seg = reinterpret_cast<int32_t*>(m->ws + m->o_seg);
-                int32_t* tile_g = reinterpret_cast<int32_t*>(m->ws + m->o_tile_g);
-                int32_t* tile_r = reinterpret_cast<int32_t*>(m->ws + m->o_tile_r);
-                int32_t* n_tiles = reinterpret_cast<int32_t*>(m->ws + m->o_ntiles);
-                float* zp = reinterpret_cast<float*>(m->ws + m->o_zp);
-                T* actp = reinterpret_cast<T*>(m->ws + m->o_actp);
-                float* yp = reinterpret_cast<float*>(m->ws + m->o_yp);
-                RouteArgs Rt;
-                Rt.w_router = L.w_router; Rt.bias = L.route_bias; Rt.D = D; Rt.E = L.n_experts + L.n_identity; Rt.E_real = L.n_experts;
-                Rt.top = L.top_k; Rt.n_groups = L.n_groups; Rt.keep = L.keep_groups; Rt.scale = L.router_scale; Rt.n_tokens = Tn;
-                Rt.score = L.router_score; Rt.plain = L.router_plain; Rt.group_top = L.group_rank_top;
-                const int pairs = Tn * L.top_k;
-                // the router reads the sublayer's input in fp32 where the block keeps it (post-norm), else its T form
-                float* r_logits = reinterpret_cast<float*>(m->ws + m->o_rlogits);
-                int32_t* r_done = reinterpret_cast<int32_t*>(m->ws + m->o_rdone);
-                const dim3 rgrid(Tn, (Rt.E + 3) / 4);
-                if (postnorm) moe_route_kernel<float><<<rgrid, 128, 0, st>>>(Rt, x, r_logits, r_done, sel_id, sel_w);
-                else moe_route_kernel<T><<<rgrid, 128, 0, st>>>(Rt, hn, r_logits, r_done, sel_id, sel_w);
-                m->launches += 1;
-                if (L.n_experts > 0) {
-                    // three forms of the two grouped products, by how many rows an expert gets: a warp per output column for
-                    // a handful of pairs (decoding), 32-row mma.sync tiles, 128-row tcgen05 tiles over rows copied into sorted order
-                    const int NF = L.ff_plain ? L.ff : 2 * L.ff;          // rows of an expert's first matrix
-                    const bool few = !kIsF32 && pairs <= kMoeGemvPairs && D % 8 == 0 && L.ff % 8 == 0;
-                    const bool big = !kIsF32 && !few && m->tc_ready && pairs / L.n_experts >= 64 && D % 8 == 0 && L.ff % 8 == 0 &&
-                                     NF >= kTcTileN && D >= kTcTileN && D >= smol::umma::kBK && L.ff >= smol::umma::kBK;
-                    const int tile_rows = big ? smol::umma::kM : kGroupTile;
-                    moe_index_kernel<<<1, 256, 0, st>>>(sel_id, pairs, L.n_experts, tile_rows, seg, perm, slot_of, tile_g, tile_r, n_tiles);
-                    const int tiles = pairs / kGroupTile + L.n_experts;
-                    GemmIo io = plain_io(D, NF);
-                    io.sw = (long long)NF * D;
-                    io.tile_group = tile_g; io.tile_row0 = tile_r; io.seg = seg; io.n_tiles = n_tiles;
-                    GemmIo io2 = plain_io(L.ff, D);
-                    io2.sw = (long long)D * L.ff;
-                    io2.tile_group = tile_g; io2.tile_row0 = tile_r; io2.seg = seg; io2.n_tiles = n_tiles;
-                    const size_t act_n = (size_t)pairs * L.ff;
-                    // a router whose weight multiplies the expert's input: the rows are copied into sorted order, each times
-                    // its weight, and the products read that copy
-                    T* ap = reinterpret_cast<T*>(m->ws + m->o_ap);
-                    if (L.route_input) {
-                        moe_gather_scaled_kernel<T><<<pairs, 128, 0, st>>>(hn, perm, L.top_k, sel_w, seg + L.n_experts, D, ap);
-                        m->launches++;
-                    }
-                    if (few) {
-                        moe_gemv_kernel<false><<<dim3((NF + 7) / 8, pairs), 256, 0, st>>>(L.route_input ? ap : hn, perm, L.route_input ? 0 : L.top_k, sel_id,
-                                                                                         seg + L.n_experts, reinterpret_cast<const bf16*>(L.w_experts_in), io.sw,
-                                                                                         zp, NF, D, expert_actp(L));
-                        // the second product applies the activation as it reads the first one's result
-                        moe_gemv_kernel<true><<<dim3((D + 7) / 8, pairs), 256, 0, st>>>(zp, perm, 0, sel_id, seg + L.n_experts,
-                                                                                        reinterpret_cast<const bf16*>(L.w_experts_out), io2.sw, yp, D, L.ff, expert_actp(L));
-                        m->launches += 1;
-                    } else {
-                        bool done = false;
-                        if (big) {
-                            if (!L.route_input) {
-                                moe_gather_kernel<<<pairs, 128, 0, st>>>(reinterpret_cast<const bf16*>(hn), perm, L.top_k, seg + L.n_experts, D,
-                                                                         reinterpret_cast<bf16*>(ap));
-                                m->launches++;
-                            }
-                            done = linear_grouped_tc(m, reinterpret_cast<const bf16*>(ap), reinterpret_cast<const bf16*>(L.w_experts_in), zp, pairs, L.n_experts,
-                                                     NF, D, io, st);
-                        }
-                        if (!done) {
-                            if (!L.route_input) { io.gather = perm; io.gather_div = L.top_k; }
-                            CU(linear_ex<T>(m, L.route_input ? ap : hn, static_cast<const T*>(L.w_experts_in), zp, pairs, NF, D, io, 1, tiles, st));
-                        }
-                        gated_act_kernel<T><<<cast_grid(act_n / 4), 256, 0, st>>>(zp, L.ff, expert_actp(L), (size_t)pairs, actp);
-                        if (!(big && linear_grouped_tc(m, reinterpret_cast<const bf16*>(actp), reinterpret_cast<const bf16*>(L.w_experts_out), yp, pairs,
-                                                       L.n_experts, D, L.ff, io2, st)))
-                            CU(linear_ex<T>(m, actp, static_cast<const T*>(L.w_experts_out), yp, pairs, D, L.ff, io2, 1, tiles, st));
-                    }
-                    m->launches += 2;
-                } else {
-                    CU(cudaMemsetAsync(slot_of, 0xff, (size_t)pairs * 4, st));
-                }
-                if (L.shared_ff > 0) {
-                    // the expert every token uses: its result lands in y and joins the routed sum in the kernel that follows
-                    const int SF = L.ff_plain ? L.shared_ff : 2 * L.shared_ff;
-                    CU(linear<T>(m, hn, static_cast<const T*>(L.w_shared_in), z, Tn, SF, D, st));
-                    gated_act_kernel<T><<<cast_grid((size_t)Tn * L.shared_ff / 4), 256, 0, st>>>(z, L.shared_ff, expert_actp(L), (size_t)Tn, act);
-                    CU(linear<T>(m, act, static_cast<const T*>(L.w_shared_out), y, Tn, D, L.shared_ff, st));
-                    m->launches += 1;
-                }
-                // summed by the norm that follows
-                routed.yp = yp; routed.slot_of = slot_of; routed.sel_w = L.route_input ? nullptr : sel_w; routed.top = L.top_k;
-            }
-            return SMOL_OK;
-        };
-        if (prenorm) {
+        if (parallel) {
+            // x += m * (mixer and shared expert, one output product; routed experts' sum); the traced row, then either the next
+            // run's norm or the row of a merging run
+            const SmolLmLayer* Ln = last ? nullptr : &m->layers[m->runs[n + 1].layer];
+            const bool merge = !last && (m->runs[n + 1].flags & SMOL_LM_RUN_MERGE_EMBED);
+            ResidualArgs Ra;
+            Ra.x = x; Ra.D = D; Ra.eps = c.norm_eps;
+            Ra.y = y; Ra.y_w = Ra.y2 = Ra.y2_w = nullptr; Ra.sy = c.residual_mult; Ra.sy2 = 0.0f;
+            Ra.rs = routed; Ra.s_routed = c.residual_mult;
+            Ra.trace = s->trace ? s->trace + n * (size_t)Tn * D : nullptr; Ra.x0 = nullptr; Ra.cat = merge ? cat : nullptr;
+            Ra.next = (Ln && !merge) ? norm_of(Ln->norm1, Ln->norm1_shift, Ln->norm1_alpha) : no_norm;
+            residual_norm_kernel<T><<<Tn, nthr, D * sizeof(float), st>>>(Ra, hn, hn);
+            m->launches += 1;
+        } else if (prenorm) {
             // x += mixer (mixers with their own projections: each normed over the width first); x += feed-forward.  The kernel
             // that ends the layer also leaves the traced row, restarts the stream where the next run asks for it and applies
             // the next layer's first norm.
@@ -2581,13 +2693,13 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             Ra.x = x; Ra.D = D; Ra.eps = c.norm_eps;
             Ra.y = y; Ra.y_w = own_proj ? L.proj_norm : nullptr; Ra.sy = own_proj ? L.mix_scale : 1.0f;
             Ra.y2 = own_proj ? y2 : nullptr; Ra.y2_w = own_proj ? L.side->proj_norm : nullptr; Ra.sy2 = own_proj ? L.side->mix_scale : 0.0f;
-            Ra.rs = no_sum;
+            Ra.rs = no_sum; Ra.s_routed = 1.0f; Ra.cat = nullptr;
             Ra.trace = has_ff ? nullptr : tr_row; Ra.x0 = has_ff ? nullptr : restart;
             Ra.next = has_ff ? norm_of(L.norm2, L.norm2_shift, L.norm2_alpha) : after;
             residual_norm_kernel<T><<<Tn, nthr, D * sizeof(float), st>>>(Ra, hn, hn);
             m->launches += 1;
             if (has_ff) {
-                const int rc = feed_forward();
+                const int rc = feed_forward(st);
                 if (rc != SMOL_OK) return rc;
                 const bool summed = routed.yp != nullptr;
                 Ra.y = (!summed || L.shared_ff > 0) ? y : nullptr; Ra.y_w = nullptr; Ra.sy = 1.0f;
@@ -2605,7 +2717,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
                                                                       hist_stride, (int)n + 2, L.depth_mix, nullptr, hn, no_sum);
             m->launches += 1;
             if (has_ff) {
-                const int rc = feed_forward();
+                const int rc = feed_forward(st);
                 if (rc != SMOL_OK) return rc;
                 post_norm_kernel<T><<<Tn, nthr, 2 * D * sizeof(float), st>>>(x, y, c.residual_alpha, L.norm2, c.norm_eps, D, hist, hist_stride,
                                                                           (int)n + 2, L.depth_mix, nullptr, hn, routed);
@@ -2613,7 +2725,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             }
         } else if (L.mlp != SMOL_LM_MLP_NONE) {
             add_norm_kernel<T><<<Tn, nthr, D * sizeof(float), st>>>(x, y, L.norm1b, L.ls1, L.norm2, c.norm_eps, D, hn, woff, L.out_bias, no_sum, hn);
-            const int rc = feed_forward();
+            const int rc = feed_forward(st);
             if (rc != SMOL_OK) return rc;
             add_norm_kernel<T><<<Tn, nthr, D * sizeof(float), st>>>(x, y, L.norm2b, L.ls2, next_norm1, c.norm_eps, D, hn, woff, nullptr, routed, hn);
             m->launches += 2;
@@ -2621,17 +2733,18 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             add_norm_kernel<T><<<Tn, nthr, D * sizeof(float), st>>>(x, y, L.norm1b, L.ls1, next_norm1, c.norm_eps, D, hn, woff, L.out_bias, no_sum, hn);
             m->launches += 1;
         }
-        if (s->trace && !prenorm) CU(cudaMemcpyAsync(s->trace + n * (size_t)Tn * D, x, (size_t)Tn * D * 4, cudaMemcpyDeviceToDevice, st));
+        if (s->trace && !prenorm && !parallel) CU(cudaMemcpyAsync(s->trace + n * (size_t)Tn * D, x, (size_t)Tn * D * 4, cudaMemcpyDeviceToDevice, st));
     }
     if (s->n_want > 0) {
         if (postnorm) post_norm_kernel<T><<<s->n_want, nthr, 2 * D * sizeof(float), st>>>(x, nullptr, c.logit_scale, m->g.final_norm, c.norm_eps, D, nullptr, 0, 0,
                                                                                       nullptr, s->want_rows, hw, RoutedSum{nullptr, nullptr, nullptr, 0});
-        else if (prenorm) prenorm_rows_kernel<T><<<s->n_want, nthr, 0, st>>>(x, s->want_rows, norm_of(m->g.final_norm, m->g.final_norm_shift, m->g.final_norm_alpha), D, hw);
+        else if (prenorm || parallel) prenorm_rows_kernel<T><<<s->n_want, nthr, 0, st>>>(x, s->want_rows, norm_of(m->g.final_norm, m->g.final_norm_shift, m->g.final_norm_alpha), D, hw);
         else norm_rows_kernel<T><<<s->n_want, nthr, 0, st>>>(x, s->want_rows, m->g.final_norm, c.norm_eps, D, hw, woff);
         m->launches++;
         CU(linear<T>(m, hw, static_cast<const T*>(m->g.head), s->logits, s->n_want, c.vocab, D, st));
-        if (!postnorm && c.logit_scale != 1.0f) {
-            scale_kernel<<<cast_grid((size_t)s->n_want * c.vocab), 256, 0, st>>>(s->logits, c.logit_scale, (size_t)s->n_want * c.vocab);
+        const float lscale = postnorm ? 1.0f : c.logit_scale;      // the post-norm block scales inside the final norm
+        if (lscale != 1.0f || c.logit_softcap > 0.0f) {
+            logit_finish_kernel<<<cast_grid((size_t)s->n_want * c.vocab), 256, 0, st>>>(s->logits, lscale, c.logit_softcap, (size_t)s->n_want * c.vocab);
             m->launches++;
         }
     }

@@ -215,10 +215,6 @@ __global__ void post_norm_kernel(float* __restrict__ x, const float* __restrict_
     }
 }
 
-__global__ void scale_kernel(float* __restrict__ v, float scale, size_t n) {
-    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) v[i] *= scale;
-}
-
 // ---------------------------------------------------------------------------------------------------------------------
 // Latent attention.  proj row layout: query latent [q_rank] | key/value latent [kv_rank] | shared rotated key [rot] | gate [H].
 // A cached position is ONE row [kv_rank + rot]: the normed latent, then the rotated key part.  Attention runs in the
@@ -321,9 +317,10 @@ struct GlaArgs {
     // heads share one query / key vector), v_src[t * v_ld + h * dv + j].  The gated linear recurrence reads them from proj.
     const float *q_src, *k_src, *v_src;
     int q_ld, k_ld, v_ld, qk_share;
-    // SCALAR form of the scan: one decay per (token, head) head_decay[t * H + h] instead of one per key channel, and the
-    // value is multiplied by head_step[t * H + h] as it enters the state.
+    // SCALAR form of the scan: one decay per (token, head) head_decay[t * head_ld + h] instead of one per key channel (head_ld
+    // 0: a constant per head), and the value is multiplied by head_step[t * head_ld + h] as it enters the state (nullptr: 1).
     const float *head_decay, *head_step;
+    int head_ld;
     int out_ld;                                        // row stride of the finished mixer output
     float out_scale;
 };
@@ -332,6 +329,7 @@ __host__ __device__ inline void gla_sources_from_proj(GlaArgs& A) {
     A.q_ld = A.k_ld = A.v_ld = A.n_in;
     A.qk_share = 1;
     A.head_decay = A.head_step = nullptr;
+    A.head_ld = A.H;
     A.out_ld = A.H * A.dv;
     A.out_scale = 1.0f;
 }
@@ -381,8 +379,9 @@ __device__ __forceinline__ void gla_stage(const GlaArgs& A, float* buf, int c0, 
     if (SCALAR) {
         float* sc = buf + 3 * PL + kDeltaChunk * CB;
         for (int tt = threadIdx.x; tt < n; tt += blockDim.x) {
-            cp_async_f<1>(sc + tt, A.head_decay + (size_t)(c0 + tt) * A.H + h);
-            cp_async_f<1>(sc + kDeltaChunk + tt, A.head_step + (size_t)(c0 + tt) * A.H + h);
+            cp_async_f<1>(sc + tt, A.head_decay + (size_t)(c0 + tt) * A.head_ld + h);
+            if (A.head_step) cp_async_f<1>(sc + kDeltaChunk + tt, A.head_step + (size_t)(c0 + tt) * A.head_ld + h);
+            else sc[kDeltaChunk + tt] = 1.0f;
         }
     }
 }
@@ -499,7 +498,7 @@ __global__ void __launch_bounds__(gla_block_cols(DK) * gla_lanes(DK)) gla_scan_k
 }
 
 // End of the mixer: each head's o divided by its root mean square over dv, times the plain weight [dv] (shared by the
-// heads), times silu(gate), written in T.  One warp per (token, head).
+// heads; nullptr: none), times silu(gate), written in T.  One warp per (token, head).
 template <class T>
 __global__ void gla_out_kernel(const GlaArgs A, const float* __restrict__ o_raw, T* __restrict__ out) {
     const int lane = threadIdx.x & 31;
@@ -512,7 +511,7 @@ __global__ void gla_out_kernel(const GlaArgs A, const float* __restrict__ o_raw,
     for (int c = lane; c < dv; c += 32) ss = fmaf(o[c], o[c], ss);
     ss = warp_sum(ss);
     const float rs = 1.0f / sqrtf(ss / (float)dv + A.eps);
-    for (int c = lane; c < dv; c += 32) out[(size_t)t * A.out_ld + h * dv + c] = from_f<T>(o[c] * rs * A.out_norm[c] * silu_(gate[c]) * A.out_scale);
+    for (int c = lane; c < dv; c += 32) out[(size_t)t * A.out_ld + h * dv + c] = from_f<T>(o[c] * rs * (A.out_norm ? A.out_norm[c] : 1.0f) * silu_(gate[c]) * A.out_scale);
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
@@ -678,9 +677,22 @@ struct RouteArgs {
     int D, E, E_real, top, n_groups, keep;
     float scale;
     int n_tokens;
-    int score;        // SMOL_LM_ROUTE_*: softmax over the outputs, or a sigmoid of each
+    int score;        // SMOL_LM_ROUTE_*: softmax over the outputs, a sigmoid of each, or the softmax over the chosen ones
     int plain;        // 1: a chosen output's weight is its score (times scale), not divided by the chosen scores' sum
     int group_top;    // a group is ranked by the sum of its group_top best choice scores (at most 1: by its best)
+    const float* logit_bias;           // added to the logits themselves [E] (nullptr: none)
+    // the logits as an earlier product left them, row t at given + t * given_ld (nullptr: the kernel takes the dot products)
+    const float* given;
+    int given_ld;
+    // few pairs (decoding): the pairs keep their order, perm and slot_of are the identity and *n_sorted the number of pairs, so
+    // that no sorting kernel is needed (perm == nullptr: not asked for; only without identity outputs)
+    int32_t *perm, *slot_of, *n_sorted;
+    // a shared expert whose gate and up values lie beside the logits: the unit's value times sigmoid(unit_gate[t * given_ld])
+    // (nullptr: 1) -> unit_out[t * unit_ld + c] in TI, c < unit_ff (0: none)
+    const float *unit_in, *unit_gate;
+    void* unit_out;
+    int unit_ff, unit_ld;
+    ActParams unit_act;
 };
 constexpr int kMaxRouted = 1024;       // router outputs (experts + identity outputs)
 constexpr int kMaxTop = 32;
@@ -691,6 +703,8 @@ constexpr int kMaxTop = 32;
 // group's score: its best choice score) cannot be chosen; the `top` best choice scores are chosen (ties: the lower
 // index; the choices are kept in that order), their weights are the scores s over their sum, times `scale`.  Ranks are
 // counted, not sorted: output e is chosen if fewer than `top` allowed outputs beat it.
+// SMOL_LM_ROUTE_CHOSEN: the choice score is the logit, and the weights are the softmax over the chosen logits.
+// With logits given by an earlier product there is one block per token (gridDim.y = 1), which also leaves the shared expert's unit.
 template <class TI>
 __global__ void __launch_bounds__(128) moe_route_kernel(const RouteArgs A, const TI* __restrict__ x, float* __restrict__ logits,
                                                         int32_t* __restrict__ done, int32_t* __restrict__ sel_id, float* __restrict__ sel_w) {
@@ -701,7 +715,14 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const RouteArgs A, const
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
     const TI* xr = x + (size_t)t * A.D;
     const int e0 = blockIdx.y * nw + warp;
-    if (e0 < A.E) {
+    if (A.unit_ff > 0) {
+        const float* u = A.unit_in + (size_t)t * A.given_ld;
+        const float gate = A.unit_gate ? sigmoidf_(A.unit_gate[(size_t)t * A.given_ld]) : 1.0f;
+        const int uo = A.unit_act.plain ? 0 : A.unit_ff;
+        TI* out = static_cast<TI*>(A.unit_out) + (size_t)t * A.unit_ld;
+        for (int c = threadIdx.x; c < A.unit_ff; c += blockDim.x) out[c] = from_f<TI>(gate * gated_unit_(A.unit_act, u[c], u[uo + c]));
+    }
+    if (!A.given && e0 < A.E) {
         const float* wr = A.w_router + (size_t)e0 * A.D;
         float acc = 0.0f;
         if (sizeof(TI) == 4 && A.D % 4 == 0) {          // rows of x and of the router start on 16-byte boundaries
@@ -719,19 +740,22 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const RouteArgs A, const
         acc = warp_sum(acc);
         if (lane == 0) logits[(size_t)t * A.E + e0] = acc;
     }
-    __threadfence();
-    __syncthreads();
-    if (threadIdx.x == 0) {
-        const int ticket = atomicAdd(&done[t], 1);
-        last = ticket == (int)gridDim.y - 1;
-        if (last) done[t] = 0;
+    if (!A.given) {
+        __threadfence();
+        __syncthreads();
+        if (threadIdx.x == 0) {
+            const int ticket = atomicAdd(&done[t], 1);
+            last = ticket == (int)gridDim.y - 1;
+            if (last) done[t] = 0;
+        }
+        __syncthreads();
+        if (!last) return;
+        __threadfence();
     }
-    __syncthreads();
-    if (!last) return;
-    __threadfence();
+    const float* lg = A.given ? A.given + (size_t)t * A.given_ld : logits + (size_t)t * A.E;
     float mx = -INFINITY;
     for (int e = threadIdx.x; e < A.E; e += blockDim.x) {
-        const float v = __ldcg(logits + (size_t)t * A.E + e);
+        const float v = __ldcg(lg + e) + (A.logit_bias ? A.logit_bias[e] : 0.0f);
         s[e] = v;
         mx = fmaxf(mx, v);
     }
@@ -746,9 +770,10 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const RouteArgs A, const
         sum = block_sum(sum, red);
     }
     for (int e = threadIdx.x; e < A.E; e += blockDim.x) {
-        const float p = A.score == SMOL_LM_ROUTE_SOFTMAX ? expf(s[e] - mx) / sum : sigmoidf_(s[e]);
+        const float v = s[e];
+        const float p = A.score == SMOL_LM_ROUTE_SIGMOID ? sigmoidf_(v) : A.score == SMOL_LM_ROUTE_SOFTMAX ? expf(v - mx) / sum : expf(v - mx);
         s[e] = p;
-        choice[e] = p + (A.bias ? A.bias[e] : 0.0f);
+        choice[e] = (A.score == SMOL_LM_ROUTE_CHOSEN ? v : p) + (A.bias ? A.bias[e] : 0.0f);
     }
     __syncthreads();
     const int size = A.E / A.n_groups;
@@ -793,7 +818,12 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const RouteArgs A, const
     if (threadIdx.x < A.top) {
         float den = 0.0f;
         for (int k = 0; k < A.top; ++k) den += top_s[k];
-        sel_w[(size_t)t * A.top + threadIdx.x] = A.plain ? top_s[threadIdx.x] * A.scale : top_s[threadIdx.x] / (den + 1e-20f) * A.scale;
+        const size_t pair = (size_t)t * A.top + threadIdx.x;
+        sel_w[pair] = A.plain ? top_s[threadIdx.x] * A.scale : top_s[threadIdx.x] / (den + 1e-20f) * A.scale;
+        if (A.perm) {
+            A.perm[pair] = A.slot_of[pair] = (int32_t)pair;
+            if (pair == 0) *A.n_sorted = A.n_tokens * A.top;
+        }
     }
 }
 

@@ -3,8 +3,11 @@
 //     x + embedding output, and mixers side by side that are each projected, RMS-normed over the width and summed,
 //   - sigmoid attention (no softmax: weight = sigmoid(score + head bias); the heads' weight maps mixed by a matrix;
 //     chunked mask; rotated, norm-divided queries and keys; the values are the key projection),
-//   - the front and back ends of two linear attentions that run on the gated linear recurrence's scan: lightning
-//     attention (constant decay per head) and HGRN2 (the forget gate is the decay, one minus it the key).
+//   - the parallel block  x += m (mixer(h) + feed-forward(h)), h = norm(x),  with a layer norm, and runs that start from a
+//     matrix applied to [x; embedding output],
+//   - the front and back ends of three linear attentions that run on the gated linear recurrence's scan: lightning
+//     attention (constant decay per head), HGRN2 (the forget gate is the decay, one minus it the key) and retention
+//     (constant decay per head, rotated queries and keys).
 // Everything here is fp32 except what is written for a matrix product or into the key/value pool (T).
 #pragma once
 
@@ -12,7 +15,8 @@ namespace smol {
 namespace lm {
 
 // ---------------------------------------------------------------------------------------------------------------------
-// Norms of the pre-norm block.  RMS: v / rms(row) * w.  Dynamic Tanh: tanh(alpha v) * w + shift, element by element.
+// Norms of the pre-norm and the parallel block.  RMS: v / rms(row) * w.  Dynamic Tanh: tanh(alpha v) * w + shift, element by
+// element.  Layer norm: (v - mean) / sqrt(variance + eps) * w + shift, the variance taken from the deviations themselves.
 struct NormSpec {
     int kind;                         // SMOL_LM_NORM_*
     const float *w, *shift, *alpha;   // w == nullptr: no norm follows
@@ -20,11 +24,50 @@ struct NormSpec {
 };
 __device__ __forceinline__ float dyt_(const NormSpec& n, float alpha, float v, int c) { return fmaf(tanhf(alpha * v), n.w[c], n.shift[c]); }
 
+// The layer norm of a row on its way to T: value(c) gives element c (read twice where the row does not fit the registers).
+template <class T, class Value>
+__device__ __forceinline__ void layer_norm_row(const NormSpec& nm, int D, T* __restrict__ out, float* red, Value value) {
+    if (D <= (int)blockDim.x * kRowRegs) {
+        float v[kRowRegs], w[kRowRegs], b[kRowRegs];
+        float s = 0.0f;
+#pragma unroll
+        for (int i = 0; i < kRowRegs; ++i) {
+            const int c = threadIdx.x + i * blockDim.x;
+            const bool in = c < D;
+            v[i] = in ? value(c) : 0.0f;
+            w[i] = in ? nm.w[c] : 0.0f;
+            b[i] = in ? nm.shift[c] : 0.0f;
+            s += v[i];
+        }
+        const float mean = block_sum(s, red) / (float)D;
+        float q = 0.0f;
+#pragma unroll
+        for (int i = 0; i < kRowRegs; ++i) {
+            v[i] -= mean;
+            if ((int)(threadIdx.x + i * blockDim.x) < D) q = fmaf(v[i], v[i], q);
+        }
+        const float r = 1.0f / sqrtf(block_sum(q, red) / (float)D + nm.eps);
+#pragma unroll
+        for (int i = 0; i < kRowRegs; ++i) {
+            const int c = threadIdx.x + i * blockDim.x;
+            if (c < D) out[c] = from_f<T>(fmaf(v[i] * r, w[i], b[i]));
+        }
+        return;
+    }
+    float s = 0.0f, q = 0.0f;
+    for (int c = threadIdx.x; c < D; c += blockDim.x) s += value(c);
+    const float mean = block_sum(s, red) / (float)D;
+    for (int c = threadIdx.x; c < D; c += blockDim.x) { const float v = value(c) - mean; q = fmaf(v, v, q); }
+    const float r = 1.0f / sqrtf(block_sum(q, red) / (float)D + nm.eps);
+    for (int c = threadIdx.x; c < D; c += blockDim.x) out[c] = from_f<T>(fmaf((value(c) - mean) * r, nm.w[c], nm.shift[c]));
+}
+
 // x[t] = embed[token[t]] * scale, kept a second time in x0 (nullptr: not needed) for the passes that restart from it;
-// hn = norm(x[t]).
+// hn = norm(x[t]).  `cat` (nullptr: not needed) holds the rows [stream | embedding output] in T that a merging run multiplies:
+// both halves start as the embedding output; nm.w == nullptr: the first run merges, its norm comes after that product.
 template <class T>
 __global__ void embed_prenorm_kernel(const int32_t* __restrict__ tokens, const T* __restrict__ embed, float scale, int D, int vocab,
-                                     const NormSpec nm, float* __restrict__ x, float* __restrict__ x0, T* __restrict__ hn) {
+                                     const NormSpec nm, float* __restrict__ x, float* __restrict__ x0, T* __restrict__ hn, T* __restrict__ cat) {
     __shared__ float red[33];
     const int t = blockIdx.x;
     int tok = tokens[t];
@@ -37,10 +80,15 @@ __global__ void embed_prenorm_kernel(const int32_t* __restrict__ tokens, const T
         const float v = to_f<T>(e[c]) * scale;
         x[o + c] = v;
         if (x0) x0[o + c] = v;
+        if (cat) cat[2 * o + c] = cat[2 * o + D + c] = from_f<T>(v);
         if (nm.kind == SMOL_LM_NORM_DYT) hn[o + c] = from_f<T>(dyt_(nm, alpha, v, c));
         ss += v * v;
     }
-    if (nm.kind == SMOL_LM_NORM_DYT) return;
+    if (nm.kind == SMOL_LM_NORM_DYT || !nm.w) return;
+    if (nm.kind == SMOL_LM_NORM_LAYER) {
+        layer_norm_row<T>(nm, D, hn + o, red, [&](int c) { return x[o + c]; });      // a thread reads what it wrote itself
+        return;
+    }
     ss = block_sum(ss, red);
     const float r = 1.0f / sqrtf(ss / (float)D + nm.eps);
     for (int c = threadIdx.x; c < D; c += blockDim.x) hn[o + c] = from_f<T>(x[o + c] * r * nm.w[c]);
@@ -57,6 +105,10 @@ __global__ void prenorm_rows_kernel(const float* __restrict__ x, const int32_t* 
         for (int c = threadIdx.x; c < D; c += blockDim.x) out[o + c] = from_f<T>(dyt_(nm, alpha, xr[c], c));
         return;
     }
+    if (nm.kind == SMOL_LM_NORM_LAYER) {
+        layer_norm_row<T>(nm, D, out + o, red, [&](int c) { return xr[c]; });
+        return;
+    }
     float ss = 0.0f;
     for (int c = threadIdx.x; c < D; c += blockDim.x) ss += xr[c] * xr[c];
     ss = block_sum(ss, red);
@@ -64,11 +116,13 @@ __global__ void prenorm_rows_kernel(const float* __restrict__ x, const int32_t* 
     for (int c = threadIdx.x; c < D; c += blockDim.x) out[o + c] = from_f<T>(xr[c] * r * nm.w[c]);
 }
 
-// End of a sublayer of the pre-norm block, fused with the norm in front of the next one.  One block per row:
-//   x <- x + sy * f(y) + sy2 * f2(y2) + (the routed experts' weighted sum)
+// End of a sublayer of the pre-norm block or of a layer of the parallel block, fused with the norm in front of the next one.
+// One block per row:
+//   x <- x + sy * f(y) + sy2 * f2(y2) + s_routed * (the routed experts' weighted sum)
 // where f(y) = y, or y / rms(y) * y_w when y_w is set (mixers side by side: each projected result is normed over the width).
 // `trace` then takes the row (the stream after the sublayer); x0, when set, joins x after that (the next run restarts from
-// stream + embedding output); hn <- next(x).
+// stream + embedding output); hn <- next(x).  `cat`, when set, takes x in T as the first half of the row a merging run
+// multiplies (no norm follows here then).
 struct ResidualArgs {
     float* x;
     int D;
@@ -76,8 +130,10 @@ struct ResidualArgs {
     const float *y, *y_w, *y2, *y2_w;     // y2 == nullptr: one result only; y == nullptr: none at all
     float sy, sy2;
     RoutedSum rs;
+    float s_routed;
     float* trace;
     const float* x0;
+    void* cat;                            // T [rows][2 * D]
     NormSpec next;
 };
 
@@ -91,7 +147,7 @@ __global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn, c
     if (D <= (int)blockDim.x * kRowRegs) {
         // the row in registers: every operand is loaded before the first reduction, so a lone row (decoding) waits for
         // global memory once
-        const bool dyt_r = A.next.w && A.next.kind == SMOL_LM_NORM_DYT;
+        const bool dyt_r = A.next.w && A.next.kind == SMOL_LM_NORM_DYT, layer_r = A.next.w && A.next.kind == SMOL_LM_NORM_LAYER;
         const float alpha_r = dyt_r ? A.next.alpha[0] : 0.0f;
         float xv[kRowRegs], yv[kRowRegs], zv[kRowRegs], a1[kRowRegs], a2[kRowRegs], e0[kRowRegs], nw[kRowRegs], nb[kRowRegs];
 #pragma unroll
@@ -105,12 +161,12 @@ __global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn, c
             a2[i] = (in && A.y2_w) ? A.y2_w[c] : 1.0f;
             e0[i] = (in && A.x0) ? A.x0[o + c] : 0.0f;
             nw[i] = (in && A.next.w) ? A.next.w[c] : 0.0f;
-            nb[i] = (in && dyt_r) ? A.next.shift[c] : 0.0f;
+            nb[i] = (in && (dyt_r || layer_r)) ? A.next.shift[c] : 0.0f;
         }
         if (A.rs.yp) {
             for (int k = 0; k < A.rs.top; ++k) {
                 const int slot = A.rs.slot_of[(size_t)blockIdx.x * A.rs.top + k];
-                const float wk = A.rs.sel_w ? A.rs.sel_w[(size_t)blockIdx.x * A.rs.top + k] : 1.0f;
+                const float wk = A.s_routed * (A.rs.sel_w ? A.rs.sel_w[(size_t)blockIdx.x * A.rs.top + k] : 1.0f);
 #pragma unroll
                 for (int i = 0; i < kRowRegs; ++i) {
                     const int c = threadIdx.x + i * blockDim.x;
@@ -140,10 +196,27 @@ __global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn, c
             v += e0[i];
             A.x[o + c] = v;
             xv[i] = v;
-            ss = fmaf(v, v, ss);
+            ss = layer_r ? ss + v : fmaf(v, v, ss);
+            if (A.cat) static_cast<T*>(A.cat)[2 * o + c] = from_f<T>(v);
             if (dyt_r) hn[o + c] = from_f<T>(fmaf(tanhf(alpha_r * v), nw[i], nb[i]));
         }
         if (!A.next.w || dyt_r) return;
+        if (layer_r) {
+            const float mean = block_sum(ss, red3[0]) / (float)D;
+            float q = 0.0f;
+#pragma unroll
+            for (int i = 0; i < kRowRegs; ++i) {
+                xv[i] -= mean;
+                if ((int)(threadIdx.x + i * blockDim.x) < D) q = fmaf(xv[i], xv[i], q);
+            }
+            const float r = 1.0f / sqrtf(block_sum(q, red3[1]) / (float)D + A.next.eps);
+#pragma unroll
+            for (int i = 0; i < kRowRegs; ++i) {
+                const int c = threadIdx.x + i * blockDim.x;
+                if (c < D) hn[o + c] = from_f<T>(fmaf(xv[i] * r, nw[i], nb[i]));
+            }
+            return;
+        }
         float q2 = 0.0f, q3 = 0.0f;
         block_sum3(ss, q2, q3, red3);
         const float r = 1.0f / sqrtf(ss / (float)D + A.next.eps);
@@ -180,16 +253,21 @@ __global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn, c
                 const float e = slot >= 0 ? A.rs.yp[(size_t)slot * D + c] : to_f<T>(hin[o + c]);
                 acc = fmaf(A.rs.sel_w ? A.rs.sel_w[(size_t)blockIdx.x * A.rs.top + k] : 1.0f, e, acc);
             }
-            v += acc;
+            v = fmaf(A.s_routed, acc, v);
         }
         if (A.trace) A.trace[o + c] = v;
         if (A.x0) v += A.x0[o + c];
         A.x[o + c] = v;
+        if (A.cat) static_cast<T*>(A.cat)[2 * o + c] = from_f<T>(v);
         if (dyt) hn[o + c] = from_f<T>(dyt_(A.next, alpha, v, c));
         else row[c] = v;
         ss = fmaf(v, v, ss);
     }
     if (!A.next.w || dyt) return;
+    if (A.next.kind == SMOL_LM_NORM_LAYER) {
+        layer_norm_row<T>(A.next, D, hn + o, red3[0], [&](int c) { return row[c]; });
+        return;
+    }
     float s2 = 0.0f, s3 = 0.0f;
     block_sum3(ss, s2, s3, red3);
     const float r = 1.0f / sqrtf(ss / (float)D + A.next.eps);
@@ -655,6 +733,49 @@ __global__ void hgrn2_prep_kernel(const LinPrepArgs A, float* __restrict__ qv, f
         qv[(size_t)t * HD + c] = silu_(row[c]);
         decay[(size_t)t * HD + c] = f;
         key[(size_t)t * HD + c] = 1.0f - f;
+    }
+}
+
+// RETENTION: proj rows q | k [H*d each] | v | gate [H*dv each]: qk[t] = the rotated q, then the rotated k times k_scale (row length
+// 2 H d); v and the constant decays go to the scan as they are.  A thread owns the same pair (or unrotated coordinate) of q and k,
+// so an angle is taken once for both.  half: coordinate i is paired with i + pairs, else 2i with 2i + 1.
+struct RetentionArgs {
+    const float* proj;
+    int n_in, H, d, pairs, half;
+    float k_scale;
+    const float* freq;             // [pairs]
+    const int32_t* tok_pos;
+};
+
+__global__ void retention_prep_kernel(const RetentionArgs A, float* __restrict__ qk) {
+    const int t = blockIdx.x, HD = A.H * A.d, per = A.d - A.pairs;
+    const int pos = A.tok_pos[t];
+    const float *q = A.proj + (size_t)t * A.n_in, *k = q + HD;
+    float *qo = qk + (size_t)t * 2 * HD, *ko = qo + HD;
+    for (int u = blockIdx.y * blockDim.x + threadIdx.x; u < A.H * per; u += gridDim.y * blockDim.x) {
+        const int h = u / per, i = u - h * per;
+        if (i < A.pairs) {
+            const int a = h * A.d + (A.half ? i : 2 * i), b = h * A.d + (A.half ? i + A.pairs : 2 * i + 1);
+            float sn, cs;
+            sincosf((float)pos * A.freq[i], &sn, &cs);
+            const float qa = q[a], qb = q[b], ka = k[a], kb = k[b];
+            qo[a] = qa * cs - qb * sn;
+            qo[b] = qb * cs + qa * sn;
+            ko[a] = (ka * cs - kb * sn) * A.k_scale;
+            ko[b] = (kb * cs + ka * sn) * A.k_scale;
+        } else {
+            const int c = h * A.d + A.pairs + i;
+            qo[c] = q[c];
+            ko[c] = k[c] * A.k_scale;
+        }
+    }
+}
+
+// The logits' last step: times scale, then bent to cap * tanh(v / cap) (cap 0: not bent).
+__global__ void logit_finish_kernel(float* __restrict__ v, float scale, float cap, size_t n) {
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+        const float z = v[i] * scale;
+        v[i] = cap > 0.0f ? cap * tanhf(z / cap) : z;
     }
 }
 

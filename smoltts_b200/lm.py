@@ -14,6 +14,10 @@ clamped gated feed-forwards, dense or routed by sigmoid scores; the logits reuse
 passes restart from stream + embedding output; mixers are a pair -- chunked sigmoid attention with mixed heads (keys and
 values in the paged pool) beside lightning attention (state in the slot), each projected and normed on its own -- or
 HGRN2; feed-forwards are gated or routed squared-relu experts with a shared expert.
+``BizulixLM`` serves the Bizulix design: parallel layers (one layer norm, read by mixer and feed-forward, whose sum joins the
+stream), a looped span whose passes start from a matrix applied to [stream; embedding output]; softmax attention with a
+query temperature and soft-capped scores (keys and values in the paged pool) or retention (state in the slot); routed
+gated experts beside a shared expert with one gate per token; soft-capped logits.
 
 The engine owns two pools -- key/value pages (``PagePool``) and state slots (``SlotPool``) -- and one step function,
 ``forward``: any number of sequences, each with its next tokens (a portion of a prompt or a single decoded token).
@@ -34,8 +38,9 @@ import torch
 
 from . import _capi_lm
 from ._errors import SMOL_ERR_CAPACITY, SmolError
-from .lm_config import (ACT_CLAMPED, ACT_GELU_TANH, ACT_RELU_SQUARED, ACT_SILU, BLOCK_POSTNORM, BLOCK_PRENORM, BLOCK_SANDWICH, MAFERAX_MLP_KINDS,
-                        MIXER_KINDS, MLP_KINDS, NORM_DYT, ROUTE_SIGMOID, GuniraxConfig, MaferaxConfig, PamasunConfig, SunutarConfig)
+from .lm_config import (ACT_CLAMPED, ACT_GELU_TANH, ACT_RELU_SQUARED, ACT_SILU, BLOCK_PARALLEL, BLOCK_POSTNORM, BLOCK_PRENORM, BLOCK_SANDWICH,
+                        MAFERAX_MLP_KINDS, MIXER_KINDS, MLP_KINDS, NORM_DYT, NORM_LAYER, ROUTE_CHOSEN, ROUTE_SIGMOID, RUN_ADD_EMBED, RUN_MERGE_EMBED,
+                        BizulixConfig, GuniraxConfig, MaferaxConfig, PamasunConfig, SunutarConfig)
 from .pool import PagePool, SlotPool
 
 _ST_DTYPES = {"BF16": torch.bfloat16, "F16": torch.float16, "F32": torch.float32, "I32": torch.int32, "I64": torch.int64}
@@ -547,6 +552,62 @@ class GuniraxLM(HybridLM):
                     c.shared_ff = L.shared_ff
                     c.w_shared_in, c.w_shared_out = mat(p + "mlp.shared.up").data_ptr(), mat(p + "mlp.shared.down").data_ptr()
         return {"config": {"block": BLOCK_PRENORM, "norm_kind": NORM_DYT, "embed_scale": cfg.embedding_scale},
-                "run_flags": cfg.run_restarts(),
+                "run_flags": [RUN_ADD_EMBED * f for f in cfg.run_restarts()],
                 "globals": {"embed": mat("embed"), "head": mat("head"), "final_norm": vec("final.norm"),
                             "final_norm_shift": vec("final.norm.b"), "final_norm_alpha": vec("final.norm.alpha")}}
+
+
+class BizulixLM(HybridLM):
+    """B200 engine of one Bizulix checkpoint."""
+
+    architecture = "Bizulix"
+    config_class = BizulixConfig
+
+    def _shapes(self, sd):
+        return self.config.tensor_shapes()
+
+    def _describe(self, sd, layers, mat, vec):
+        cfg, D = self.config, self.config.width
+
+        def norm(c, field, name):
+            setattr(c, field, vec(name).data_ptr())
+            setattr(c, field + "_shift", vec(name + ".b").data_ptr())
+
+        for i, L in enumerate(cfg.layers):
+            p, m, c = f"l{i}.", L.mixer, layers[i]
+            norm(c, "norm1", p + "norm1")
+            c.mixer, c.heads, c.dim, c.vdim = MIXER_KINDS[m.kind], m.heads, m.dim, m.vdim
+            # one input product per layer: the mixer's rows, then what the feed-forward needs of the same input
+            rows, cols = [p + "mix.q", p + "mix.k", p + "mix.v"], [sd[p + "mix.o"].float()]
+            if m.kind == "attention":
+                c.kv_heads, c.score_scale, c.softcap, c.no_gate = m.kv_heads, m.scale, m.softcap, 1
+                c.q_temp_coef, c.q_temp_every = m.temp_coef, m.temp_every
+            else:
+                rows.append(p + "mix.g")
+                c.kv_heads, c.score_scale = m.heads, m.dim ** -0.5
+                c.rot_dims, c.rot_base, c.rot_half = m.rot.dims, m.rot.base, 1
+                c.rot_stretch, c.rot_low, c.rot_high, c.rot_original = m.rot.factor, m.rot.low, m.rot.high, m.rot.original
+                c.head_decay = vec(torch.tensor(m.decay, dtype=torch.float32)).data_ptr()
+            c.mlp = MAFERAX_MLP_KINDS["moe" if L.ff else None]
+            if L.ff:
+                c.ff, c.mlp_act = L.ff, ACT_SILU
+                c.n_experts, c.n_identity, c.top_k, c.n_groups, c.keep_groups, c.router_scale = L.experts, 0, L.top, 1, 1, 1.0
+                c.router_score, c.router_bias = ROUTE_CHOSEN, vec(p + "mlp.router.b").data_ptr()
+                c.w_experts_in = mat(*[f"{p}mlp.e{e}.{nm}" for e in range(L.experts) for nm in ("gate", "up")]).data_ptr()
+                c.w_experts_out = mat(*[f"{p}mlp.e{e}.down" for e in range(L.experts)]).data_ptr()
+                if L.shared_ff:
+                    c.shared_ff, c.shared_gate = L.shared_ff, 1
+                    rows += [p + "mlp.shared.gate", p + "mlp.shared.up"]
+                    cols.append(sd[p + "mlp.shared.down"].float())
+                rows.append(p + "mlp.router")
+                if L.shared_ff:
+                    rows.append(p + "mlp.shared.sg")
+            n_in = sum(int(sd[r].shape[0]) for r in rows)
+            if n_in % 8:
+                rows.append(torch.zeros(8 - n_in % 8, D))
+            c.w_in, c.w_out = mat(*rows).data_ptr(), mat(torch.cat(cols, 1)).data_ptr()
+        g = {"embed": mat("embed"), "head": mat("head"), "final_norm": vec("final.norm"), "final_norm_shift": vec("final.norm.b")}
+        if cfg.looped:
+            g["w_merge"] = mat("loop.in")
+        return {"config": {"block": BLOCK_PARALLEL, "norm_kind": NORM_LAYER, "residual_mult": cfg.residual_mult, "logit_softcap": cfg.logit_softcap},
+                "run_flags": [RUN_MERGE_EMBED * f for f in cfg.run_merges()], "globals": g}

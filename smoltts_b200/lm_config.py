@@ -15,14 +15,15 @@ from typing import Any, Dict, List, Optional
 
 # values of SMOL_LM_MIX_* (include/smoltts_b200_lm.h)
 MIXER_KINDS = {"attention": 0, "general_delta": 1, "latent_attention": 2, "gla": 3, "state_space": 4, "sigmoid_attention": 5,
-               "lightning": 6, "hgrn2": 7}
+               "lightning": 6, "hgrn2": 7, "retention": 8}
 MLP_KINDS = {None: 0, "dense": 1}                        # SMOL_LM_MLP_* of Pamasun: "dense" = up, PolyNorm, down
 # SMOL_LM_MLP_* of Maferax: "dense" = gated (tanh-form gelu), "moe" = routed mixture of gated (silu) experts
 MAFERAX_MLP_KINDS = {None: 0, "dense": 2, "moe": 3}
 ACT_GELU_TANH, ACT_SILU, ACT_CLAMPED, ACT_RELU_SQUARED = 0, 1, 2, 3      # SMOL_LM_ACT_*
-ROUTE_SOFTMAX, ROUTE_SIGMOID = 0, 1                      # SMOL_LM_ROUTE_*
-BLOCK_SANDWICH, BLOCK_POSTNORM, BLOCK_PRENORM = 0, 1, 2   # SMOL_LM_BLOCK_*
-NORM_RMS, NORM_DYT = 0, 1                                # SMOL_LM_NORM_*
+ROUTE_SOFTMAX, ROUTE_SIGMOID, ROUTE_CHOSEN = 0, 1, 2     # SMOL_LM_ROUTE_*
+BLOCK_SANDWICH, BLOCK_POSTNORM, BLOCK_PRENORM, BLOCK_PARALLEL = 0, 1, 2, 3   # SMOL_LM_BLOCK_*
+NORM_RMS, NORM_DYT, NORM_LAYER = 0, 1, 2                 # SMOL_LM_NORM_*
+RUN_ADD_EMBED, RUN_MERGE_EMBED = 1, 2                    # SMOL_LM_RUN_*
 
 
 @dataclass
@@ -847,3 +848,210 @@ class GuniraxConfig:
                 n = n * self.layers[i].router.top / max(self.layers[i].router.experts, 1)
             per_layer[i] += n
         return int(sum(per_layer[i] for i in self.layer_runs()) + 2 * self.vocab * self.width)
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Bizulix: parallel layers -- one layer norm whose result both the mixer and the feed-forward read, their sum times a
+# residual multiplier joins the stream.  A span of layers may run several times with shared weights; every pass (the first
+# one too) starts from a matrix applied to [stream; embedding output].  Mixers: softmax attention without rotation whose
+# queries are scaled by a temperature that grows with the logarithm of the position and whose scores are soft-capped, or
+# retention (linear attention, one constant decay per head, rotated queries and keys, weightless RMS division per head and
+# a silu gate).  Feed-forward: routed gated (silu) experts weighted by the softmax over the chosen router logits, and a
+# shared expert under a sigmoid gate per token.  The logits are soft-capped.
+
+
+@dataclass
+class TemperatureAttentionSpec:
+    kind = "attention"
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    softcap: float        # score <- softcap * tanh(score / softcap); 0: none
+    temp_coef: float      # the query at position p is multiplied by 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)
+    temp_every: float
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "TemperatureAttentionSpec":
+        t = d.get("q_temp") or {}
+        spec = cls(int(d["heads"]), int(d.get("kv_heads", d["heads"])), int(d["dim"]), int(d.get("vdim", d["dim"])), float(d["scale"]),
+                   float(d.get("softcap") or 0.0), float(t.get("coef", 0.0)), float(t.get("every", 1.0)))
+        if spec.heads % spec.kv_heads or spec.temp_every <= 0 or spec.softcap < 0:
+            raise ValueError("attention: heads must be a multiple of kv_heads, q_temp.every positive and softcap not negative")
+        return spec
+
+    def to_dict(self) -> Dict[str, Any]:
+        every = int(self.temp_every) if self.temp_every == int(self.temp_every) else self.temp_every
+        return {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale, "softcap": self.softcap,
+                "q_temp": {"coef": self.temp_coef, "every": every}}
+
+
+@dataclass
+class RetentionSpec:
+    kind = "retention"
+    heads: int
+    dim: int
+    vdim: int
+    decay: List[float]    # one per head
+    rot: RotarySpec       # coordinate i < dims / 2 is paired with coordinate i + dims / 2
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "RetentionSpec":
+        decay = d["decay"]
+        if isinstance(decay, (int, float)):      # one number: every head's decay
+            decay = [decay] * int(d["heads"])
+        spec = cls(int(d["heads"]), int(d["dim"]), int(d.get("vdim", d["dim"])), [float(v) for v in decay], RotarySpec.from_dict(d["rot"]))
+        if len(spec.decay) != spec.heads or spec.rot.dims > spec.dim:
+            raise ValueError("retention: one decay per head, rot.dims at most dim")
+        return spec
+
+    def to_dict(self) -> Dict[str, Any]:
+        return {"heads": self.heads, "dim": self.dim, "vdim": self.vdim, "decay": list(self.decay), "rot": self.rot.to_dict()}
+
+
+@dataclass
+class BizulixLayer:
+    mixer: Any                               # TemperatureAttentionSpec | RetentionSpec
+    ff: int = 0                              # size of one expert (0: the layer has no feed-forward)
+    experts: int = 0
+    top: int = 0
+    shared_ff: int = 0                       # size of the shared expert (0: none)
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "BizulixLayer":
+        kinds = {"attention": TemperatureAttentionSpec, "retention": RetentionSpec}
+        if d["type"] not in kinds:
+            raise ValueError(f"unknown mixer type {d['type']!r}; have {sorted(kinds)}")
+        L = cls(kinds[d["type"]].from_dict(d["mixer"]))
+        mlp = d.get("mlp")
+        if not mlp:
+            return L
+        if mlp["kind"] != "moe":
+            raise ValueError(f"unknown feed-forward kind {mlp['kind']!r}")
+        L.ff, L.experts, L.top = int(mlp["expert"]["ff"]), int(mlp["router"]["experts"]), int(mlp["router"]["top"])
+        L.shared_ff = int((mlp.get("shared") or {}).get("ff", 0))
+        if L.ff < 1 or not 1 <= L.top <= L.experts:
+            raise ValueError("router: top must lie between 1 and the number of experts, and an expert's size be positive")
+        return L
+
+    def to_dict(self) -> Dict[str, Any]:
+        mlp = None
+        if self.ff:
+            mlp = {"kind": "moe", "expert": {"ff": self.ff}, "router": {"experts": self.experts, "top": self.top}}
+            if self.shared_ff:
+                mlp["shared"] = {"ff": self.shared_ff}
+        return {"type": self.mixer.kind, "mixer": self.mixer.to_dict(), "mlp": mlp}
+
+
+@dataclass
+class BizulixConfig:
+    architecture: str = "Bizulix"
+    vocab: int = 0
+    width: int = 0
+    norm_eps: float = 1e-6
+    residual_mult: float = 1.0
+    logit_softcap: float = 0.0               # logits <- cap * tanh(logits / cap); 0: none
+    layers: List[BizulixLayer] = field(default_factory=list)
+    loop_start: int = 0
+    loop_stop: int = 0
+    loop_times: int = 1
+    extra: Dict[str, Any] = field(default_factory=dict, repr=False)
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "BizulixConfig":
+        loop = d.get("loop") or {}
+        known = {"architecture", "vocab", "width", "norm", "residual_mult", "logit_softcap", "layers", "loop"}
+        cfg = cls(architecture=d.get("architecture", "Bizulix"), vocab=int(d["vocab"]), width=int(d["width"]), norm_eps=float(d["norm"]["eps"]),
+                  residual_mult=float(d.get("residual_mult", 1.0)), logit_softcap=float(d.get("logit_softcap") or 0.0),
+                  layers=[BizulixLayer.from_dict(x) for x in d["layers"]],
+                  loop_start=int(loop.get("start", 0)), loop_stop=int(loop.get("stop", 0)), loop_times=int(loop.get("times", 1)),
+                  extra={k: v for k, v in d.items() if k not in known})
+        if cfg.looped and (cfg.loop_times < 1 or not 0 <= cfg.loop_start < cfg.loop_stop <= len(cfg.layers)):
+            raise ValueError(f"loop {cfg.loop_start}..{cfg.loop_stop} x {cfg.loop_times} does not fit {len(cfg.layers)} layers")
+        return cfg
+
+    @classmethod
+    def from_pretrained(cls, pathname: str) -> "BizulixConfig":
+        path = Path(pathname)
+        if path.is_dir():
+            path = path / "config.json"
+        with open(path, "r", encoding="utf-8") as f:
+            return cls.from_dict(json.load(f))
+
+    def to_dict(self) -> Dict[str, Any]:
+        d = dict(self.extra)
+        d.update(architecture=self.architecture, vocab=self.vocab, width=self.width, norm={"eps": self.norm_eps}, residual_mult=self.residual_mult,
+                 logit_softcap=self.logit_softcap, layers=[x.to_dict() for x in self.layers])
+        if self.looped:
+            d["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
+        return d
+
+    def save(self, path: str) -> None:
+        with open(path, "w") as f:
+            json.dump(self.to_dict(), f, indent=1, sort_keys=True)
+
+    @property
+    def looped(self) -> bool:
+        """Whether the model has a looped span; one that runs once still opens with the merge of stream and embedding."""
+        return self.loop_stop > self.loop_start
+
+    def layer_runs(self) -> List[int]:
+        """Layer index of every layer run, in execution order."""
+        n, a, b = len(self.layers), self.loop_start, self.loop_stop
+        if not self.looped:
+            return list(range(n))
+        return list(range(a)) + list(range(a, b)) * self.loop_times + list(range(b, n))
+
+    def run_merges(self) -> List[int]:
+        """1 for the runs that open a pass of the loop (stream and embedding output are merged before them), else 0."""
+        out = [0] * len(self.layer_runs())
+        if self.looped:
+            for rep in range(self.loop_times):
+                out[self.loop_start + rep * (self.loop_stop - self.loop_start)] = 1
+        return out
+
+    def tensor_shapes(self) -> Dict[str, tuple]:
+        """Checkpoint tensor names and shapes."""
+        D, V = self.width, self.vocab
+        out: Dict[str, tuple] = {"embed": (V, D), "head": (V, D), "final.norm": (D,), "final.norm.b": (D,)}
+        if self.looped:
+            out["loop.in"] = (D, 2 * D)
+        for i, L in enumerate(self.layers):
+            p, m = f"l{i}.", L.mixer
+            kv = m.kv_heads if m.kind == "attention" else m.heads
+            out.update({p + "norm1": (D,), p + "norm1.b": (D,), p + "mix.q": (m.heads * m.dim, D), p + "mix.k": (kv * m.dim, D),
+                        p + "mix.v": (kv * m.vdim, D), p + "mix.o": (D, m.heads * m.vdim)})
+            if m.kind == "retention":
+                out[p + "mix.g"] = (m.heads * m.vdim, D)
+            if L.ff:
+                for e in range(L.experts):
+                    out.update({f"{p}mlp.e{e}.gate": (L.ff, D), f"{p}mlp.e{e}.up": (L.ff, D), f"{p}mlp.e{e}.down": (D, L.ff)})
+                out.update({p + "mlp.router": (L.experts, D), p + "mlp.router.b": (L.experts,)})
+                if L.shared_ff:
+                    out.update({p + "mlp.shared.gate": (L.shared_ff, D), p + "mlp.shared.up": (L.shared_ff, D), p + "mlp.shared.down": (D, L.shared_ff),
+                                p + "mlp.shared.sg": (1, D)})
+        return out
+
+    # ---- accounting used by the benchmark ----
+    def _elements_by_part(self, active_only: bool) -> Dict[Any, float]:
+        """Matrix elements of every layer (key: its index) and of the other matrices (key: tensor name)."""
+        out: Dict[Any, float] = {}
+        for k, s in self.tensor_shapes().items():
+            if len(s) != 2 or k == "embed":
+                continue
+            part: Any = int(k[1:k.index(".")]) if k[0] == "l" and k[1].isdigit() else k
+            n = float(s[0] * s[1])
+            if active_only and ".mlp.e" in k:
+                n *= self.layers[part].top / self.layers[part].experts
+            out[part] = out.get(part, 0.0) + n
+        return out
+
+    def weight_elements(self, active_only: bool = False) -> int:
+        """Matrix elements of the model without the embedding table (looped layers once: their weights are shared);
+        ``active_only``: those one token touches (``top`` experts)."""
+        return int(sum(self._elements_by_part(active_only).values()))
+
+    def matmul_flops_per_token(self) -> int:
+        per = self._elements_by_part(True)
+        return int(2 * (sum(per.get(i, 0.0) for i in self.layer_runs()) + sum(self.run_merges()) * per.get("loop.in", 0.0) + per["head"]))
