@@ -1,7 +1,7 @@
 """Prefill and decode throughput of the hybrid language-model engine at layer sizes that resemble a real model's:
 the Pamasun design beside the DualAR slow transformer (the package's closest model: attention + gated MLP layers), and the
 Maferax and Sunutar designs beside Pamasun at equal width, depth and head count (``--lm-design maferax`` / ``sunutar``),
-and the Gunirax design beside Sunutar (``--lm-design gunirax``).
+the Gunirax design beside Sunutar (``--lm-design gunirax``), and the Bizulix design beside Maferax (``--lm-design bizulix``).
 
 ``python bench.py --lm`` prints one JSON line: for every size, tokens/s of a whole-prompt prefill and of single-token
 decode steps against a filled cache, each with its distance from the roofline (matrix-product + attention flops over the
@@ -367,6 +367,110 @@ def bench_gunirax(name: str, prompt: int, batch: int, decode_steps: int, warmup:
             "gpu_launches": int(launches)}
 
 
+BIZULIX_SIZES = {
+    # layers after Maferax's pattern (r = retention heads x (dim keys, vdim values), a = attention heads x dim over kv_heads); every layer
+    # has routed experts (top of experts, size eff) and a shared expert of size eff; `loop`: a span of layers and how often it runs
+    "w768": dict(width=768, layers=10, heads=12, kv_heads=4, dim=64, vdim=64, experts=16, top=2, eff=1024, vocab=2368, pattern="raa", loop=None),
+    "w768loop": dict(width=768, layers=6, heads=12, kv_heads=4, dim=64, vdim=64, experts=16, top=2, eff=1024, vocab=2368, pattern="raa", loop=(1, 3, 3)),
+    "w1536": dict(width=1536, layers=12, heads=12, kv_heads=4, dim=128, vdim=128, experts=32, top=3, eff=1024, vocab=8192, pattern="raa", loop=None),
+}
+
+
+def bizulix_config(width, layers, heads, kv_heads, dim, vdim, experts, top, eff, vocab, pattern, loop) -> dict:
+    ls = []
+    for i in range(layers):
+        mlp = {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": experts, "top": top}, "shared": {"ff": eff}}
+        if pattern[i % len(pattern)] == "a":
+            ls.append({"type": "attention", "mlp": mlp,
+                       "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "softcap": 30.0,
+                                 "q_temp": {"coef": 0.1, "every": 1024}}})
+        else:
+            ls.append({"type": "retention", "mlp": mlp,
+                       "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": [1.0 - 2.0 ** (-5 - 3 * h / max(heads - 1, 1)) for h in range(heads)],
+                                 "rot": {"base": 10000.0, "dims": dim}}})
+    cfg = {"architecture": "Bizulix", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "logit_softcap": 15.0, "layers": ls}
+    if loop:
+        cfg["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return cfg
+
+
+def bizulix_state_dict(cfg, seed: int = 0) -> Dict[str, torch.Tensor]:
+    g = torch.Generator().manual_seed(seed)
+    sd = {}
+    for k, s in cfg.tensor_shapes().items():
+        if len(s) == 2:
+            sd[k] = (torch.randn(*s, generator=g) * (s[1] ** -0.5)).bfloat16()
+        elif k.endswith(".b"):
+            sd[k] = (torch.randn(*s, generator=g) * 0.05).bfloat16()
+        else:
+            sd[k] = torch.ones(s).bfloat16()
+    sd["embed"] = torch.randn(*sd["embed"].shape, generator=g).bfloat16()
+    return sd
+
+
+def bench_bizulix(name: str, prompt: int, batch: int, decode_steps: int, warmup: int, steps: int, peaks) -> dict:
+    """Like bench_maferax.  Prefill flops: matrix products of the weights one token touches (per layer run), attention
+    (2 dim + 2 vdim per visible key and head) and retention (6 dim vdim per head and token); decode bytes: the weights one step
+    touches in every layer run (every expert only if the batch's choices can cover them all; a looped layer's weights count per
+    pass), the keys and values, and the states (read and written)."""
+    from .lm import BizulixLM
+    from .lm_config import BizulixConfig
+
+    hbm, tflops, _ = peaks
+    spec = BIZULIX_SIZES[name]
+    cfg = BizulixConfig.from_dict(bizulix_config(**spec))
+    model = BizulixLM(cfg, dtype=torch.bfloat16, max_tokens=batch * (prompt + 64 + decode_steps), max_seqs=batch, page_size=64,
+                      max_step_tokens=2048, max_want=batch)
+    model.load_state_dict(bizulix_state_dict(cfg, 0))
+    g = torch.Generator().manual_seed(1)
+    toks = torch.randint(0, cfg.vocab, (batch, prompt + decode_steps), generator=g).tolist()
+    n_attn = sum(cfg.layers[i].mixer.kind == "attention" for i in cfg.layer_runs())
+    n_ret = len(cfg.layer_runs()) - n_attn
+    H, G, d, dv, D = spec["heads"], spec["kv_heads"], spec["dim"], spec["vdim"], cfg.width
+    flops_token = cfg.matmul_flops_per_token()
+
+    def prefill():
+        seq = model.open_sequence()
+        for lo in range(0, prompt, model.max_step_tokens):
+            part = toks[0][lo:min(prompt, lo + model.max_step_tokens)]
+            model.forward([(seq, part, [len(part) - 1] if lo + len(part) == prompt else [])])
+        model.close_sequence(seq)
+
+    l0 = model.launch_count
+    ms_p = _timed(prefill, warmup, steps)
+    launches = model.launch_count - l0
+    flops_p = prompt * (flops_token - 2 * cfg.vocab * D) + n_attn * H * (2 * d + 2 * dv) * prompt * (prompt + 1) / 2 + n_ret * 6 * H * d * dv * prompt
+    seqs = [model.open_sequence() for _ in range(batch)]
+    for b, s in enumerate(seqs):
+        for lo in range(0, prompt, model.max_step_tokens):
+            model.forward([(s, toks[b][lo:min(prompt, lo + model.max_step_tokens)], [])])
+
+    def decode():
+        for i in range(decode_steps):
+            model.forward([(s, [toks[b][prompt + i]], [0]) for b, s in enumerate(seqs)])
+        for s in seqs:
+            s.length = prompt
+
+    l0 = model.launch_count
+    ms_d = _timed(decode, 2, steps) / decode_steps
+    launches += model.launch_count - l0
+    extra = min(batch * spec["top"], spec["experts"]) - spec["top"]      # experts a step touches beyond one token's
+    touched = flops_token / 2 + len(cfg.layer_runs()) * extra * 3 * D * spec["eff"]
+    kv_bytes = n_attn * G * (d + dv) * 2 * (prompt + decode_steps / 2) * batch
+    st_bytes = n_ret * 2 * H * d * dv * 4 * batch
+    bytes_d = 2 * touched + kv_bytes + st_bytes
+    model.check_device_errors()
+    for s in seqs:
+        model.close_sequence(s)
+    return {"model": f"Bizulix {name}", "spec": spec, "parameters_m": round(cfg.weight_elements() / 1e6, 1),
+            "active_parameters_m": round(cfg.weight_elements(active_only=True) / 1e6, 1),
+            "prefill": {"prompt": prompt, "tokens_per_s": prompt / ms_p * 1e3, "ms": ms_p, "tflops": flops_p / ms_p / 1e9,
+                        "of_peak": flops_p / ms_p / 1e9 / tflops},
+            "decode": {"batch": batch, "context": prompt, "tokens_per_s": batch / ms_d * 1e3, "ms_per_step": ms_d,
+                       "gbs": bytes_d / ms_d / 1e6, "of_peak": bytes_d / ms_d / 1e6 / hbm},
+            "gpu_launches": int(launches)}
+
+
 def pamasun_config(width, layers, heads, kv_heads, dim, ff, vocab, pattern) -> dict:
     ls = []
     for i in range(layers):
@@ -538,7 +642,17 @@ def run(args, root: str) -> None:
     peaks = _peaks(root)
     t0 = time.time()
     entries: List[dict] = []
-    if getattr(args, "lm_design", "pamasun") == "gunirax":
+    if getattr(args, "lm_design", "pamasun") == "bizulix":
+        # Bizulix beside Maferax (the engine's closest design: every layer either an attention over the paged pool or a linear recurrence
+        # on the shared scan, routed silu experts) at equal width, depth, heads, state sizes and active feed-forward size
+        names = [n for n in (args.lm_sizes.split(",") if args.lm_sizes else ["w768", "w768loop", "w1536"])]
+        for n in names:
+            for batch in (1, 4):
+                entries.append(bench_bizulix(n, args.lm_prompt, batch, 16, args.warmup, args.steps, peaks))
+        for n in sorted({"w1536" if n == "w1536" else "w768" for n in names}):
+            for batch in (1, 4):
+                entries.append(bench_maferax(n, args.lm_prompt, batch, 16, args.warmup, args.steps, peaks))
+    elif getattr(args, "lm_design", "pamasun") == "gunirax":
         # Gunirax beside Sunutar (the engine's closest design: every mixer a pair of an attention and a recurrence on the same input,
         # dense and routed feed-forwards) at equal width, depth, heads and state sizes
         names = [n for n in (args.lm_sizes.split(",") if args.lm_sizes else ["w768", "w768dense", "w1536"])]
