@@ -840,6 +840,13 @@ __global__ void __launch_bounds__(kAttnWarps * 32) attn_kernel(const AttnArgs A,
 constexpr int kGraphMaxTokens = 64;   // steps of at most this many tokens are replayed from a captured graph
 constexpr int kShortSeq = 8;          // a sequence with at most this many tokens in a step takes this path
 
+__device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
+    const uint32_t a = (uint32_t)__cvta_generic_to_shared(smem);
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(a), "l"(gmem));
+}
+__device__ __forceinline__ void cp_async_commit_group() { asm volatile("cp.async.commit_group;" ::); }
+template <int N> __device__ __forceinline__ void cp_async_wait_group() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
 // q (fp32, shared memory) . k (one cached key row), 16-byte loads where the row allows them
 template <class T> __device__ __forceinline__ float key_dot(const float* qs, const T* k, int d);
 template <> __device__ __forceinline__ float key_dot<float>(const float* qs, const float* k, int d) {
@@ -919,15 +926,17 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
             const size_t in_pg = (size_t)g * A.page_size + j % A.page_size;
             if (c < kchunks) {
                 const T* src = base + A.k_off + in_pg * A.k_ld;
-                if (kvec) *reinterpret_cast<uint4*>(Ks + row * ldk + c * kPad) = *reinterpret_cast<const uint4*>(src + c * kPad);
+                if (kvec) cp_async16(Ks + row * ldk + c * kPad, src + c * kPad);
                 else Ks[row * ldk + c] = src[c];
             } else {
                 const int cv = c - kchunks;
                 const T* src = base + A.v_off + in_pg * A.v_ld;
-                if (vvec) *reinterpret_cast<uint4*>(Vs + row * ldv + cv * kPad) = *reinterpret_cast<const uint4*>(src + cv * kPad);
+                if (vvec) cp_async16(Vs + row * ldv + cv * kPad, src + cv * kPad);
                 else Vs[row * ldv + cv] = src[cv];
             }
         }
+        cp_async_commit_group();
+        cp_async_wait_group<0>();
         __syncthreads();
         if (!active) continue;
         const int j = j0 + lane;
@@ -1027,13 +1036,6 @@ __device__ __forceinline__ void ldmatrix_x2_trans(uint32_t& r0, uint32_t& r1, co
     asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(a));
 }
 
-// rows x cols bf16 from `src(row)` (nullptr: a row of zeros) into dst[row * LD + col], columns cols .. DP-1 zeroed.
-__device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
-    const uint32_t a = (uint32_t)__cvta_generic_to_shared(smem);
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(a), "l"(gmem));
-}
-__device__ __forceinline__ void cp_async_commit_group() { asm volatile("cp.async.commit_group;" ::); }
-template <int N> __device__ __forceinline__ void cp_async_wait_group() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // 64 rows of `cols` bf16 into a [64][DP + 8] tile; src(row) is the row's address or nullptr (zero row).  ASYNC: whole
 // 16-byte pieces of aligned rows go by cp.async (the caller commits and waits); everything else is stored directly.
@@ -1078,9 +1080,9 @@ __global__ void __launch_bounds__(128) attn_flash_kernel(const AttnArgs A, const
     bf16* Vs = VK ? Ks : Ks + 2 * kTile;
     const int s = blockIdx.y;
     const int t0 = A.seq_start[s], n = A.seq_start[s + 1] - t0;
-    const int tile = gridDim.x - 1 - blockIdx.x;      // the tiles with the most keys start first
+    const int tile = gridDim.z - 1 - blockIdx.z;      // the tiles with the most keys start first, those of every head together
     if (n <= kShortSeq || tile * 64 >= n) return;
-    const int h = blockIdx.z, g = h / (A.H / A.G);
+    const int h = blockIdx.x, g = h / (A.H / A.G);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
     const int pos0 = A.tok_pos[t0];
     const int32_t* bt = A.block_table + (size_t)s * A.max_pages;
@@ -1865,11 +1867,16 @@ extern "C" size_t smol_lm_workspace_bytes(const SmolLm* m) { return m ? m->total
 extern "C" int64_t smol_lm_launch_count(const SmolLm* m) { return m ? m->launches : 0; }
 extern "C" int32_t* smol_lm_error_word(SmolLm* m) { return (m && m->bound) ? reinterpret_cast<int32_t*>(m->ws + m->o_err) : nullptr; }
 
+// Shared memory the scan asks for when another kernel runs beside it: at most two of its blocks then share an SM (left to
+// itself the hardware packs them onto the few SMs that happen to have room, and a scan is bound by its slowest block), and
+// one still fits beside a tcgen05 product's block.
+constexpr int kScanSpread = 76 * 1024;
+
 template <int DK>
 static cudaError_t scan_attribute() {
     cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(2 * delta_buf_floats(DK) * sizeof(float)));
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(gla_scan_kernel<DK, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(2 * gla_buf_floats(DK) * sizeof(float)));
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(gla_scan_kernel<DK, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(2 * gla_buf_floats(DK) * sizeof(float)));
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(gla_scan_kernel<DK, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, std::max(kScanSpread, (int)(2 * gla_buf_floats(DK) * sizeof(float))));
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(gla_scan_kernel<DK, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, std::max(kScanSpread, (int)(2 * gla_buf_floats(DK) * sizeof(float))));
     return e;
 }
 static constexpr int flash_smem_bytes(int DK, int DV, bool vk) { return 2 * 64 * ((DK + 8) + (vk ? 0 : DV + 8)) * (int)sizeof(bf16); }
@@ -1948,8 +1955,10 @@ extern "C" int smol_lm_bind(SmolLm* m, const SmolLmGlobals* g, void* d_workspace
         CU(cudaEventCreateWithFlags(&m->ff_done, cudaEventDisableTiming));
     }
     if ((size_t)m->cfg.width * 4 > 48 * 1024) {
-        CU(cudaFuncSetAttribute(residual_norm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, m->cfg.width * 4));
-        CU(cudaFuncSetAttribute(residual_norm_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, m->cfg.width * 4));
+        CU((cudaFuncSetAttribute(residual_norm_kernel<float, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, m->cfg.width * 4)));
+        CU((cudaFuncSetAttribute(residual_norm_kernel<float, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, m->cfg.width * 4)));
+        CU((cudaFuncSetAttribute(residual_norm_kernel<bf16, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, m->cfg.width * 4)));
+        CU((cudaFuncSetAttribute(residual_norm_kernel<bf16, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, m->cfg.width * 4)));
     }
     m->bound = true;
     return SMOL_OK;
@@ -2073,20 +2082,22 @@ static cudaError_t launch_scan(const DeltaArgs& A, int n_seqs, const float* dec,
 }
 
 template <int DK>
-static cudaError_t launch_gla_scan(const GlaArgs& A, int n_seqs, const float* dec, float* pool, float* o_raw, cudaStream_t st) {
+static cudaError_t launch_gla_scan(const GlaArgs& A, int n_seqs, const float* dec, float* pool, float* o_raw, cudaStream_t st, size_t min_smem) {
     constexpr int CB = gla_block_cols(DK), threads = CB * gla_lanes(DK);
     const int groups = (A.dv + CB - 1) / CB;
-    if (A.head_decay) gla_scan_kernel<DK, true><<<n_seqs * A.H * groups, threads, 2 * gla_buf_floats(DK) * sizeof(float), st>>>(A, dec, pool, o_raw);
-    else gla_scan_kernel<DK, false><<<n_seqs * A.H * groups, threads, 2 * gla_buf_floats(DK) * sizeof(float), st>>>(A, dec, pool, o_raw);
+    const size_t smem = std::max(2 * gla_buf_floats(DK) * sizeof(float), min_smem);
+    if (A.head_decay) gla_scan_kernel<DK, true><<<n_seqs * A.H * groups, threads, smem, st>>>(A, dec, pool, o_raw);
+    else gla_scan_kernel<DK, false><<<n_seqs * A.H * groups, threads, smem, st>>>(A, dec, pool, o_raw);
     return cudaGetLastError();
 }
 // the scan over key sizes up to 256: the smallest built size that holds A.d
-static cudaError_t launch_gla_scan_any(const GlaArgs& A, int n_seqs, const float* dec, float* pool, float* o_raw, cudaStream_t st) {
-    if (A.d <= 16) return launch_gla_scan<16>(A, n_seqs, dec, pool, o_raw, st);
-    if (A.d <= 32) return launch_gla_scan<32>(A, n_seqs, dec, pool, o_raw, st);
-    if (A.d <= 64) return launch_gla_scan<64>(A, n_seqs, dec, pool, o_raw, st);
-    if (A.d <= 128) return launch_gla_scan<128>(A, n_seqs, dec, pool, o_raw, st);
-    return launch_gla_scan<256>(A, n_seqs, dec, pool, o_raw, st);
+static cudaError_t launch_gla_scan_any(const GlaArgs& A, int n_seqs, const float* dec, float* pool, float* o_raw, cudaStream_t st,
+                                        size_t min_smem = 0) {
+    if (A.d <= 16) return launch_gla_scan<16>(A, n_seqs, dec, pool, o_raw, st, min_smem);
+    if (A.d <= 32) return launch_gla_scan<32>(A, n_seqs, dec, pool, o_raw, st, min_smem);
+    if (A.d <= 64) return launch_gla_scan<64>(A, n_seqs, dec, pool, o_raw, st, min_smem);
+    if (A.d <= 128) return launch_gla_scan<128>(A, n_seqs, dec, pool, o_raw, st, min_smem);
+    return launch_gla_scan<256>(A, n_seqs, dec, pool, o_raw, st, min_smem);
 }
 
 // The attention kernels over the rows of a step: prompt portions on the tensor-core form (bf16, `flash`) or the
@@ -2106,7 +2117,7 @@ static void launch_attention(SmolLm* m, const SmolLmStep* s, AttnArgs& A, bool f
     if (A.window > 0) A.n_splits = std::min(A.n_splits, ((A.window - 1) / m->split_len + 2 + 3) / 4 * 4);      // ranges a window can touch
     if (max_n > kShortSeq) {
         if (flash) {
-            dim3 grid((max_n + 63) / 64, s->n_seqs, A.H);
+            dim3 grid(A.H, s->n_seqs, (max_n + 63) / 64);
             const int hp = std::max(A.d, A.dv);
             const bf16* qb = reinterpret_cast<const bf16*>(qbuf);
             const bf16* pl = reinterpret_cast<const bf16*>(pool);
@@ -2195,6 +2206,16 @@ static bool launch_sigmoid_flash(SmolLm* m, const SmolLmStep* s, SigmoidArgs& S,
     }
     if (done) m->launches += 1;
     return done;
+}
+
+template <class T>
+static void launch_residual_norm(const ResidualArgs& A, int rows, int threads, T* hn, cudaStream_t st) {
+    uintptr_t at = 0;
+    for (const void* p : {(const void*)A.x, (const void*)A.y, (const void*)A.y2, (const void*)A.y_w, (const void*)A.y2_w, (const void*)A.rs.yp, (const void*)A.trace,
+                          (const void*)A.x0, (const void*)A.cat, (const void*)A.next.w, (const void*)A.next.shift, (const void*)hn})
+        at |= reinterpret_cast<uintptr_t>(p);
+    if (A.D % 4 == 0 && at % 16 == 0) residual_norm_kernel<T, true><<<rows, threads, A.D * sizeof(float), st>>>(A, hn);
+    else residual_norm_kernel<T, false><<<rows, threads, A.D * sizeof(float), st>>>(A, hn);
 }
 
 template <class T>
@@ -2411,7 +2432,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             A.q_src = conv; A.k_src = conv + hd; A.v_src = pj + 2 * hd;
             A.q_ld = A.k_ld = 2 * hd; A.v_ld = n_in;
             A.head_decay = M.head_decay; A.head_ld = 0;
-            CU(launch_gla_scan_any(A, s->n_seqs, nullptr, m->slots, oraw, st));
+            CU(launch_gla_scan_any(A, s->n_seqs, nullptr, m->slots, oraw, st, parallel && Tn > kGraphMaxTokens ? kScanSpread : 0));
             A.out_ld = ld; A.out_scale = M.mix_scale;
             gla_out_kernel<T><<<(Tn * M.heads + 3) / 4, 128, 0, st>>>(A, oraw, mix_at);
             m->launches += 3;
@@ -2462,7 +2483,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
                 Rt.given = nullptr; Rt.given_ld = n_in; Rt.perm = Rt.slot_of = Rt.n_sorted = nullptr;
                 Rt.unit_in = Rt.unit_gate = nullptr; Rt.unit_out = nullptr; Rt.unit_ff = Rt.unit_ld = 0; Rt.unit_act = expert_actp(L);
                 const int pairs = Tn * L.top_k;
-                const bool few = !kIsF32 && L.n_experts > 0 && pairs <= kMoeGemvPairs && D % 8 == 0 && L.ff % 8 == 0;
+                const bool few = !kIsF32 && L.n_experts > 0 && pairs <= kMoeGemvPairs && D % 8 == 0 && L.ff % 8 == 0 && L.ff <= 16384;
                 const bool direct = few && L.n_identity == 0;      // the pairs stay in their order: nothing to sort
                 if (direct) { Rt.perm = perm; Rt.slot_of = slot_of; Rt.n_sorted = seg + L.n_experts; }
                 // the router reads the sublayer's input in fp32 where the block keeps it (post-norm), else its T form
@@ -2511,7 +2532,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
                                                                                          seg + L.n_experts, reinterpret_cast<const bf16*>(L.w_experts_in), io.sw,
                                                                                          zp, NF, D, expert_actp(L));
                         // the second product applies the activation as it reads the first one's result
-                        moe_gemv_kernel<true><<<dim3((D + 7) / 8, pairs), 256, 0, st>>>(zp, perm, 0, sel_id, seg + L.n_experts,
+                        moe_gemv_kernel<true><<<dim3((D + 7) / 8, pairs), 256, L.ff * sizeof(bf16), st>>>(zp, perm, 0, sel_id, seg + L.n_experts,
                                                                                         reinterpret_cast<const bf16*>(L.w_experts_out), io2.sw, yp, D, L.ff, expert_actp(L));
                         m->launches += 1;
                     } else {
@@ -2551,13 +2572,16 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             }
             return SMOL_OK;
         };
+        // Parallel block: both sublayers read the same projection, so the feed-forward runs on its own stream beside the mixer.
+        const bool beside = parallel && L.mlp != SMOL_LM_MLP_NONE;
         if (parallel && L.mlp != SMOL_LM_MLP_NONE) {
-            // both sublayers read the same projection: the feed-forward runs on its own stream beside the mixer
-            CU(cudaEventRecord(m->ff_start, st));
-            CU(cudaStreamWaitEvent(m->ff_stream, m->ff_start, 0));
-            const int rc = feed_forward(m->ff_stream);
+            if (beside) {
+                CU(cudaEventRecord(m->ff_start, st));
+                CU(cudaStreamWaitEvent(m->ff_stream, m->ff_start, 0));
+            }
+            const int rc = feed_forward(beside ? m->ff_stream : st);
             if (rc != SMOL_OK) return rc;
-            CU(cudaEventRecord(m->ff_done, m->ff_stream));
+            if (beside) CU(cudaEventRecord(m->ff_done, m->ff_stream));
         }
         if (pairable(L)) {
             int rc = run_mixer(L, R, proj, L.in_bias, mix, own_proj ? mix_cols_of(L) : mix_ld);
@@ -2662,7 +2686,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             m->launches += 3;
             mix_cols = L.heads * L.dim;
         }
-        if (parallel && L.mlp != SMOL_LM_MLP_NONE) CU(cudaStreamWaitEvent(st, m->ff_done, 0));      // also: w_out covers the shared expert's unit
+        if (beside) CU(cudaStreamWaitEvent(st, m->ff_done, 0));      // also: w_out covers the shared expert's unit
         CU(linear<T>(m, mix_in, static_cast<const T*>(L.w_out), y, Tn, D, mix_cols, st));
         if (own_proj) CU(linear<T>(m, mix2, static_cast<const T*>(L.side->w_out), y2, Tn, D, mix_cols_of(*L.side), st));
         const bool last = n + 1 == m->runs.size();
@@ -2678,7 +2702,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             Ra.rs = routed; Ra.s_routed = c.residual_mult;
             Ra.trace = s->trace ? s->trace + n * (size_t)Tn * D : nullptr; Ra.x0 = nullptr; Ra.cat = merge ? cat : nullptr;
             Ra.next = (Ln && !merge) ? norm_of(Ln->norm1, Ln->norm1_shift, Ln->norm1_alpha) : no_norm;
-            residual_norm_kernel<T><<<Tn, nthr, D * sizeof(float), st>>>(Ra, hn, hn);
+            launch_residual_norm<T>(Ra, Tn, nthr, hn, st);
             m->launches += 1;
         } else if (prenorm) {
             // x += mixer (mixers with their own projections: each normed over the width first); x += feed-forward.  The kernel
@@ -2696,7 +2720,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             Ra.rs = no_sum; Ra.s_routed = 1.0f; Ra.cat = nullptr;
             Ra.trace = has_ff ? nullptr : tr_row; Ra.x0 = has_ff ? nullptr : restart;
             Ra.next = has_ff ? norm_of(L.norm2, L.norm2_shift, L.norm2_alpha) : after;
-            residual_norm_kernel<T><<<Tn, nthr, D * sizeof(float), st>>>(Ra, hn, hn);
+            launch_residual_norm<T>(Ra, Tn, nthr, hn, st);
             m->launches += 1;
             if (has_ff) {
                 const int rc = feed_forward(st);
@@ -2706,7 +2730,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
                 Ra.y2 = nullptr; Ra.y2_w = nullptr; Ra.sy2 = 0.0f;
                 Ra.rs = routed;
                 Ra.trace = tr_row; Ra.x0 = restart; Ra.next = after;
-                residual_norm_kernel<T><<<Tn, nthr, D * sizeof(float), st>>>(Ra, hn, hn);
+                launch_residual_norm<T>(Ra, Tn, nthr, hn, st);
                 m->launches += 1;
             }
         } else if (postnorm) {

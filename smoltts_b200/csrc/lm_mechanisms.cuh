@@ -720,7 +720,20 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const RouteArgs A, const
         const float gate = A.unit_gate ? sigmoidf_(A.unit_gate[(size_t)t * A.given_ld]) : 1.0f;
         const int uo = A.unit_act.plain ? 0 : A.unit_ff;
         TI* out = static_cast<TI*>(A.unit_out) + (size_t)t * A.unit_ld;
-        for (int c = threadIdx.x; c < A.unit_ff; c += blockDim.x) out[c] = from_f<TI>(gate * gated_unit_(A.unit_act, u[c], u[uo + c]));
+        for (int c0 = threadIdx.x; c0 < A.unit_ff; c0 += blockDim.x * 8) {      // eight loads of each row go out at a time
+            float g[8], v[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const int c = c0 + i * blockDim.x;
+                g[i] = c < A.unit_ff ? u[c] : 0.0f;
+                v[i] = c < A.unit_ff ? u[uo + c] : 0.0f;
+            }
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const int c = c0 + i * blockDim.x;
+                if (c < A.unit_ff) out[c] = from_f<TI>(gate * gated_unit_(A.unit_act, g[i], v[i]));
+            }
+        }
     }
     if (!A.given && e0 < A.E) {
         const float* wr = A.w_router + (size_t)e0 * A.D;
@@ -903,36 +916,43 @@ __global__ void moe_gather_scaled_kernel(const T* __restrict__ h, const int32_t*
 // pieces, the expert's weight row is streamed once.  Sorted row r belongs to pair perm[r], whose router output names the
 // expert; it reads a's row perm[r] / gather_div (gather_div == 0: row r itself).  Needs K % 8 == 0 and 16-byte aligned rows.
 // ACT: a is instead the fp32 result of the first product [rows][2 K] (gate | up), and the row is the gated unit's value,
-// rounded to bf16 as the tile forms round it.
+// rounded to bf16 as the tile forms round it (K bf16 of dynamic shared memory).
 constexpr int kMoeGemvPairs = 32;
 template <bool ACT>
 __global__ void __launch_bounds__(256) moe_gemv_kernel(const void* __restrict__ a_any, const int32_t* __restrict__ perm, int gather_div,
                                                        const int32_t* __restrict__ sel_id, const int32_t* __restrict__ n_sorted,
                                                        const bf16* __restrict__ w, long long w_stride, float* __restrict__ y, int N, int K,
                                                        const ActParams act) {
+    extern __shared__ __align__(16) unsigned char unit_smem[];      // ACT: the row's unit values [K]
     const int r = blockIdx.y;
     if (r >= *n_sorted) return;
     const int lane = threadIdx.x & 31, n = blockIdx.x * 8 + (threadIdx.x >> 5);
-    if (n >= N) return;
     const int pair = perm[r];
-    const bf16* wr = w + (long long)sel_id[pair] * w_stride + (size_t)n * K;
+    const bf16* wr = w + (long long)sel_id[pair] * w_stride + (size_t)min(n, N - 1) * K;
     float acc = 0.0f;
     if (ACT) {
+        // the activation is taken once per block; each warp's first weights are on their way meanwhile
+        bf16* unit = reinterpret_cast<bf16*>(unit_smem);
         const float* zr = static_cast<const float*>(a_any) + (size_t)r * (act.plain ? K : 2 * K);
         const int uo = act.plain ? 0 : K;
+        const uint4 w_first = lane * 8 < K ? ldg_stream(wr + lane * 8) : make_uint4(0, 0, 0, 0);
+        for (int k = threadIdx.x * 4; k < K; k += blockDim.x * 4) {
+            const float4 g = *reinterpret_cast<const float4*>(zr + k), u = *reinterpret_cast<const float4*>(zr + uo + k);
+            store4<bf16>(unit + k, gated_unit_(act, g.x, u.x), gated_unit_(act, g.y, u.y), gated_unit_(act, g.z, u.z), gated_unit_(act, g.w, u.w));
+        }
+        __syncthreads();
         for (int k = lane * 8; k < K; k += 256) {
-            const uint4 wv = ldg_stream(wr + k);
-            const float4 g0 = *reinterpret_cast<const float4*>(zr + k), g1 = *reinterpret_cast<const float4*>(zr + k + 4);
-            const float4 u0 = *reinterpret_cast<const float4*>(zr + uo + k), u1 = *reinterpret_cast<const float4*>(zr + uo + k + 4);
-            acc = fmaf(bf16_round(gated_unit_(act, g0.x, u0.x)), bf_lo(wv.x), acc); acc = fmaf(bf16_round(gated_unit_(act, g0.y, u0.y)), bf_hi(wv.x), acc);
-            acc = fmaf(bf16_round(gated_unit_(act, g0.z, u0.z)), bf_lo(wv.y), acc); acc = fmaf(bf16_round(gated_unit_(act, g0.w, u0.w)), bf_hi(wv.y), acc);
-            acc = fmaf(bf16_round(gated_unit_(act, g1.x, u1.x)), bf_lo(wv.z), acc); acc = fmaf(bf16_round(gated_unit_(act, g1.y, u1.y)), bf_hi(wv.z), acc);
-            acc = fmaf(bf16_round(gated_unit_(act, g1.z, u1.z)), bf_lo(wv.w), acc); acc = fmaf(bf16_round(gated_unit_(act, g1.w, u1.w)), bf_hi(wv.w), acc);
+            const uint4 wv = k == lane * 8 ? w_first : ldg_stream(wr + k), av = *reinterpret_cast<const uint4*>(unit + k);
+            acc = fmaf(bf_lo(av.x), bf_lo(wv.x), acc); acc = fmaf(bf_hi(av.x), bf_hi(wv.x), acc);
+            acc = fmaf(bf_lo(av.y), bf_lo(wv.y), acc); acc = fmaf(bf_hi(av.y), bf_hi(wv.y), acc);
+            acc = fmaf(bf_lo(av.z), bf_lo(wv.z), acc); acc = fmaf(bf_hi(av.z), bf_hi(wv.z), acc);
+            acc = fmaf(bf_lo(av.w), bf_lo(wv.w), acc); acc = fmaf(bf_hi(av.w), bf_hi(wv.w), acc);
         }
         acc = warp_sum(acc);
-        if (lane == 0) y[(size_t)r * N + n] = acc;
+        if (lane == 0 && n < N) y[(size_t)r * N + n] = acc;
         return;
     }
+    if (n >= N) return;
     const bf16* ar = static_cast<const bf16*>(a_any) + (size_t)(gather_div > 0 ? pair / gather_div : r) * K;
     for (int k = lane * 8; k < K; k += 256) {
         const uint4 wv = ldg_stream(wr + k), av = ldg_v4(ar + k);

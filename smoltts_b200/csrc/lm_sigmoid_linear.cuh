@@ -24,41 +24,89 @@ struct NormSpec {
 };
 __device__ __forceinline__ float dyt_(const NormSpec& n, float alpha, float v, int c) { return fmaf(tanhf(alpha * v), n.w[c], n.shift[c]); }
 
-// The layer norm of a row on its way to T: value(c) gives element c (read twice where the row does not fit the registers).
+// A row of D <= 8 blockDim elements in registers, 8 per thread: VEC (D % 4 == 0, rows 16-byte aligned) two 16-byte pieces of
+// neighbours, else single elements blockDim apart.  Elements beyond D hold `fill`.
+template <bool VEC> __device__ __forceinline__ int row_col(int i) {
+    return VEC ? 4 * (int)(threadIdx.x + (i / 4) * blockDim.x) + i % 4 : (int)(threadIdx.x + i * blockDim.x);
+}
+template <bool VEC>
+__device__ __forceinline__ void row_load(const float* __restrict__ p, int D, float fill, float (&v)[kRowRegs]) {
+#pragma unroll
+    for (int i = 0; i < kRowRegs; i += VEC ? 4 : 1) {
+        const int c = row_col<VEC>(i);
+        if (VEC) {
+            const float4 t = c < D ? *reinterpret_cast<const float4*>(p + c) : make_float4(fill, fill, fill, fill);
+            v[i] = t.x; v[i + 1] = t.y; v[i + 2] = t.z; v[i + 3] = t.w;
+        } else {
+            v[i] = c < D ? p[c] : fill;
+        }
+    }
+}
+template <bool VEC, class T>
+__device__ __forceinline__ void row_store(T* __restrict__ p, int D, const float (&v)[kRowRegs]) {
+#pragma unroll
+    for (int i = 0; i < kRowRegs; i += VEC ? 4 : 1) {
+        const int c = row_col<VEC>(i);
+        if (c >= D) continue;
+        if (VEC) store4<T>(p + c, v[i], v[i + 1], v[i + 2], v[i + 3]);
+        else p[c] = from_f<T>(v[i]);
+    }
+}
+
+// Mean and summed squared deviations of a row held in registers.  Every warp takes both over its own elements, the warps'
+// pairs are then joined exactly (deviations around the row's mean), so the block meets once.  `red` holds 3 x 33 floats.
+template <bool VEC>
+__device__ __forceinline__ void row_stats(const float (&v)[kRowRegs], int D, float (*red)[33], float& mean, float& m2) {
+    float s = 0.0f, n = 0.0f;
+#pragma unroll
+    for (int i = 0; i < kRowRegs; ++i)
+        if (row_col<VEC>(i) < D) { s += v[i]; n += 1.0f; }
+    s = warp_sum(s);
+    n = warp_sum(n);
+    const float wm = s / fmaxf(n, 1.0f);
+    float q = 0.0f;
+#pragma unroll
+    for (int i = 0; i < kRowRegs; ++i)
+        if (row_col<VEC>(i) < D) q = fmaf(v[i] - wm, v[i] - wm, q);
+    q = warp_sum(q);
+    const int w = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+    if ((threadIdx.x & 31) == 0) { red[0][w] = s; red[1][w] = q; red[2][w] = n; }
+    __syncthreads();
+    s = 0.0f;
+    for (int i = 0; i < nw; ++i) s += red[0][i];
+    mean = s / (float)D;
+    m2 = 0.0f;
+    for (int i = 0; i < nw; ++i) {
+        const float d = red[0][i] / fmaxf(red[2][i], 1.0f) - mean;
+        m2 += fmaf(red[2][i] * d, d, red[1][i]);
+    }
+}
+
+// The layer norm of a row on its way to T: value(c) gives element c (read several times where the row does not fit the registers).
 template <class T, class Value>
-__device__ __forceinline__ void layer_norm_row(const NormSpec& nm, int D, T* __restrict__ out, float* red, Value value) {
+__device__ __forceinline__ void layer_norm_row(const NormSpec& nm, int D, T* __restrict__ out, float (*red)[33], Value value) {
     if (D <= (int)blockDim.x * kRowRegs) {
         float v[kRowRegs], w[kRowRegs], b[kRowRegs];
-        float s = 0.0f;
 #pragma unroll
         for (int i = 0; i < kRowRegs; ++i) {
-            const int c = threadIdx.x + i * blockDim.x;
-            const bool in = c < D;
-            v[i] = in ? value(c) : 0.0f;
-            w[i] = in ? nm.w[c] : 0.0f;
-            b[i] = in ? nm.shift[c] : 0.0f;
-            s += v[i];
+            const int c = row_col<false>(i);
+            v[i] = c < D ? value(c) : 0.0f;
         }
-        const float mean = block_sum(s, red) / (float)D;
-        float q = 0.0f;
+        row_load<false>(nm.w, D, 0.0f, w);
+        row_load<false>(nm.shift, D, 0.0f, b);
+        float mean, m2;
+        row_stats<false>(v, D, red, mean, m2);
+        const float r = 1.0f / sqrtf(m2 / (float)D + nm.eps);
 #pragma unroll
-        for (int i = 0; i < kRowRegs; ++i) {
-            v[i] -= mean;
-            if ((int)(threadIdx.x + i * blockDim.x) < D) q = fmaf(v[i], v[i], q);
-        }
-        const float r = 1.0f / sqrtf(block_sum(q, red) / (float)D + nm.eps);
-#pragma unroll
-        for (int i = 0; i < kRowRegs; ++i) {
-            const int c = threadIdx.x + i * blockDim.x;
-            if (c < D) out[c] = from_f<T>(fmaf(v[i] * r, w[i], b[i]));
-        }
+        for (int i = 0; i < kRowRegs; ++i) v[i] = fmaf((v[i] - mean) * r, w[i], b[i]);
+        row_store<false, T>(out, D, v);
         return;
     }
     float s = 0.0f, q = 0.0f;
     for (int c = threadIdx.x; c < D; c += blockDim.x) s += value(c);
-    const float mean = block_sum(s, red) / (float)D;
+    const float mean = block_sum(s, red[0]) / (float)D;
     for (int c = threadIdx.x; c < D; c += blockDim.x) { const float v = value(c) - mean; q = fmaf(v, v, q); }
-    const float r = 1.0f / sqrtf(block_sum(q, red) / (float)D + nm.eps);
+    const float r = 1.0f / sqrtf(block_sum(q, red[1]) / (float)D + nm.eps);
     for (int c = threadIdx.x; c < D; c += blockDim.x) out[c] = from_f<T>(fmaf((value(c) - mean) * r, nm.w[c], nm.shift[c]));
 }
 
@@ -68,7 +116,7 @@ __device__ __forceinline__ void layer_norm_row(const NormSpec& nm, int D, T* __r
 template <class T>
 __global__ void embed_prenorm_kernel(const int32_t* __restrict__ tokens, const T* __restrict__ embed, float scale, int D, int vocab,
                                      const NormSpec nm, float* __restrict__ x, float* __restrict__ x0, T* __restrict__ hn, T* __restrict__ cat) {
-    __shared__ float red[33];
+    __shared__ float red[3][33];
     const int t = blockIdx.x;
     int tok = tokens[t];
     tok = tok < 0 ? 0 : (tok >= vocab ? vocab - 1 : tok);
@@ -89,7 +137,7 @@ __global__ void embed_prenorm_kernel(const int32_t* __restrict__ tokens, const T
         layer_norm_row<T>(nm, D, hn + o, red, [&](int c) { return x[o + c]; });      // a thread reads what it wrote itself
         return;
     }
-    ss = block_sum(ss, red);
+    ss = block_sum(ss, red[0]);
     const float r = 1.0f / sqrtf(ss / (float)D + nm.eps);
     for (int c = threadIdx.x; c < D; c += blockDim.x) hn[o + c] = from_f<T>(x[o + c] * r * nm.w[c]);
 }
@@ -97,7 +145,7 @@ __global__ void embed_prenorm_kernel(const int32_t* __restrict__ tokens, const T
 // The norm of selected rows -> T (the final norm of the rows whose logits are wanted).
 template <class T>
 __global__ void prenorm_rows_kernel(const float* __restrict__ x, const int32_t* __restrict__ rows, const NormSpec nm, int D, T* __restrict__ out) {
-    __shared__ float red[33];
+    __shared__ float red[3][33];
     const float* xr = x + (size_t)(rows ? rows[blockIdx.x] : blockIdx.x) * D;
     const size_t o = (size_t)blockIdx.x * D;
     if (nm.kind == SMOL_LM_NORM_DYT) {
@@ -111,7 +159,7 @@ __global__ void prenorm_rows_kernel(const float* __restrict__ x, const int32_t* 
     }
     float ss = 0.0f;
     for (int c = threadIdx.x; c < D; c += blockDim.x) ss += xr[c] * xr[c];
-    ss = block_sum(ss, red);
+    ss = block_sum(ss, red[0]);
     const float r = 1.0f / sqrtf(ss / (float)D + nm.eps);
     for (int c = threadIdx.x; c < D; c += blockDim.x) out[o + c] = from_f<T>(xr[c] * r * nm.w[c]);
 }
@@ -121,7 +169,7 @@ __global__ void prenorm_rows_kernel(const float* __restrict__ x, const int32_t* 
 //   x <- x + sy * f(y) + sy2 * f2(y2) + s_routed * (the routed experts' weighted sum)
 // where f(y) = y, or y / rms(y) * y_w when y_w is set (mixers side by side: each projected result is normed over the width).
 // `trace` then takes the row (the stream after the sublayer); x0, when set, joins x after that (the next run restarts from
-// stream + embedding output); hn <- next(x).  `cat`, when set, takes x in T as the first half of the row a merging run
+// stream + embedding output); hn <- next(x).  Routed experts: every choice has a row (no identity outputs here).  `cat`, when set, takes x in T as the first half of the row a merging run
 // multiplies (no norm follows here then).
 struct ResidualArgs {
     float* x;
@@ -137,8 +185,8 @@ struct ResidualArgs {
     NormSpec next;
 };
 
-template <class T>
-__global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn, const T* __restrict__ hin) {
+template <class T, bool VEC>
+__global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn) {
     extern __shared__ float row[];
     __shared__ float red3[3][33];
     const int D = A.D;
@@ -146,35 +194,44 @@ __global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn, c
     float r1 = A.sy, r2 = A.sy2;
     if (D <= (int)blockDim.x * kRowRegs) {
         // the row in registers: every operand is loaded before the first reduction, so a lone row (decoding) waits for
-        // global memory once
+        // global memory once (the routed rows: a second time, for their places)
+        constexpr int kAhead = 4;             // choices whose places and weights are read ahead
         const bool dyt_r = A.next.w && A.next.kind == SMOL_LM_NORM_DYT, layer_r = A.next.w && A.next.kind == SMOL_LM_NORM_LAYER;
         const float alpha_r = dyt_r ? A.next.alpha[0] : 0.0f;
-        float xv[kRowRegs], yv[kRowRegs], zv[kRowRegs], a1[kRowRegs], a2[kRowRegs], e0[kRowRegs], nw[kRowRegs], nb[kRowRegs];
+        int slot_r[kAhead];
+        float wt_r[kAhead];
 #pragma unroll
-        for (int i = 0; i < kRowRegs; ++i) {
-            const int c = threadIdx.x + i * blockDim.x;
-            const bool in = c < D;
-            xv[i] = in ? A.x[o + c] : 0.0f;
-            yv[i] = (in && A.y) ? A.y[o + c] : 0.0f;
-            zv[i] = (in && A.y2) ? A.y2[o + c] : 0.0f;
-            a1[i] = (in && A.y_w) ? A.y_w[c] : 1.0f;
-            a2[i] = (in && A.y2_w) ? A.y2_w[c] : 1.0f;
-            e0[i] = (in && A.x0) ? A.x0[o + c] : 0.0f;
-            nw[i] = (in && A.next.w) ? A.next.w[c] : 0.0f;
-            nb[i] = (in && (dyt_r || layer_r)) ? A.next.shift[c] : 0.0f;
+        for (int k = 0; k < kAhead; ++k) {
+            const bool in = A.rs.yp && k < A.rs.top;
+            slot_r[k] = in ? A.rs.slot_of[(size_t)blockIdx.x * A.rs.top + k] : 0;
+            wt_r[k] = in ? A.s_routed * (A.rs.sel_w ? A.rs.sel_w[(size_t)blockIdx.x * A.rs.top + k] : 1.0f) : 0.0f;
         }
-        if (A.rs.yp) {
-            for (int k = 0; k < A.rs.top; ++k) {
-                const int slot = A.rs.slot_of[(size_t)blockIdx.x * A.rs.top + k];
-                const float wk = A.s_routed * (A.rs.sel_w ? A.rs.sel_w[(size_t)blockIdx.x * A.rs.top + k] : 1.0f);
+        float xv[kRowRegs], yv[kRowRegs], nw[kRowRegs], nb[kRowRegs];
+        row_load<VEC>(A.x + o, D, 0.0f, xv);
+        if (A.y) row_load<VEC>(A.y + o, D, 0.0f, yv);
+        if (A.next.w) row_load<VEC>(A.next.w, D, 0.0f, nw);
+        if (dyt_r || layer_r) row_load<VEC>(A.next.shift, D, 0.0f, nb);
+        auto add_routed = [&](int slot, float wk) {
+            float e[kRowRegs];
+            row_load<VEC>(A.rs.yp + (size_t)slot * D, D, 0.0f, e);
 #pragma unroll
-                for (int i = 0; i < kRowRegs; ++i) {
-                    const int c = threadIdx.x + i * blockDim.x;
-                    if (c < D) xv[i] = fmaf(wk, slot >= 0 ? A.rs.yp[(size_t)slot * D + c] : to_f<T>(hin[o + c]), xv[i]);
-                }
-            }
+            for (int i = 0; i < kRowRegs; ++i) xv[i] = fmaf(wk, e[i], xv[i]);
+        };
+        if (A.rs.yp) {
+#pragma unroll
+            for (int k = 0; k < kAhead; ++k)
+                if (k < A.rs.top) add_routed(slot_r[k], wt_r[k]);
+            for (int k = kAhead; k < A.rs.top; ++k)
+                add_routed(A.rs.slot_of[(size_t)blockIdx.x * A.rs.top + k],
+                           A.s_routed * (A.rs.sel_w ? A.rs.sel_w[(size_t)blockIdx.x * A.rs.top + k] : 1.0f));
         }
         if (A.y_w || A.y2_w) {
+            float zv[kRowRegs], a1[kRowRegs], a2[kRowRegs];
+#pragma unroll
+            for (int i = 0; i < kRowRegs; ++i) zv[i] = 0.0f, a1[i] = a2[i] = 1.0f;
+            if (A.y2) row_load<VEC>(A.y2 + o, D, 0.0f, zv);
+            if (A.y_w) row_load<VEC>(A.y_w, D, 1.0f, a1);
+            if (A.y2_w) row_load<VEC>(A.y2_w, D, 1.0f, a2);
             float s1 = 0.0f, s2 = 0.0f, s3 = 0.0f;
 #pragma unroll
             for (int i = 0; i < kRowRegs; ++i) {
@@ -185,46 +242,41 @@ __global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn, c
             if (A.y_w) r1 = A.sy / sqrtf(s1 / (float)D + A.eps);
             if (A.y2_w) r2 = A.sy2 / sqrtf(s2 / (float)D + A.eps);
             __syncthreads();
-        }
-        float ss = 0.0f;
 #pragma unroll
-        for (int i = 0; i < kRowRegs; ++i) {
-            const int c = threadIdx.x + i * blockDim.x;
-            if (c >= D) continue;
-            float v = fmaf(r2 * a2[i], zv[i], fmaf(r1 * a1[i], yv[i], xv[i]));
-            if (A.trace) A.trace[o + c] = v;
-            v += e0[i];
-            A.x[o + c] = v;
-            xv[i] = v;
-            ss = layer_r ? ss + v : fmaf(v, v, ss);
-            if (A.cat) static_cast<T*>(A.cat)[2 * o + c] = from_f<T>(v);
-            if (dyt_r) hn[o + c] = from_f<T>(fmaf(tanhf(alpha_r * v), nw[i], nb[i]));
-        }
-        if (!A.next.w || dyt_r) return;
-        if (layer_r) {
-            const float mean = block_sum(ss, red3[0]) / (float)D;
-            float q = 0.0f;
+            for (int i = 0; i < kRowRegs; ++i) xv[i] = fmaf(r2 * a2[i], zv[i], fmaf(r1 * a1[i], yv[i], xv[i]));
+        } else if (A.y) {
 #pragma unroll
-            for (int i = 0; i < kRowRegs; ++i) {
-                xv[i] -= mean;
-                if ((int)(threadIdx.x + i * blockDim.x) < D) q = fmaf(xv[i], xv[i], q);
-            }
-            const float r = 1.0f / sqrtf(block_sum(q, red3[1]) / (float)D + A.next.eps);
-#pragma unroll
-            for (int i = 0; i < kRowRegs; ++i) {
-                const int c = threadIdx.x + i * blockDim.x;
-                if (c < D) hn[o + c] = from_f<T>(fmaf(xv[i] * r, nw[i], nb[i]));
-            }
-            return;
+            for (int i = 0; i < kRowRegs; ++i) xv[i] = fmaf(r1, yv[i], xv[i]);
         }
-        float q2 = 0.0f, q3 = 0.0f;
-        block_sum3(ss, q2, q3, red3);
-        const float r = 1.0f / sqrtf(ss / (float)D + A.next.eps);
+        if (A.trace) row_store<VEC, float>(A.trace + o, D, xv);
+        if (A.x0) {
+            float e0[kRowRegs];
+            row_load<VEC>(A.x0 + o, D, 0.0f, e0);
 #pragma unroll
-        for (int i = 0; i < kRowRegs; ++i) {
-            const int c = threadIdx.x + i * blockDim.x;
-            if (c < D) hn[o + c] = from_f<T>(xv[i] * r * nw[i]);
+            for (int i = 0; i < kRowRegs; ++i) xv[i] += e0[i];
         }
+        row_store<VEC, float>(A.x + o, D, xv);
+        if (A.cat) row_store<VEC, T>(static_cast<T*>(A.cat) + 2 * o, D, xv);
+        if (!A.next.w) return;
+        if (dyt_r) {
+#pragma unroll
+            for (int i = 0; i < kRowRegs; ++i) xv[i] = fmaf(tanhf(alpha_r * xv[i]), nw[i], nb[i]);
+        } else if (layer_r) {
+            float mean, m2;
+            row_stats<VEC>(xv, D, red3, mean, m2);
+            const float r = 1.0f / sqrtf(m2 / (float)D + A.next.eps);
+#pragma unroll
+            for (int i = 0; i < kRowRegs; ++i) xv[i] = fmaf((xv[i] - mean) * r, nw[i], nb[i]);
+        } else {
+            float ss = 0.0f, q2 = 0.0f, q3 = 0.0f;
+#pragma unroll
+            for (int i = 0; i < kRowRegs; ++i) ss = fmaf(xv[i], xv[i], ss);      // beyond D: zeros
+            block_sum3(ss, q2, q3, red3);
+            const float r = 1.0f / sqrtf(ss / (float)D + A.next.eps);
+#pragma unroll
+            for (int i = 0; i < kRowRegs; ++i) xv[i] = xv[i] * r * nw[i];
+        }
+        row_store<VEC, T>(hn + o, D, xv);
         return;
     }
     if (A.y_w || A.y2_w) {
@@ -250,8 +302,7 @@ __global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn, c
             float acc = 0.0f;
             for (int k = 0; k < A.rs.top; ++k) {
                 const int slot = A.rs.slot_of[(size_t)blockIdx.x * A.rs.top + k];
-                const float e = slot >= 0 ? A.rs.yp[(size_t)slot * D + c] : to_f<T>(hin[o + c]);
-                acc = fmaf(A.rs.sel_w ? A.rs.sel_w[(size_t)blockIdx.x * A.rs.top + k] : 1.0f, e, acc);
+                acc = fmaf(A.rs.sel_w ? A.rs.sel_w[(size_t)blockIdx.x * A.rs.top + k] : 1.0f, A.rs.yp[(size_t)slot * D + c], acc);
             }
             v = fmaf(A.s_routed, acc, v);
         }
@@ -265,7 +316,7 @@ __global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn, c
     }
     if (!A.next.w || dyt) return;
     if (A.next.kind == SMOL_LM_NORM_LAYER) {
-        layer_norm_row<T>(A.next, D, hn + o, red3[0], [&](int c) { return row[c]; });
+        layer_norm_row<T>(A.next, D, hn + o, red3, [&](int c) { return row[c]; });
         return;
     }
     float s2 = 0.0f, s3 = 0.0f;
