@@ -23,7 +23,7 @@
 extern "C" {
 #endif
 
-#define SMOL_LM_ABI_VERSION 5
+#define SMOL_LM_ABI_VERSION 6
 
 enum { SMOL_LM_BF16 = 0, SMOL_LM_F32 = 1 };
 /* token mixers */
@@ -42,8 +42,12 @@ enum {
                                           per head; RMS norm over all heads together and a sigmoid gate per channel */
     SMOL_LM_MIX_HGRN2 = 7,             /* linear attention whose forget gate f (bounded below per channel) also writes: key = 1 - f;
                                           state [dim, vdim] per head; RMS norm per head */
-    SMOL_LM_MIX_RETENTION = 8          /* linear attention with one constant decay per head and rotated queries and keys; state
+    SMOL_LM_MIX_RETENTION = 8,         /* linear attention with one constant decay per head and rotated queries and keys; state
                                           [dim, vdim] per head; weightless RMS division per head and a silu gate per channel */
+    SMOL_LM_MIX_GATED_DELTA = 9,       /* delta rule with one decay and one step size per head and token behind short causal
+                                          convolutions; state [dim, vdim] per head plus the convolutions' last inputs in the slot */
+    SMOL_LM_MIX_MLSTM = 10             /* matrix memory with exponential input and sigmoid forget gate; state [dim, vdim], key sum
+                                          [dim] and running maximum per head in the slot */
 };
 /* feed-forward kinds */
 enum {
@@ -72,6 +76,9 @@ enum {
                                           stream becomes a weighted sum of the embedding output and every layer's result */
     SMOL_LM_BLOCK_PRENORM = 2,         /* x += sublayer(norm(x)) with the norm SmolLmConfig.norm_kind names; a run flagged
                                           SMOL_LM_RUN_ADD_EMBED starts from x + the embedding output */
+    SMOL_LM_BLOCK_OUTNORM = 4,         /* x += rms_divide(sublayer(x)) * norm: only the sublayers' outputs are normed, by norm1 and norm2
+                                          (plain weights); out_bias joins the mixer's output before that.  Feed-forwards: none or
+                                          dense.  w_in has zero rows behind the mixers' up to a multiple of 8 */
     SMOL_LM_BLOCK_PARALLEL = 3         /* x += residual_mult * (mixer(h) + feed-forward(h)), h = norm1(x) read by both (norms as in the
                                           pre-norm block).  Feed-forwards: none or routed.  w_in holds, after the mixer's rows, what
                                           the feed-forward needs of the same input: the shared expert's gate and up rows [shared_ff
@@ -209,6 +216,27 @@ typedef struct SmolLmLayer {
     /* --- feed-forward options --- */
     const float* router_bias; /* added to the router's logits themselves [n_experts + n_identity] (NULL: none) */
     int32_t shared_gate;      /* 1: the shared expert's result is multiplied by sigmoid of one gate row's product with the input (parallel block) */
+    /* --- options of the softmax attention: differential form.  n_maps 2: every head has two score maps over the same values -- w_in
+     *     rows q [heads][2][dim] | k [kv_heads][2][dim] | v | gate, q_norm / k_norm [dim] shared by heads and maps; with a and b the
+     *     maps' results the head's is rms_divide(a - diff_lambda * b) * diff_scale, before its gate (0 or 1: one map) --- */
+    int32_t n_maps;
+    float diff_lambda, diff_scale;
+    int32_t kv_from;          /* 1 + index of an earlier layer of the same kind and sizes whose cached keys and values this one reads (its
+                                 latest run's); w_in then holds no k and v rows.  0: own keys and values */
+    /* --- options of the softmax attention with norm_whole: rotation of q and k after the norm by rot_dims / rot_base / rot_half as in
+     *     retention; rot_yarn > 0 interpolates the frequencies: with dim(t) = rot_dims ln(rot_original / (2 pi t)) / (2 ln rot_base),
+     *     lo = max(floor(dim(rot_fast)), 0), hi = min(ceil(dim(rot_slow)), rot_dims - 1), pair i goes from f to f / rot_yarn along
+     *     clamp((i - lo) / max(hi - lo, 0.001), 0, 1); rot_mult multiplies cosine and sine (0: 1) --- */
+    float rot_mult, rot_yarn, rot_fast, rot_slow;
+    /* --- gated delta rule (w_in rows: q | k [kv_heads*dim each] | v | gate [heads*vdim each] | step [heads] | decay [heads]): q, k and v
+     *     pass the convolution conv_w [2*kv_heads*dim + heads*vdim][conv_taps] and silu; q and k become unit vectors (sum of squares +
+     *     unit_eps), q times score_scale; b = sigmoid(step), w = exp(-exp(a_log) softplus(decay + dt_bias)); S <- w S,
+     *     S <- S + k (b (v - S^T k))^T, o = S^T q; RMS division per head, times out_norm [vdim], times silu(gate) --- */
+    /* --- mLSTM (w_in rows: q | k [heads*dim each] | v | gate [heads*vdim each] | input [heads] | forget [heads]; rate_bias and decay_bias
+     *     [heads] join the input and forget rows): i = gate_cap tanh(input / gate_cap), f = ln sigmoid(gate_cap tanh(forget / gate_cap)),
+     *     m <- max(f + m, i), S <- exp(f + m_old - m) S + exp(i - m) k v^T, n likewise with k alone, q times score_scale,
+     *     o = S^T q / (max(|n.q|, exp(-m)) + den_eps); RMS division per head, times out_norm [heads*vdim], times sigmoid(gate) --- */
+    float gate_cap, den_eps;
 } SmolLmLayer;
 
 typedef struct SmolLmConfig {

@@ -11,7 +11,7 @@ import os
 from . import build as _build
 from ._errors import SMOL_OK, SmolError
 
-SMOL_LM_ABI_VERSION = 5
+SMOL_LM_ABI_VERSION = 6
 SMOL_LM_BF16, SMOL_LM_F32 = 0, 1
 
 
@@ -39,7 +39,9 @@ SmolLmLayer._fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "kv_heads", "
     (n, C.c_void_p) for n in ("head_bias", "talk")] + [(n, C.c_float) for n in ("rot_stretch", "rot_low", "rot_high", "rot_original")] + [
     (n, C.c_void_p) for n in ("head_decay", "forget_lower", "proj_norm")] + [
     (n, C.c_int32) for n in ("ff_plain", "group_rank_top", "shared_ff")] + [(n, C.c_void_p) for n in ("w_shared_in", "w_shared_out")] + [
-    ("q_temp_coef", C.c_float), ("q_temp_every", C.c_float), ("rot_half", C.c_int32), ("router_bias", C.c_void_p), ("shared_gate", C.c_int32)]
+    ("q_temp_coef", C.c_float), ("q_temp_every", C.c_float), ("rot_half", C.c_int32), ("router_bias", C.c_void_p), ("shared_gate", C.c_int32), ("n_maps", C.c_int32),
+    ("diff_lambda", C.c_float), ("diff_scale", C.c_float), ("kv_from", C.c_int32)] + [
+    (n, C.c_float) for n in ("rot_mult", "rot_yarn", "rot_fast", "rot_slow", "gate_cap", "den_eps")]
 
 
 class SmolLmConfig(C.Structure):

@@ -598,6 +598,9 @@ __global__ void __launch_bounds__(kTcThreads, 1) gemm_tc_kernel(const __grid_con
 // a query at position i to the keys 0 <= i - j < window; `softcap` > 0 bends the scaled score to softcap * tanh(score /
 // softcap) before the penalties; `slope` takes slope_h * (i - j) off.  The result is multiplied by out_scale and written
 // with the row stride out_ld (two mixers side by side share one buffer).
+// Differential attention (maps 2): every head has two softmax maps over the same values -- query rows [H][maps][d], key rows
+// [G][maps][d], a cached position holding G * maps key rows and G value rows; with a and b the maps' results a head's output is
+// o = a - diff_lambda * b, divided by its root mean square over dv, times diff_scale, before the gate.
 struct AttnArgs {
     const float* proj;
     int n_in;
@@ -619,6 +622,12 @@ struct AttnArgs {
     int window, has_gate, out_ld;
     float softcap, two_over_cap, out_scale;      // two_over_cap = 2 / softcap (0 without a cap)
     float temp_coef = 0.0f, temp_every = 0.0f;   // query temperature (temp_every 0: none), see attn_temperature
+    int maps = 1;                                // softmax maps per head
+    float diff_lambda = 0.0f, diff_scale = 1.0f;
+    int own_kv = 1;                              // 0: the cached keys and values are another layer's, the projection holds none
+    int rot_pairs = 0, rot_half = 0;             // rotated pairs of q and k (whole-projection norms only): i with i + rot_pairs, or 2i with 2i + 1
+    float rot_mult = 1.0f;                       // multiplies cosine and sine
+    const float* freq = nullptr;                 // [rot_pairs]
 };
 
 // what a query at `pos` is multiplied by: 1 + coef * ln(floor((pos + 1) / every) + 1)
@@ -643,17 +652,18 @@ __device__ __forceinline__ float attn_score(const AttnArgs& A, float dot, int di
     return s;
 }
 
-// One warp per (token, slot): slots 0..H-1 norm a query head into qbuf (times the query temperature), H..H+G-1 norm a key head
-// into the pool, H+G..H+2G-1 copy a value head into the pool.  q_norm / k_norm == nullptr: no norm.
+// One warp per (token, slot): the first H * maps slots norm a query row into qbuf (times the query temperature), the next
+// G * maps norm a key row into the pool, the last G copy a value head into the pool (own_kv 0: query rows only).
+// q_norm / k_norm == nullptr: no norm.
 template <class T>
 __global__ void attn_prep_kernel(const AttnArgs A, T* __restrict__ qbuf, T* __restrict__ pool) {
     const int lane = threadIdx.x & 31;
     const int unit = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    const int slots = A.H + 2 * A.G;
+    const int HQ = A.H * A.maps, GK = A.G * A.maps, slots = HQ + (A.own_kv ? GK + A.G : 0);
     if (unit >= A.n_tokens * slots) return;
     const int t = unit / slots, s = unit % slots;
     const float* row = A.proj + (size_t)t * A.n_in;
-    if (s < A.H) {
+    if (s < HQ) {
         const float* q = row + s * A.d;
         const float* qb = A.bias ? A.bias + s * A.d : nullptr;
         float ss = 0.0f;
@@ -661,7 +671,7 @@ __global__ void attn_prep_kernel(const AttnArgs A, T* __restrict__ qbuf, T* __re
         ss = warp_sum(ss);
         const float r = (A.q_norm ? 1.0f / sqrtf(ss / (float)A.d + A.eps) : 1.0f) * attn_temperature(A, A.tok_pos[t]);
         for (int c = lane; c < A.d; c += 32)
-            qbuf[((size_t)t * A.H + s) * A.d + c] = from_f<T>((q[c] + (qb ? qb[c] : 0.0f)) * r * (A.q_norm ? A.q_norm[c] : 1.0f));
+            qbuf[((size_t)t * HQ + s) * A.d + c] = from_f<T>((q[c] + (qb ? qb[c] : 0.0f)) * r * (A.q_norm ? A.q_norm[c] : 1.0f));
         return;
     }
     const int pos = A.tok_pos[t];
@@ -672,10 +682,10 @@ __global__ void attn_prep_kernel(const AttnArgs A, T* __restrict__ qbuf, T* __re
         return;
     }
     T* base = pool + (size_t)page * A.page_elems;
-    if (s < A.H + A.G) {
-        const int gk = s - A.H;
-        const float* k = row + A.H * A.d + gk * A.d;
-        const float* kb = A.bias ? A.bias + A.H * A.d + gk * A.d : nullptr;
+    if (s < HQ + GK) {
+        const int gk = s - HQ;
+        const float* k = row + HQ * A.d + gk * A.d;
+        const float* kb = A.bias ? A.bias + HQ * A.d + gk * A.d : nullptr;
         float ss = 0.0f;
         for (int c = lane; c < A.d; c += 32) { const float v = k[c] + (kb ? kb[c] : 0.0f); ss += v * v; }
         ss = warp_sum(ss);
@@ -683,9 +693,9 @@ __global__ void attn_prep_kernel(const AttnArgs A, T* __restrict__ qbuf, T* __re
         T* dst = base + A.k_off + ((size_t)gk * A.page_size + in_pg) * A.d;
         for (int c = lane; c < A.d; c += 32) dst[c] = from_f<T>((k[c] + (kb ? kb[c] : 0.0f)) * r * (A.k_norm ? A.k_norm[c] : 1.0f));
     } else {
-        const int gv = s - A.H - A.G;
-        const float* v = row + (A.H + A.G) * A.d + gv * A.dv;
-        const float* vb = A.bias ? A.bias + (A.H + A.G) * A.d + gv * A.dv : nullptr;
+        const int gv = s - HQ - GK;
+        const float* v = row + (HQ + GK) * A.d + gv * A.dv;
+        const float* vb = A.bias ? A.bias + (HQ + GK) * A.d + gv * A.dv : nullptr;
         T* dst = base + A.v_off + ((size_t)gv * A.page_size + in_pg) * A.dv;
         for (int c = lane; c < A.dv; c += 32) dst[c] = from_f<T>(v[c] + (vb ? vb[c] : 0.0f));
     }
@@ -694,11 +704,14 @@ __global__ void attn_prep_kernel(const AttnArgs A, T* __restrict__ qbuf, T* __re
 // The same preparation with query and key norms over the WHOLE projection: one root mean square for all query heads of a
 // token (weights q_norm [H*d]) and one for all key heads (k_norm [G*d]).  One block per token.  Loads go out kPrepBatch
 // at a time before their first use: a lone token (decoding) waits for memory a few times, not once per element.
+// ROT: queries and keys are rotated after the norm, the token's cosines and sines taken once for all heads.
 constexpr int kPrepBatch = 4;
+constexpr int kMaxRotPairs = 256;
 
-template <class T>
+template <class T, bool ROT>
 __global__ void __launch_bounds__(256) attn_prep_whole_kernel(const AttnArgs A, T* __restrict__ qbuf, T* __restrict__ pool) {
     __shared__ float red[2][33];
+    __shared__ float turn[2][ROT ? kMaxRotPairs : 1];
     const int t = blockIdx.x, nq = A.H * A.d, nk = A.G * A.d, nv = A.G * A.dv;
     const float* row = A.proj + (size_t)t * A.n_in;
     const int pos = A.tok_pos[t];
@@ -720,6 +733,13 @@ __global__ void __launch_bounds__(256) attn_prep_whole_kernel(const AttnArgs A, 
         }
         return ss;
     };
+    if (ROT)
+        for (int i = threadIdx.x; i < A.rot_pairs; i += blockDim.x) {
+            float sn, cs;
+            sincosf((float)pos * A.freq[i], &sn, &cs);
+            turn[0][i] = cs * A.rot_mult;
+            turn[1][i] = sn * A.rot_mult;
+        }
     float sq = sum_sq(0, nq), sk = sum_sq(nq, nk);
     sq = warp_sum(sq);
     sk = warp_sum(sk);
@@ -747,13 +767,44 @@ __global__ void __launch_bounds__(256) attn_prep_whole_kernel(const AttnArgs A, 
             }
         }
     };
-    emit(0, nq, rq * attn_temperature(A, pos), A.q_norm, [&](int c, float v) { qbuf[(size_t)t * nq + c] = from_f<T>(v); });
+    // the same with the rotation: a rotated element also reads its pair's other one
+    auto emit_rotated = [&](int lo, int n, float mul, const float* weight, auto store) {
+        for (int c0 = threadIdx.x; c0 < n; c0 += blockDim.x * kPrepBatch) {
+            float v[kPrepBatch], o[kPrepBatch], cs[kPrepBatch], sn[kPrepBatch];
+#pragma unroll
+            for (int u = 0; u < kPrepBatch; ++u) {
+                const int c = c0 + u * blockDim.x, i = c % A.d;
+                int p = 0, other = -1;
+                bool first = true;
+                if (c < n && i < 2 * A.rot_pairs) {
+                    first = A.rot_half ? i < A.rot_pairs : i % 2 == 0;
+                    p = A.rot_half ? (first ? i : i - A.rot_pairs) : i / 2;
+                    const int step = A.rot_half ? A.rot_pairs : 1;
+                    other = first ? c + step : c - step;
+                }
+                v[u] = c < n ? (row[lo + c] + (A.bias ? A.bias[lo + c] : 0.0f)) * (weight ? weight[c] : 1.0f) : 0.0f;
+                o[u] = other >= 0 ? (row[lo + other] + (A.bias ? A.bias[lo + other] : 0.0f)) * (weight ? weight[other] : 1.0f) : 0.0f;
+                cs[u] = other >= 0 ? turn[0][p] : 1.0f;
+                sn[u] = other >= 0 ? (first ? -turn[1][p] : turn[1][p]) : 0.0f;
+            }
+#pragma unroll
+            for (int u = 0; u < kPrepBatch; ++u) {
+                const int c = c0 + u * blockDim.x;
+                if (c < n) store(c, (v[u] * mul) * cs[u] + (o[u] * mul) * sn[u]);
+            }
+        }
+    };
+    auto emit_qk = [&](int lo, int n, float mul, const float* weight, auto store) {
+        if constexpr (ROT) emit_rotated(lo, n, mul, weight, store);
+        else emit(lo, n, mul, weight, store);
+    };
+    emit_qk(0, nq, rq * attn_temperature(A, pos), A.q_norm, [&](int c, float v) { qbuf[(size_t)t * nq + c] = from_f<T>(v); });
     if (page < 0 || page >= A.n_pages) {
         if (threadIdx.x == 0) atomicExch(A.err, 1);
         return;
     }
     T* base = pool + (size_t)page * A.page_elems;
-    emit(nq, nk, rk, A.k_norm, [&](int c, float v) {
+    emit_qk(nq, nk, rk, A.k_norm, [&](int c, float v) {
         const int g = c / A.d, i = c - g * A.d;
         base[A.k_off + ((size_t)g * A.page_size + in_pg) * A.d + i] = from_f<T>(v);
     });
@@ -774,7 +825,25 @@ __device__ __forceinline__ float attn_gate(const AttnArgs& A, size_t t, int h, i
     return A.out_scale * sigmoidf_(A.proj[t * A.n_in + A.gate_off + (size_t)h * A.gate_ld + (size_t)c * A.gate_step]);
 }
 
-template <class T, int MAXV>
+// A head's finished result from the columns a warp holds (column lane + 32 e in o[e], the maps already joined): the
+// differential form's division by the root mean square, then the gate.
+template <class T, int MAXV, int MAPS>
+__device__ __forceinline__ void attn_finish(const AttnArgs& A, size_t t, int h, int lane, float (&o)[MAXV], T* __restrict__ out) {
+    float r = 1.0f;
+    if (MAPS == 2) {
+        float ss = 0.0f;
+#pragma unroll
+        for (int e = 0; e < MAXV; ++e) ss = fmaf(o[e], o[e], ss);      // columns beyond dv hold zeros
+        r = A.diff_scale / sqrtf(warp_sum(ss) / (float)A.dv + A.eps);
+    }
+#pragma unroll
+    for (int e = 0; e < MAXV; ++e) {
+        const int c = lane + e * 32;
+        if (c < A.dv) out[t * A.out_ld + h * A.dv + c] = from_f<T>((MAPS == 2 ? o[e] * r : o[e]) * attn_gate(A, t, h, c));
+    }
+}
+
+template <class T, int MAXV, int MAPS>
 __global__ void __launch_bounds__(kAttnWarps * 32) attn_kernel(const AttnArgs A, const T* __restrict__ qbuf, const T* __restrict__ pool,
                                                                T* __restrict__ out) {
     extern __shared__ float qs_all[];
@@ -784,52 +853,55 @@ __global__ void __launch_bounds__(kAttnWarps * 32) attn_kernel(const AttnArgs A,
     const int t = unit / A.H, h = unit % A.H;
     const int g = h / (A.H / A.G);
     float* qs = qs_all + warp * A.d;
-    for (int c = lane; c < A.d; c += 32) qs[c] = to_f<T>(qbuf[((size_t)t * A.H + h) * A.d + c]);
-    __syncwarp();
     const int pos = A.tok_pos[t];
     const int32_t* bt = A.block_table + (size_t)A.tok_seq[t] * A.max_pages;
     const float r1 = A.r1 ? A.r1[h] : 0.0f, r2 = A.r1 ? A.r2[h] : 0.0f, slope = A.slope ? A.slope[h] : 0.0f;
-    float m = A.sink ? A.sink[h] : -INFINITY, l = A.sink ? 1.0f : 0.0f;
-    float o[MAXV];
+    float sum[MAXV];                    // the maps' joined result
 #pragma unroll
-    for (int e = 0; e < MAXV; ++e) o[e] = 0.0f;
-    for (int j0 = attn_first_key(A, pos); j0 <= pos; j0 += 32) {
-        const int j = j0 + lane;
-        float s = -INFINITY;
-        const T* vrow = nullptr;
-        if (j <= pos) {
-            const int page = bt[j / A.page_size], in_pg = j % A.page_size;
-            const T* base = pool + (size_t)page * A.page_elems;
-            const T* k = base + A.k_off + ((size_t)g * A.page_size + in_pg) * A.k_ld;
-            vrow = base + A.v_off + ((size_t)g * A.page_size + in_pg) * A.v_ld;
-            float dot = 0.0f;
-            for (int c = 0; c < A.d; ++c) dot = fmaf(qs[c], to_f<T>(k[c]), dot);
-            s = attn_score<false>(A, dot, pos - j, r1, r2, slope);
-        }
-        const float mn = fmaxf(m, warp_max(s));          // finite: lane 0 of every round holds a visible key
-        const float p = (j <= pos) ? expf(s - mn) : 0.0f;
-        const float corr = expf(m - mn);
-        l = l * corr + warp_sum(p);
-        m = mn;
+    for (int map = 0; map < MAPS; ++map) {
+        __syncwarp();
+        for (int c = lane; c < A.d; c += 32) qs[c] = to_f<T>(qbuf[(((size_t)t * A.H + h) * MAPS + map) * A.d + c]);
+        __syncwarp();
+        float m = A.sink ? A.sink[h] : -INFINITY, l = A.sink ? 1.0f : 0.0f;
+        float o[MAXV];
 #pragma unroll
-        for (int e = 0; e < MAXV; ++e) o[e] *= corr;
-        const int cnt = min(32, pos - j0 + 1);
-        for (int jj = 0; jj < cnt; ++jj) {
-            const float pj = __shfl_sync(0xffffffffu, p, jj);
-            const T* vr = reinterpret_cast<const T*>(__shfl_sync(0xffffffffu, reinterpret_cast<unsigned long long>(vrow), jj));
+        for (int e = 0; e < MAXV; ++e) o[e] = 0.0f;
+        for (int j0 = attn_first_key(A, pos); j0 <= pos; j0 += 32) {
+            const int j = j0 + lane;
+            float s = -INFINITY;
+            const T* vrow = nullptr;
+            if (j <= pos) {
+                const int page = bt[j / A.page_size], in_pg = j % A.page_size;
+                const T* base = pool + (size_t)page * A.page_elems;
+                const T* k = base + A.k_off + ((size_t)(g * MAPS + map) * A.page_size + in_pg) * A.k_ld;
+                vrow = base + A.v_off + ((size_t)g * A.page_size + in_pg) * A.v_ld;
+                float dot = 0.0f;
+                for (int c = 0; c < A.d; ++c) dot = fmaf(qs[c], to_f<T>(k[c]), dot);
+                s = attn_score<false>(A, dot, pos - j, r1, r2, slope);
+            }
+            const float mn = fmaxf(m, warp_max(s));          // finite: lane 0 of every round holds a visible key
+            const float p = (j <= pos) ? expf(s - mn) : 0.0f;
+            const float corr = expf(m - mn);
+            l = l * corr + warp_sum(p);
+            m = mn;
 #pragma unroll
-            for (int e = 0; e < MAXV; ++e) {
-                const int c = lane + e * 32;
-                if (c < A.dv) o[e] = fmaf(pj, to_f<T>(vr[c]), o[e]);
+            for (int e = 0; e < MAXV; ++e) o[e] *= corr;
+            const int cnt = min(32, pos - j0 + 1);
+            for (int jj = 0; jj < cnt; ++jj) {
+                const float pj = __shfl_sync(0xffffffffu, p, jj);
+                const T* vr = reinterpret_cast<const T*>(__shfl_sync(0xffffffffu, reinterpret_cast<unsigned long long>(vrow), jj));
+#pragma unroll
+                for (int e = 0; e < MAXV; ++e) {
+                    const int c = lane + e * 32;
+                    if (c < A.dv) o[e] = fmaf(pj, to_f<T>(vr[c]), o[e]);
+                }
             }
         }
-    }
-    const float inv = 1.0f / l;
+        const float inv = 1.0f / l;
 #pragma unroll
-    for (int e = 0; e < MAXV; ++e) {
-        const int c = lane + e * 32;
-        if (c < A.dv) out[(size_t)t * A.out_ld + h * A.dv + c] = from_f<T>(o[e] * inv * attn_gate(A, t, h, c));
+        for (int e = 0; e < MAXV; ++e) sum[e] = map == 0 ? o[e] * inv : fmaf(-A.diff_lambda, o[e] * inv, sum[e]);
     }
+    attn_finish<T, MAXV, MAPS>(A, t, h, lane, sum, out);
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
@@ -879,7 +951,8 @@ template <> __device__ __forceinline__ float key_dot<bf16>(const float* qs, cons
 
 template <class T, int MAXV>
 __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const T* __restrict__ qbuf, const T* __restrict__ pool) {
-    // One block per (row, key/value head x group of up to 8 of its query heads, key range); one warp per query head.
+    // One block per (row, key/value head x group of up to 8 of its query rows, key range); one warp per query row (a query
+    // head, or one of its maps: the block then stages every map's keys beside the values they share).
     // 32 keys and values at a time are staged in shared memory (rows padded by 16 bytes: conflict-free row-per-lane
     // reads), so that no global load sits inside the softmax / value loops.
     extern __shared__ __align__(16) unsigned char sm_raw[];
@@ -894,20 +967,20 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
     if (range * A.split_len > pos) return;
     const int j_lo = max(range * A.split_len, j_first);
     const int j_hi = min(pos, (range + 1) * A.split_len - 1);
-    const int Gq = A.H / A.G, nwarp = blockDim.x >> 5;
+    const int Gq = A.H / A.G * A.maps, nwarp = blockDim.x >> 5;
     const int groups = (Gq + nwarp - 1) / nwarp;
     const int g = blockIdx.y / groups, hq = (blockIdx.y % groups) * nwarp + (threadIdx.x >> 5);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bool active = hq < Gq;
-    const int h = g * Gq + (active ? hq : 0);
+    const int h = g * Gq + (active ? hq : 0), map = h % A.maps, head = h / A.maps;      // h: query row
     const int ldk = A.d + kPad, ldv = A.v_in_k ? ldk : A.dv + kPad;
     float* qs = reinterpret_cast<float*>(sm_raw) + warp * A.d;
     float* ps = reinterpret_cast<float*>(sm_raw) + nwarp * A.d + warp * 32;
     T* Ks = reinterpret_cast<T*>(sm_raw + (((size_t)nwarp * (A.d + 32) * 4 + 15) / 16) * 16);
-    T* Vs = A.v_in_k ? Ks : Ks + 32 * ldk;
+    T* Vs = A.v_in_k ? Ks : Ks + 32 * ldk * A.maps;
     const int32_t* bt = A.block_table + (size_t)s * A.max_pages;
-    for (int c = lane; c < A.d; c += 32) qs[c] = to_f<T>(qbuf[((size_t)t * A.H + h) * A.d + c]);
-    const float r1 = A.r1 ? A.r1[h] : 0.0f, r2 = A.r1 ? A.r2[h] : 0.0f, slope = A.slope ? A.slope[h] : 0.0f;
+    for (int c = lane; c < A.d; c += 32) qs[c] = to_f<T>(qbuf[((size_t)t * A.H * A.maps + h) * A.d + c]);
+    const float r1 = A.r1 ? A.r1[head] : 0.0f, r2 = A.r1 ? A.r2[head] : 0.0f, slope = A.slope ? A.slope[head] : 0.0f;
     float m = -INFINITY, l = 0.0f;
     float o[MAXV];
 #pragma unroll
@@ -915,7 +988,7 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
     // whole 16-byte pieces when every cached row starts on a 16-byte boundary (pages are 16-byte aligned)
     const bool kvec = (A.d * sizeof(T)) % 16 == 0 && (A.k_ld * sizeof(T)) % 16 == 0 && (A.k_off * sizeof(T)) % 16 == 0;
     const bool vvec = (A.dv * sizeof(T)) % 16 == 0 && (A.v_ld * sizeof(T)) % 16 == 0 && (A.v_off * sizeof(T)) % 16 == 0;
-    const int kchunks = kvec ? A.d / kPad : A.d, vchunks = A.v_in_k ? 0 : (vvec ? A.dv / kPad : A.dv);
+    const int kchunk1 = kvec ? A.d / kPad : A.d, kchunks = kchunk1 * A.maps, vchunks = A.v_in_k ? 0 : (vvec ? A.dv / kPad : A.dv);
     for (int j0 = j_lo; j0 <= j_hi; j0 += 32) {
         const int cnt = min(32, j_hi - j0 + 1);
         __syncthreads();
@@ -923,14 +996,16 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
             const int row = idx / (kchunks + vchunks), c = idx % (kchunks + vchunks);
             const int j = j0 + row;
             const T* base = pool + (size_t)bt[j / A.page_size] * A.page_elems;
-            const size_t in_pg = (size_t)g * A.page_size + j % A.page_size;
+            const int in_pg = j % A.page_size;
             if (c < kchunks) {
-                const T* src = base + A.k_off + in_pg * A.k_ld;
-                if (kvec) cp_async16(Ks + row * ldk + c * kPad, src + c * kPad);
-                else Ks[row * ldk + c] = src[c];
+                const int km = c / kchunk1, ck = c - km * kchunk1;
+                const T* src = base + A.k_off + ((size_t)(g * A.maps + km) * A.page_size + in_pg) * A.k_ld;
+                T* dst = Ks + (km * 32 + row) * ldk;
+                if (kvec) cp_async16(dst + ck * kPad, src + ck * kPad);
+                else dst[ck] = src[ck];
             } else {
                 const int cv = c - kchunks;
-                const T* src = base + A.v_off + in_pg * A.v_ld;
+                const T* src = base + A.v_off + ((size_t)g * A.page_size + in_pg) * A.v_ld;
                 if (vvec) cp_async16(Vs + row * ldv + cv * kPad, src + cv * kPad);
                 else Vs[row * ldv + cv] = src[cv];
             }
@@ -942,7 +1017,7 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
         const int j = j0 + lane;
         float sc = -INFINITY;
         if (lane < cnt) {
-            sc = attn_score<false>(A, key_dot<T>(qs, Ks + lane * ldk, A.d), pos - j, r1, r2, slope);
+            sc = attn_score<false>(A, key_dot<T>(qs, Ks + (map * 32 + lane) * ldk, A.d), pos - j, r1, r2, slope);
         }
         const float mn = fmaxf(m, warp_max(sc));          // finite: lane 0 of every round holds a valid key
         const float p = lane < cnt ? expf(sc - mn) : 0.0f;
@@ -964,7 +1039,7 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
         __syncwarp();
     }
     if (!active) return;
-    float* dst = A.part + (((size_t)blockIdx.x * A.H + h) * A.n_splits + blockIdx.z) * (A.dv + 2);
+    float* dst = A.part + (((size_t)blockIdx.x * A.H * A.maps + h) * A.n_splits + blockIdx.z) * (A.dv + 2);
     if (lane == 0) { dst[0] = m; dst[1] = l; }
 #pragma unroll
     for (int e = 0; e < MAXV; ++e) {
@@ -973,8 +1048,8 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
     }
 }
 
-// One warp per (row, query head): merges the ranges; the sink enters here, once, with no value.
-template <class T, int MAXV>
+// One warp per (row, query head): merges the ranges of every map and joins the maps; the sink enters here, once, with no value.
+template <class T, int MAXV, int MAPS>
 __global__ void __launch_bounds__(128) attn_merge_kernel(const AttnArgs A, T* __restrict__ out) {
     const int lane = threadIdx.x & 31;
     const int unit = blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -985,43 +1060,45 @@ __global__ void __launch_bounds__(128) attn_merge_kernel(const AttnArgs A, T* __
     if (n > kShortSeq || r >= n) return;
     const int t = t0 + r, pos = A.tok_pos[t];
     const int ns = pos / A.split_len - attn_first_key(A, pos) / A.split_len + 1;
-    const float* src = A.part + ((size_t)x * A.H + h) * A.n_splits * (A.dv + 2);
-    // lanes take the ranges' maxima and weights side by side; the value columns are then summed range by range with the
-    // weights handed on by shuffles, so that no load waits for an earlier one
     const float sink = A.sink ? A.sink[h] : -INFINITY;
-    float M = sink;
-    for (int z = lane; z < ns; z += 32) M = fmaxf(M, src[(size_t)z * (A.dv + 2)]);
-    M = warp_max(M);
-    float l = 0.0f;
-    float o[MAXV];
+    float sum[MAXV];                    // the maps' joined result
 #pragma unroll
-    for (int e = 0; e < MAXV; ++e) o[e] = 0.0f;
-    for (int z0 = 0; z0 < ns; z0 += 32) {
-        const int z = z0 + lane, cnt = min(32, ns - z0);
-        float wz = 0.0f;
-        if (z < ns) {
-            const float* p = src + (size_t)z * (A.dv + 2);
-            wz = expf(p[0] - M);
-            l = fmaf(p[1], wz, l);
-        }
+    for (int map = 0; map < MAPS; ++map) {
+        const float* src = A.part + (((size_t)x * A.H + h) * MAPS + map) * A.n_splits * (A.dv + 2);
+        // lanes take the ranges' maxima and weights side by side; the value columns are then summed range by range with the
+        // weights handed on by shuffles, so that no load waits for an earlier one
+        float M = sink;
+        for (int z = lane; z < ns; z += 32) M = fmaxf(M, src[(size_t)z * (A.dv + 2)]);
+        M = warp_max(M);
+        float l = 0.0f;
+        float o[MAXV];
+#pragma unroll
+        for (int e = 0; e < MAXV; ++e) o[e] = 0.0f;
+        for (int z0 = 0; z0 < ns; z0 += 32) {
+            const int z = z0 + lane, cnt = min(32, ns - z0);
+            float wz = 0.0f;
+            if (z < ns) {
+                const float* p = src + (size_t)z * (A.dv + 2);
+                wz = expf(p[0] - M);
+                l = fmaf(p[1], wz, l);
+            }
 #pragma unroll 4
-        for (int i = 0; i < cnt; ++i) {
-            const float w = __shfl_sync(0xffffffffu, wz, i);
-            const float* p = src + (size_t)(z0 + i) * (A.dv + 2) + 2;
+            for (int i = 0; i < cnt; ++i) {
+                const float w = __shfl_sync(0xffffffffu, wz, i);
+                const float* p = src + (size_t)(z0 + i) * (A.dv + 2) + 2;
 #pragma unroll
-            for (int e = 0; e < MAXV; ++e) {
-                const int c = lane + e * 32;
-                if (c < A.dv) o[e] = fmaf(p[c], w, o[e]);
+                for (int e = 0; e < MAXV; ++e) {
+                    const int c = lane + e * 32;
+                    if (c < A.dv) o[e] = fmaf(p[c], w, o[e]);
+                }
             }
         }
-    }
-    l = warp_sum(l) + expf(sink - M);
-    const float inv = 1.0f / l;
+        l = warp_sum(l) + expf(sink - M);
+        const float inv = 1.0f / l;
 #pragma unroll
-    for (int e = 0; e < MAXV; ++e) {
-        const int c = lane + e * 32;
-        if (c < A.dv) out[(size_t)t * A.out_ld + h * A.dv + c] = from_f<T>(o[e] * inv * attn_gate(A, t, h, c));
+        for (int e = 0; e < MAXV; ++e) sum[e] = map == 0 ? o[e] * inv : fmaf(-A.diff_lambda, o[e] * inv, sum[e]);
     }
+    attn_finish<T, MAXV, MAPS>(A, t, h, lane, sum, out);
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
@@ -1039,11 +1116,11 @@ __device__ __forceinline__ void ldmatrix_x2_trans(uint32_t& r0, uint32_t& r1, co
 
 // 64 rows of `cols` bf16 into a [64][DP + 8] tile; src(row) is the row's address or nullptr (zero row).  ASYNC: whole
 // 16-byte pieces of aligned rows go by cp.async (the caller commits and waits); everything else is stored directly.
-template <int DP, bool ASYNC, class RowPtr>
+template <int DP, bool ASYNC, int NTHR, class RowPtr>
 __device__ __forceinline__ void stage_rows(bf16* dst, int cols, RowPtr src) {
     constexpr int LD = DP + 8;
     const bool vec = (cols % 8) == 0;
-    for (int idx = threadIdx.x; idx < 64 * (DP / 8); idx += 128) {
+    for (int idx = threadIdx.x; idx < 64 * (DP / 8); idx += NTHR) {
         const int row = idx / (DP / 8), c = (idx % (DP / 8)) * 8;
         const bf16* p = src(row);
         uint4 v = make_uint4(0, 0, 0, 0);
@@ -1070,31 +1147,36 @@ __device__ __forceinline__ void stage_rows(bf16* dst, int cols, RowPtr src) {
 // serves bf16 only, whose products carry 2^-9.
 // DK / DV: key and value sizes padded to multiples of 16.  VK: the values are the first columns of the key rows (a cached
 // latent that serves as both), so only key tiles are staged and DV <= DK.
-template <int DK, int DV, bool VK>
-__global__ void __launch_bounds__(128) attn_flash_kernel(const AttnArgs A, const bf16* __restrict__ qbuf, const bf16* __restrict__ pool,
+// MAPS 2 (differential attention): four warps per map, both over the one staged value tile; at the end the second map's rows
+// pass through shared memory to the first map's warps, which join and finish them.
+template <int DK, int DV, bool VK, int MAPS>
+__global__ void __launch_bounds__(128 * MAPS) attn_flash_kernel(const AttnArgs A, const bf16* __restrict__ qbuf, const bf16* __restrict__ pool,
                                                          bf16* __restrict__ out) {
     constexpr int LD = DK + 8, kTile = 64 * LD, LDV = VK ? LD : DV + 8, kTileV = 64 * LDV;
-    static_assert(!VK || DV <= DK, "values inside the key rows");
-    extern __shared__ __align__(16) unsigned char flash_smem[];      // keys [2][64][LD], values [2][64][LDV]: two tiles in turn
+    static_assert(!VK || (DV <= DK && MAPS == 1), "values inside the key rows");
+    constexpr int NTHR = 128 * MAPS;
+    extern __shared__ __align__(16) unsigned char flash_smem[];      // keys [2][MAPS][64][LD], values [2][64][LDV]: two tiles in turn
     bf16* Ks = reinterpret_cast<bf16*>(flash_smem);
-    bf16* Vs = VK ? Ks : Ks + 2 * kTile;
+    bf16* Vs = VK ? Ks : Ks + 2 * MAPS * kTile;
     const int s = blockIdx.y;
     const int t0 = A.seq_start[s], n = A.seq_start[s + 1] - t0;
     const int tile = gridDim.z - 1 - blockIdx.z;      // the tiles with the most keys start first, those of every head together
     if (n <= kShortSeq || tile * 64 >= n) return;
     const int h = blockIdx.x, g = h / (A.H / A.G);
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
+    const int map = MAPS == 1 ? 0 : threadIdx.x / 128, warp = (threadIdx.x >> 5) % 4, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
     const int pos0 = A.tok_pos[t0];
     const int32_t* bt = A.block_table + (size_t)s * A.max_pages;
     // queries of the tile -> A fragments
-    stage_rows<DK, false>(Ks, A.d, [&](int row) -> const bf16* {
-        return tile * 64 + row < n ? qbuf + ((size_t)(t0 + tile * 64 + row) * A.H + h) * A.d : nullptr;
-    });
+#pragma unroll
+    for (int mp = 0; mp < MAPS; ++mp)
+        stage_rows<DK, false, NTHR>(Ks + mp * kTile, A.d, [&](int row) -> const bf16* {
+            return tile * 64 + row < n ? qbuf + (((size_t)(t0 + tile * 64 + row) * A.H + h) * MAPS + mp) * A.d : nullptr;
+        });
     __syncthreads();
     uint32_t qf[DK / 16][4];
 #pragma unroll
     for (int kk = 0; kk < DK / 16; ++kk) {
-        const bf16* p = Ks + (warp * 16 + gq) * LD + kk * 16 + tq * 2;
+        const bf16* p = Ks + map * kTile + (warp * 16 + gq) * LD + kk * 16 + tq * 2;
         qf[kk][0] = *reinterpret_cast<const uint32_t*>(p);
         qf[kk][1] = *reinterpret_cast<const uint32_t*>(p + 8 * LD);
         qf[kk][2] = *reinterpret_cast<const uint32_t*>(p + 8);
@@ -1118,13 +1200,15 @@ __global__ void __launch_bounds__(128) attn_flash_kernel(const AttnArgs A, const
         for (int e = 0; e < 4; ++e) o[nt][e] = 0.0f;
     // the next tile of keys and values is on its way (cp.async) while the current one is multiplied
     auto stage_tile = [&](int j0, int buf) {
-        auto row_of = [&](int row, size_t off, int width) -> const bf16* {
+        auto row_of = [&](int row, size_t off, int width, int in_head) -> const bf16* {
             const int j = j0 + row;
             if (j > last_pos) return nullptr;
-            return pool + (size_t)bt[j / A.page_size] * A.page_elems + off + ((size_t)g * A.page_size + j % A.page_size) * width;
+            return pool + (size_t)bt[j / A.page_size] * A.page_elems + off + ((size_t)in_head * A.page_size + j % A.page_size) * width;
         };
-        stage_rows<DK, true>(Ks + buf * kTile, A.d, [&](int row) { return row_of(row, A.k_off, A.k_ld); });
-        if (!VK) stage_rows<DV, true>(Vs + buf * kTileV, A.dv, [&](int row) { return row_of(row, A.v_off, A.v_ld); });
+#pragma unroll
+        for (int mp = 0; mp < MAPS; ++mp)
+            stage_rows<DK, true, NTHR>(Ks + (buf * MAPS + mp) * kTile, A.d, [&](int row) { return row_of(row, A.k_off, A.k_ld, g * MAPS + mp); });
+        if (!VK) stage_rows<DV, true, NTHR>(Vs + buf * kTileV, A.dv, [&](int row) { return row_of(row, A.v_off, A.v_ld, g); });
         cp_async_commit_group();
     };
     stage_tile(j_start, 0);
@@ -1137,7 +1221,7 @@ __global__ void __launch_bounds__(128) attn_flash_kernel(const AttnArgs A, const
             cp_async_wait_group<0>();
         }
         __syncthreads();
-        const bf16* Kt = Ks + buf * kTile;
+        const bf16* Kt = Ks + (buf * MAPS + map) * kTile;
         const bf16* Vt = Vs + buf * kTileV;
         if (j0 <= pos0 + tile * 64 + warp * 16 + 15 && j0 + 63 > pos0 + tile * 64 + warp * 16 - win) {      // this warp's rows see a key of the tile
             float S[8][4];
@@ -1205,7 +1289,38 @@ __global__ void __launch_bounds__(128) attn_flash_kernel(const AttnArgs A, const
     l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 1);
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
-    const float inv_a = 1.0f / l_a, inv_b = 1.0f / l_b;
+    float inv_a = 1.0f / l_a, inv_b = 1.0f / l_b;
+    if (MAPS == 2) {
+        // (the loop's last barrier has passed: the key and value tiles are free)
+        constexpr int LDX = DV + 2;
+        float* other = reinterpret_cast<float*>(flash_smem);       // [64][LDX]
+        const int ra = warp * 16 + gq;
+        if (map == 1) {
+#pragma unroll
+            for (int nt = 0; nt < DV / 8; ++nt) {
+                *reinterpret_cast<float2*>(other + ra * LDX + nt * 8 + tq * 2) = make_float2(o[nt][0] * inv_a, o[nt][1] * inv_a);
+                *reinterpret_cast<float2*>(other + (ra + 8) * LDX + nt * 8 + tq * 2) = make_float2(o[nt][2] * inv_b, o[nt][3] * inv_b);
+            }
+        }
+        __syncthreads();
+        if (map == 1) return;
+        float sa = 0.0f, sb = 0.0f;
+#pragma unroll
+        for (int nt = 0; nt < DV / 8; ++nt) {
+            const float2 xa = *reinterpret_cast<const float2*>(other + ra * LDX + nt * 8 + tq * 2);
+            const float2 xb = *reinterpret_cast<const float2*>(other + (ra + 8) * LDX + nt * 8 + tq * 2);
+            o[nt][0] = fmaf(-A.diff_lambda, xa.x, o[nt][0] * inv_a); o[nt][1] = fmaf(-A.diff_lambda, xa.y, o[nt][1] * inv_a);
+            o[nt][2] = fmaf(-A.diff_lambda, xb.x, o[nt][2] * inv_b); o[nt][3] = fmaf(-A.diff_lambda, xb.y, o[nt][3] * inv_b);
+            sa = fmaf(o[nt][0], o[nt][0], fmaf(o[nt][1], o[nt][1], sa));
+            sb = fmaf(o[nt][2], o[nt][2], fmaf(o[nt][3], o[nt][3], sb));
+        }
+        sa += __shfl_xor_sync(0xffffffffu, sa, 1);
+        sa += __shfl_xor_sync(0xffffffffu, sa, 2);
+        sb += __shfl_xor_sync(0xffffffffu, sb, 1);
+        sb += __shfl_xor_sync(0xffffffffu, sb, 2);
+        inv_a = A.diff_scale / sqrtf(sa / (float)A.dv + A.eps);     // columns beyond dv hold zeros
+        inv_b = A.diff_scale / sqrtf(sb / (float)A.dv + A.eps);
+    }
 #pragma unroll
     for (int nt = 0; nt < DV / 8; ++nt)
 #pragma unroll
@@ -1485,6 +1600,7 @@ __global__ void __launch_bounds__(kThreads) lm_sample_kernel(const float* __rest
 
 #include "lm_mechanisms.cuh"
 #include "lm_sigmoid_linear.cuh"
+#include "lm_delta_mlstm.cuh"
 
 // =====================================================================================================================
 // Host side
@@ -1507,7 +1623,8 @@ struct RunInfo {
     size_t k_off = 0, v_off = 0;   // attention: element offsets inside a page
     size_t state_off = 0;          // recurrent: float offset inside a slot
     size_t freq_off = 0;           // latent attention: float offset of the run's rotation frequencies in the table
-    size_t conv_off = 0;           // state-space: float offset of the convolution's last inputs inside a slot
+    size_t conv_off = 0;           // state-space, gated delta: float offset of the convolution's last inputs inside a slot
+    size_t unit_off = 0, m_off = 0;   // mLSTM: float offsets of the key sums and the running maxima inside a slot
     int flags = 0;                 // SMOL_LM_RUN_*
 };
 
@@ -1558,10 +1675,19 @@ struct SmolLm {
     }
 };
 
+constexpr int kAttnSplitSmemMax = 200 * 1024;      // shared memory the few-token attention may ask for
+
 static size_t al256(size_t v) { return (v + 255) / 256 * 256; }
 
+// softmax attention: score maps per head, and the rows of q, k and v in the input projection
+static int maps_of(const SmolLmLayer& L) { return L.n_maps > 1 ? L.n_maps : 1; }
+static int attn_qkv_rows(const SmolLmLayer& L) {
+    return L.heads * maps_of(L) * L.dim + (L.kv_from > 0 ? 0 : L.kv_heads * (maps_of(L) * L.dim + L.vdim));
+}
 static int n_in_of(const SmolLmLayer& L) {
-    if (L.mixer == SMOL_LM_MIX_SINK_ATTENTION) return L.heads * L.dim + L.kv_heads * L.dim + L.kv_heads * L.vdim + (L.no_gate ? 0 : L.heads * L.vdim);
+    if (L.mixer == SMOL_LM_MIX_SINK_ATTENTION) return attn_qkv_rows(L) + (L.no_gate ? 0 : L.heads * L.vdim);
+    if (L.mixer == SMOL_LM_MIX_GATED_DELTA) return 2 * L.kv_heads * L.dim + 2 * L.heads * L.vdim + 2 * L.heads;
+    if (L.mixer == SMOL_LM_MIX_MLSTM) return 2 * L.heads * L.dim + 2 * L.heads * L.vdim + 2 * L.heads;
     if (L.mixer == SMOL_LM_MIX_STATE_SPACE) return 2 * L.heads * L.vdim + 2 * L.bc_groups * L.n_state + L.heads;
     if (L.mixer == SMOL_LM_MIX_LATENT_ATTENTION) return L.q_rank + L.kv_rank + L.rot_dim + L.heads;
     if (L.mixer == SMOL_LM_MIX_GATED_LINEAR) return 2 * L.heads * L.dim + 2 * L.heads * L.vdim + L.rank;
@@ -1575,7 +1701,7 @@ static int n_in_of(const SmolLmLayer& L) {
 static int mix_cols_of(const SmolLmLayer& L) { return L.mixer == SMOL_LM_MIX_GENERAL_DELTA ? L.heads * L.dim : L.heads * L.vdim; }
 static bool pairable(const SmolLmLayer& L) {
     return L.mixer == SMOL_LM_MIX_SINK_ATTENTION || L.mixer == SMOL_LM_MIX_STATE_SPACE || L.mixer == SMOL_LM_MIX_SIGMOID_ATTENTION ||
-           L.mixer == SMOL_LM_MIX_LIGHTNING || L.mixer == SMOL_LM_MIX_RETENTION;
+           L.mixer == SMOL_LM_MIX_LIGHTNING || L.mixer == SMOL_LM_MIX_RETENTION || L.mixer == SMOL_LM_MIX_GATED_DELTA || L.mixer == SMOL_LM_MIX_MLSTM;
 }
 // Parallel block: the rows of the fused input projection that serve the feed-forward (shared expert's gate and up, router, shared
 // gate), and the projection's whole height (a multiple of 8).
@@ -1583,8 +1709,14 @@ static int ff_rows_of(const SmolLmLayer& L) {
     return L.mlp == SMOL_LM_MLP_EXPERTS ? (L.ff_plain ? 1 : 2) * L.shared_ff + L.n_experts + L.n_identity + (L.shared_gate ? 1 : 0) : 0;
 }
 static int parallel_n_in_of(const SmolLmLayer& L) { return (n_in_of(L) + ff_rows_of(L) + 7) / 8 * 8; }
-// base^(-2i/dims) for the dims/2 rotated pairs of a latent or sigmoid attention, stretched band by band when L.rot_stretch
-// is set (see the header)
+// Height of a layer's fused input projection.
+static int full_n_in_of(const SmolLmLayer& L, int block) {
+    if (block == SMOL_LM_BLOCK_PARALLEL) return parallel_n_in_of(L);
+    const int n = n_in_of(L) + (L.side ? n_in_of(*L.side) : 0);
+    return block == SMOL_LM_BLOCK_OUTNORM ? (n + 7) / 8 * 8 : n;
+}
+// base^(-2i/dims) for the dims/2 rotated pairs of a rotating mixer, stretched band by band when L.rot_stretch is set,
+// interpolated along a ramp when L.rot_yarn is (see the header)
 static void push_frequencies(std::vector<float>& table, const SmolLmLayer& L, bool stretch) {
     const double two_pi = 6.283185307179586476925286766559;
     for (int i = 0; i < L.rot_dims / 2; ++i) {
@@ -1597,6 +1729,12 @@ static void push_frequencies(std::vector<float>& table, const SmolLmLayer& L, bo
                 const double b = (orig / wl - L.rot_low) / ((double)L.rot_high - L.rot_low);
                 f = (1.0 - b) * f / L.rot_stretch + b * f;
             }
+        }
+        if (L.rot_yarn > 0.0f) {
+            auto dim_of = [&](double turns) { return L.rot_dims * log(L.rot_original / (two_pi * turns)) / (2.0 * log((double)L.rot_base)); };
+            const double lo = std::max(floor(dim_of(L.rot_fast)), 0.0), hi = std::min(ceil(dim_of(L.rot_slow)), L.rot_dims - 1.0);
+            const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+            f = f / L.rot_yarn * ramp + f * (1.0 - ramp);
         }
         table.push_back((float)f);
     }
@@ -1632,16 +1770,67 @@ extern "C" int smol_lm_create(const SmolLmConfig* cfg, const SmolLmLayer* layers
         if (L.in_bias && !pairable(L)) return fail(SMOL_ERR_UNSUPPORTED, "in_bias: softmax attention and the state-space recurrence only");
         if (L.mixer == SMOL_LM_MIX_SINK_ATTENTION) {
             if (L.kv_heads < 1 || L.heads % L.kv_heads != 0 || L.vdim < 1) return fail(SMOL_ERR_INVALID, "attention: heads must be a multiple of kv_heads");
-            if (L.vdim > 32 * kAttnMaxV) return fail(SMOL_ERR_UNSUPPORTED, "attention: value size above 256");
+            if (L.vdim > 32 * kAttnMaxV) return fail(SMOL_ERR_UNSUPPORTED, "attention: value size above 512");
             if (L.window < 0 || L.softcap < 0.0f || L.q_temp_every < 0.0f) return fail(SMOL_ERR_INVALID, "attention: window, softcap and q_temp_every must not be negative");
             if (!L.q_norm != !L.k_norm || (L.norm_whole && !L.q_norm)) return fail(SMOL_ERR_INVALID, "attention: q_norm and k_norm come together, norm_whole needs them");
-            r.k_off = m->page_elems;
-            r.v_off = r.k_off + (size_t)L.kv_heads * cfg->page_size * L.dim;
-            m->page_elems = r.v_off + (size_t)L.kv_heads * cfg->page_size * L.vdim;
-            m->max_q = std::max(m->max_q, L.heads * L.dim);
-            m->max_heads = std::max(m->max_heads, L.heads);
+            const int maps = maps_of(L);
+            if (maps > 2 || (maps == 2 && (L.norm_whole || L.sink))) return fail(SMOL_ERR_UNSUPPORTED, "attention: at most two maps, norms per map and no sink with two");
+            if (L.rot_dims < 0 || L.rot_dims > L.dim || L.rot_dims % 2) return fail(SMOL_ERR_INVALID, "attention: rot_dims even and at most dim");
+            if (L.rot_dims > 0 && (!L.norm_whole || L.rot_dims > 2 * kMaxRotPairs)) return fail(SMOL_ERR_UNSUPPORTED, "attention: rotation needs norm_whole and at most 512 coordinates");
+            const size_t split_smem = ((size_t)std::min(L.heads / L.kv_heads * maps, 8) * (L.dim + 32) * 4 + 15) / 16 * 16 +
+                                      (size_t)32 * (maps * (L.dim + 16 / m->esize) + L.vdim + 16 / m->esize) * m->esize;
+            if (split_smem > (size_t)kAttnSplitSmemMax) return fail(SMOL_ERR_UNSUPPORTED, "attention: key and value sizes need more shared memory than an SM has");
+            if (L.kv_from > 0) {
+                // another layer's cache, as its latest run leaves it
+                const RunInfo* lender = nullptr;
+                for (const RunInfo& o : m->runs)
+                    if (o.layer == L.kv_from - 1) lender = &o;
+                if (!lender) return fail(SMOL_ERR_INVALID, "attention: kv_from must name an earlier layer");
+                const SmolLmLayer& O = m->layers[lender->layer];
+                if (O.mixer != L.mixer || O.kv_from > 0 || O.kv_heads != L.kv_heads || O.dim != L.dim || O.vdim != L.vdim || maps_of(O) != maps || L.norm_whole)
+                    return fail(SMOL_ERR_INVALID, "attention: kv_from must name an attention layer with own keys and values and the same sizes");
+                r.k_off = lender->k_off;
+                r.v_off = lender->v_off;
+            } else {
+                r.k_off = m->page_elems;
+                r.v_off = r.k_off + (size_t)L.kv_heads * maps * cfg->page_size * L.dim;
+                m->page_elems = r.v_off + (size_t)L.kv_heads * cfg->page_size * L.vdim;
+            }
+            r.freq_off = m->freq_table.size();
+            push_frequencies(m->freq_table, L, true);
+            m->max_q = std::max(m->max_q, L.heads * maps * L.dim);
+            m->max_heads = std::max(m->max_heads, L.heads * maps);
             m->max_vdim = std::max(m->max_vdim, L.vdim);
             m->max_mix = std::max(m->max_mix, L.heads * L.vdim);
+        } else if (L.mixer == SMOL_LM_MIX_GATED_DELTA) {
+            if (L.dim > 256 || L.conv_taps > kMaxTaps) return fail(SMOL_ERR_UNSUPPORTED, "gated delta rule: key size above 256 or more than 16 taps");
+            if (L.vdim < 1 || L.kv_heads < 1 || L.heads % L.kv_heads != 0 || L.conv_taps < 1 || !L.conv_w || !L.a_log || !L.dt_bias || !L.out_norm)
+                return fail(SMOL_ERR_INVALID, "gated delta rule: heads must be a multiple of kv_heads, vdim and taps positive, conv_w, a_log, dt_bias and out_norm set");
+            const int ch = 2 * L.kv_heads * L.dim + L.heads * L.vdim;
+            r.state_off = m->slot_floats;
+            m->slot_floats += (size_t)L.heads * L.dim * L.vdim;
+            r.conv_off = m->slot_floats;
+            m->slot_floats += (size_t)(L.conv_taps - 1) * ch;
+            m->slot_floats = (m->slot_floats + 3) / 4 * 4;
+            m->max_hd = std::max(m->max_hd, L.heads * L.vdim);
+            m->max_mix = std::max(m->max_mix, L.heads * L.vdim);
+            m->max_conv = std::max(m->max_conv, ch);
+            m->max_ssd_heads = std::max(m->max_ssd_heads, (2 * L.heads + L.kv_heads + 1) / 2);        // decay, step, k.q
+        } else if (L.mixer == SMOL_LM_MIX_MLSTM) {
+            if (L.dim > 256) return fail(SMOL_ERR_UNSUPPORTED, "recurrent mixer: key size above 256");
+            if (L.vdim < 1 || !(L.gate_cap > 0.0f) || !L.rate_bias || !L.decay_bias || !L.out_norm)
+                return fail(SMOL_ERR_INVALID, "mLSTM: vdim and gate_cap must be positive, rate_bias, decay_bias and out_norm set");
+            r.state_off = m->slot_floats;
+            m->slot_floats += (size_t)L.heads * L.dim * L.vdim;
+            r.unit_off = m->slot_floats;
+            m->slot_floats += (size_t)L.heads * L.dim;
+            r.m_off = m->slot_floats;
+            m->slot_floats += L.heads;
+            m->slot_floats = (m->slot_floats + 3) / 4 * 4;
+            m->max_hd = std::max(m->max_hd, L.heads * L.vdim);
+            m->max_mix = std::max(m->max_mix, L.heads * L.vdim);
+            m->max_conv = std::max(m->max_conv, 1);
+            m->max_ssd_heads = std::max(m->max_ssd_heads, 2 * L.heads);        // decay, write weight, floor, key sum . query
         } else if (L.mixer == SMOL_LM_MIX_STATE_SPACE) {
             if (L.vdim < 1 || L.n_state < 1 || L.bc_groups < 1 || L.heads % L.bc_groups != 0 || L.conv_taps < 1 || L.norm_parts < 1 ||
                 (L.heads * L.vdim) % L.norm_parts != 0)
@@ -1743,7 +1932,12 @@ extern "C" int smol_lm_create(const SmolLmConfig* cfg, const SmolLmLayer* layers
         if (r.flags & SMOL_LM_RUN_ADD_EMBED) m->any_restart = true;
         if (r.flags & SMOL_LM_RUN_MERGE_EMBED) m->any_merge = true;
         int rc = place(L, r);
-        const bool prenorm = cfg->block == SMOL_LM_BLOCK_PRENORM, parallel = cfg->block == SMOL_LM_BLOCK_PARALLEL;
+        const bool prenorm = cfg->block == SMOL_LM_BLOCK_PRENORM, parallel = cfg->block == SMOL_LM_BLOCK_PARALLEL, outnorm = cfg->block == SMOL_LM_BLOCK_OUTNORM;
+        if (rc == SMOL_OK && outnorm) {
+            if (!L.norm1 || (L.mlp != SMOL_LM_MLP_NONE && !L.norm2)) rc = fail(SMOL_ERR_INVALID, "output-norm block: norm weights");
+            else if ((L.mlp != SMOL_LM_MLP_NONE && L.mlp != SMOL_LM_MLP_GATED) || !pairable(L))
+                rc = fail(SMOL_ERR_UNSUPPORTED, "output-norm block: dense gated feed-forwards or none; no HGRN2, latent attention, gated linear or generalized delta mixers");
+        }
         if (rc == SMOL_OK && L.side) {
             if (!pairable(L) || !pairable(*L.side)) rc = fail(SMOL_ERR_UNSUPPORTED, "mixers side by side: softmax or sigmoid attention, the state-space recurrence, lightning attention");
             else if (cfg->block == SMOL_LM_BLOCK_POSTNORM || parallel) rc = fail(SMOL_ERR_UNSUPPORTED, "mixers side by side need the sandwich or the pre-norm block");
@@ -1765,7 +1959,7 @@ extern "C" int smol_lm_create(const SmolLmConfig* cfg, const SmolLmLayer* layers
         }
         if (rc == SMOL_OK && ((r.flags & SMOL_LM_RUN_ADD_EMBED) && !prenorm)) rc = fail(SMOL_ERR_UNSUPPORTED, "runs that add the embedding output need the pre-norm block");
         if (rc == SMOL_OK && ((r.flags & SMOL_LM_RUN_MERGE_EMBED) || L.shared_gate) && !parallel) rc = fail(SMOL_ERR_UNSUPPORTED, "merging runs and gated shared experts need the parallel block");
-        if (rc == SMOL_OK && !prenorm && !parallel && (L.shared_ff > 0 || L.proj_norm || L.mixer >= SMOL_LM_MIX_SIGMOID_ATTENTION ||
+        if (rc == SMOL_OK && !prenorm && !parallel && !outnorm && (L.shared_ff > 0 || L.proj_norm || L.mixer >= SMOL_LM_MIX_SIGMOID_ATTENTION ||
                                          (L.side && L.side->mixer >= SMOL_LM_MIX_SIGMOID_ATTENTION)))
             rc = fail(SMOL_ERR_UNSUPPORTED, "shared experts, proj_norm, sigmoid / lightning attention, HGRN2 and retention need the pre-norm or the parallel block");
         if (rc == SMOL_OK && L.shared_ff > 0 && (L.mlp != SMOL_LM_MLP_EXPERTS || (!parallel && (!L.w_shared_in || !L.w_shared_out)))) rc = fail(SMOL_ERR_INVALID, "shared expert: routed feed-forwards only, with both matrices");
@@ -1792,7 +1986,7 @@ extern "C" int smol_lm_create(const SmolLmConfig* cfg, const SmolLmLayer* layers
             if (L.shared_ff > 0 && !parallel) m->max_ff = std::max(m->max_ff, (L.ff_plain ? 1 : 2) * L.shared_ff);
             if (parallel) m->max_mix = std::max(m->max_mix, mix_cols_of(L) + L.shared_ff);
         }
-        m->max_in = std::max(m->max_in, parallel ? parallel_n_in_of(L) : n_in_of(L) + (L.side ? n_in_of(*L.side) : 0));
+        m->max_in = std::max(m->max_in, full_n_in_of(L, cfg->block));
         m->runs.push_back(r);
         m->side_runs.push_back(rs);
     }
@@ -1876,10 +2070,11 @@ template <int DK>
 static cudaError_t scan_attribute() {
     cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(2 * delta_buf_floats(DK) * sizeof(float)));
     if (e == cudaSuccess) e = cudaFuncSetAttribute(gla_scan_kernel<DK, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, std::max(kScanSpread, (int)(2 * gla_buf_floats(DK) * sizeof(float))));
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(gated_delta_scan_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, std::max(kScanSpread, (int)(2 * gated_delta_buf_floats(DK) * sizeof(float))));
     if (e == cudaSuccess) e = cudaFuncSetAttribute(gla_scan_kernel<DK, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, std::max(kScanSpread, (int)(2 * gla_buf_floats(DK) * sizeof(float))));
     return e;
 }
-static constexpr int flash_smem_bytes(int DK, int DV, bool vk) { return 2 * 64 * ((DK + 8) + (vk ? 0 : DV + 8)) * (int)sizeof(bf16); }
+static constexpr int flash_smem_bytes(int DK, int DV, bool vk, int maps = 1) { return 2 * 64 * (maps * (DK + 8) + (vk ? 0 : DV + 8)) * (int)sizeof(bf16); }
 
 template <int DK, int HPW>
 static cudaError_t sigmoid_flash_attributes() {
@@ -1895,8 +2090,8 @@ static cudaError_t set_kernel_attributes() {
     if (e == cudaSuccess) e = scan_attribute<64>();
     if (e == cudaSuccess) e = scan_attribute<128>();
     if (e == cudaSuccess) e = scan_attribute<256>();
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_split_kernel<T, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_split_kernel<T, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_split_kernel<T, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, kAttnSplitSmemMax);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_split_kernel<T, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, kAttnSplitSmemMax);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(sigmoid_attn_kernel<T, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(sigmoid_attn_kernel<T, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(sigmoid_split_kernel<T, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSigmoidSmemMax);
@@ -1907,9 +2102,17 @@ static cudaError_t set_kernel_attributes() {
     if (e == cudaSuccess) e = sigmoid_flash_attributes<128, 1>();
     if (e == cudaSuccess) e = sigmoid_flash_attributes<32, 2>();
     if (e == cudaSuccess) e = sigmoid_flash_attributes<64, 2>();
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_flash_kernel<128, 128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, flash_smem_bytes(128, 128, false));
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_flash_kernel<192, 128, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, flash_smem_bytes(192, 128, true));
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_flash_kernel<192, 192, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, flash_smem_bytes(192, 192, true));
+#define SMOL_FLASH_ATTR(DK, DV, VK, MAPS)                                                                                        \
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_flash_kernel<DK, DV, VK, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                                   flash_smem_bytes(DK, DV, VK, MAPS))
+    SMOL_FLASH_ATTR(128, 128, false, 1);
+    SMOL_FLASH_ATTR(64, 128, false, 1);
+    SMOL_FLASH_ATTR(192, 128, true, 1);
+    SMOL_FLASH_ATTR(192, 192, true, 1);
+    SMOL_FLASH_ATTR(64, 64, false, 2);
+    SMOL_FLASH_ATTR(64, 128, false, 2);
+    SMOL_FLASH_ATTR(128, 128, false, 2);
+#undef SMOL_FLASH_ATTR
     return e;
 }
 
@@ -2084,7 +2287,7 @@ static cudaError_t launch_scan(const DeltaArgs& A, int n_seqs, const float* dec,
 template <int DK>
 static cudaError_t launch_gla_scan(const GlaArgs& A, int n_seqs, const float* dec, float* pool, float* o_raw, cudaStream_t st, size_t min_smem) {
     constexpr int CB = gla_block_cols(DK), threads = CB * gla_lanes(DK);
-    const int groups = (A.dv + CB - 1) / CB;
+    const int groups = (A.dv + (A.unit_out ? 1 : 0) + CB - 1) / CB;
     const size_t smem = std::max(2 * gla_buf_floats(DK) * sizeof(float), min_smem);
     if (A.head_decay) gla_scan_kernel<DK, true><<<n_seqs * A.H * groups, threads, smem, st>>>(A, dec, pool, o_raw);
     else gla_scan_kernel<DK, false><<<n_seqs * A.H * groups, threads, smem, st>>>(A, dec, pool, o_raw);
@@ -2100,9 +2303,17 @@ static cudaError_t launch_gla_scan_any(const GlaArgs& A, int n_seqs, const float
     return launch_gla_scan<256>(A, n_seqs, dec, pool, o_raw, st, min_smem);
 }
 
+template <int DK>
+static cudaError_t launch_gated_delta(const GatedDeltaArgs& A, int n_seqs, const float* qkv, const float* head, float* pool, float* o_raw, cudaStream_t st) {
+    constexpr int CB = gla_block_cols(DK), threads = CB * gla_lanes(DK);
+    const int groups = (A.dv + CB - 1) / CB;
+    gated_delta_scan_kernel<DK><<<n_seqs * A.H * groups, threads, 2 * gated_delta_buf_floats(DK) * sizeof(float), st>>>(A, qkv, head, pool, o_raw);
+    return cudaGetLastError();
+}
+
 // The attention kernels over the rows of a step: prompt portions on the tensor-core form (bf16, `flash`) or the
 // warp-per-row form, sequences of few tokens on the split-range form.  `A` is complete except for the fields set here.
-template <class T, int MAXV>
+template <class T, int MAXV, int MAPS>
 static void launch_attention(SmolLm* m, const SmolLmStep* s, AttnArgs& A, bool flash, const T* qbuf, const T* pool, T* mix, cudaStream_t st) {
     const SmolLmConfig& c = m->cfg;
     const int Tn = s->n_tokens;
@@ -2122,30 +2333,36 @@ static void launch_attention(SmolLm* m, const SmolLmStep* s, AttnArgs& A, bool f
             const bf16* qb = reinterpret_cast<const bf16*>(qbuf);
             const bf16* pl = reinterpret_cast<const bf16*>(pool);
             bf16* mx = reinterpret_cast<bf16*>(mix);
-#define SMOL_FLASH(DK, DV, VK) attn_flash_kernel<DK, DV, VK><<<grid, 128, flash_smem_bytes(DK, DV, VK), st>>>(A, qb, pl, mx)
-            if (A.v_in_k) {
-                if (A.d <= 64) SMOL_FLASH(64, 64, true);
+#define SMOL_FLASH(DK, DV, VK) attn_flash_kernel<DK, DV, VK, MAPS><<<grid, 128 * MAPS, flash_smem_bytes(DK, DV, VK, MAPS), st>>>(A, qb, pl, mx)
+            bool done = false;
+            if constexpr (MAPS == 1) {
+                done = A.v_in_k != 0;
+                if (!A.v_in_k) {
+                } else if (A.d <= 64) SMOL_FLASH(64, 64, true);
                 else if (A.d <= 128) SMOL_FLASH(128, 128, true);
                 else if (A.dv <= 128) SMOL_FLASH(192, 128, true);
                 else SMOL_FLASH(192, 192, true);
+            }
+            if (done) {
             } else if (hp <= 32) SMOL_FLASH(32, 32, false);
             else if (hp <= 64) SMOL_FLASH(64, 64, false);
+            else if (A.d <= 64) SMOL_FLASH(64, 128, false);
             else SMOL_FLASH(128, 128, false);
 #undef SMOL_FLASH
         } else {
             // every row, also those of short sequences
             const int au = Tn * A.H;
-            attn_kernel<T, MAXV><<<(au + kAttnWarps - 1) / kAttnWarps, kAttnWarps * 32, kAttnWarps * A.d * sizeof(float), st>>>(A, qbuf, pool, mix);
+            attn_kernel<T, MAXV, MAPS><<<(au + kAttnWarps - 1) / kAttnWarps, kAttnWarps * 32, kAttnWarps * A.d * sizeof(float), st>>>(A, qbuf, pool, mix);
         }
         m->launches += 1;
     }
     if (min_n <= kShortSeq && (flash || max_n <= kShortSeq)) {
-        const int Gq = A.H / A.G, nwarp = std::min(Gq, 8), groups = (Gq + nwarp - 1) / nwarp;
+        const int Gq = A.H / A.G * MAPS, nwarp = std::min(Gq, 8), groups = (Gq + nwarp - 1) / nwarp;
         const int pad = 16 / (int)sizeof(T);
-        const size_t smem = ((size_t)nwarp * (A.d + 32) * 4 + 15) / 16 * 16 + (size_t)32 * (A.d + pad + (A.v_in_k ? 0 : A.dv + pad)) * sizeof(T);
+        const size_t smem = ((size_t)nwarp * (A.d + 32) * 4 + 15) / 16 * 16 + (size_t)32 * (MAPS * (A.d + pad) + (A.v_in_k ? 0 : A.dv + pad)) * sizeof(T);
         dim3 grid(A.short_rows, A.G * groups, A.n_splits);
         attn_split_kernel<T, MAXV><<<grid, nwarp * 32, smem, st>>>(A, qbuf, pool);
-        attn_merge_kernel<T, MAXV><<<(A.short_rows * A.H + 3) / 4, 128, 0, st>>>(A, mix);
+        attn_merge_kernel<T, MAXV, MAPS><<<(A.short_rows * A.H + 3) / 4, 128, 0, st>>>(A, mix);
         m->launches += 2;
     }
 }
@@ -2212,7 +2429,7 @@ template <class T>
 static void launch_residual_norm(const ResidualArgs& A, int rows, int threads, T* hn, cudaStream_t st) {
     uintptr_t at = 0;
     for (const void* p : {(const void*)A.x, (const void*)A.y, (const void*)A.y2, (const void*)A.y_w, (const void*)A.y2_w, (const void*)A.rs.yp, (const void*)A.trace,
-                          (const void*)A.x0, (const void*)A.cat, (const void*)A.next.w, (const void*)A.next.shift, (const void*)hn})
+                          (const void*)A.x0, (const void*)A.cat, (const void*)A.y_b, (const void*)A.next.w, (const void*)A.next.shift, (const void*)hn})
         at |= reinterpret_cast<uintptr_t>(p);
     if (A.D % 4 == 0 && at % 16 == 0) residual_norm_kernel<T, true><<<rows, threads, A.D * sizeof(float), st>>>(A, hn);
     else residual_norm_kernel<T, false><<<rows, threads, A.D * sizeof(float), st>>>(A, hn);
@@ -2240,13 +2457,13 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
     T* pool = static_cast<T*>(m->pages);
     const int nthr = D >= 1024 ? 256 : 128;
     const bool postnorm = c.block == SMOL_LM_BLOCK_POSTNORM, parallel = c.block == SMOL_LM_BLOCK_PARALLEL;
-    const bool prenorm = c.block == SMOL_LM_BLOCK_PRENORM;
+    const bool prenorm = c.block == SMOL_LM_BLOCK_PRENORM, outnorm = c.block == SMOL_LM_BLOCK_OUTNORM;
     float* x0 = m->any_restart ? reinterpret_cast<float*>(m->ws + m->o_x0) : nullptr;
     T* cat = m->any_merge ? reinterpret_cast<T*>(m->ws + m->o_cat) : nullptr;
     T* mix2 = reinterpret_cast<T*>(m->ws + m->o_mix2);
     float* y2 = reinterpret_cast<float*>(m->ws + m->o_y2);
     auto norm_of = [&](const float* w, const float* shift, const float* alpha) { return NormSpec{c.norm_kind, w, shift, alpha, c.norm_eps}; };
-    const NormSpec no_norm{c.norm_kind, nullptr, nullptr, nullptr, c.norm_eps};
+    const NormSpec no_norm{c.norm_kind, nullptr, nullptr, nullptr, c.norm_eps}, copy_row{kNormCopy, nullptr, nullptr, nullptr, c.norm_eps};
     const size_t hist_stride = (size_t)Tn * D;
     constexpr bool kIsF32 = sizeof(T) == 4;
     const float woff = c.norm_plain ? 0.0f : 1.0f;
@@ -2256,6 +2473,8 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
 
     if (postnorm) {
         embed_gain_norm_kernel<T><<<Tn, nthr, 0, st>>>(s->tokens, static_cast<const T*>(m->g.embed), D, c.vocab, m->g.embed_norm, c.norm_eps, x, hist, hn);
+    } else if (outnorm) {
+        embed_prenorm_kernel<T><<<Tn, nthr, 0, st>>>(s->tokens, static_cast<const T*>(m->g.embed), c.embed_scale, D, c.vocab, copy_row, x, nullptr, hn, nullptr);
     } else if (prenorm || parallel) {
         const SmolLmLayer& L0 = m->layers[m->runs[0].layer];
         const bool merge = m->runs[0].flags & SMOL_LM_RUN_MERGE_EMBED;
@@ -2269,7 +2488,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
     for (size_t n = 0; n < m->runs.size(); ++n) {
         const RunInfo& R = m->runs[n];
         const SmolLmLayer& L = m->layers[R.layer];
-        const int n_in_main = n_in_of(L), n_in = parallel ? parallel_n_in_of(L) : n_in_main + (L.side ? n_in_of(*L.side) : 0);
+        const int n_in_main = n_in_of(L), n_in = full_n_in_of(L, c.block);
         if (R.flags & SMOL_LM_RUN_MERGE_EMBED) {
             // the stream starts anew from the merged rows, which the previous run's last kernel (or the embedding) has left in cat
             CU(linear<T>(m, cat, static_cast<const T*>(m->g.w_merge), x, Tn, D, 2 * D, st));
@@ -2293,22 +2512,30 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             A.n_tokens = Tn; A.err = err;
             A.G = M.kv_heads; A.d = M.dim; A.dv = M.vdim;
             A.k_ld = M.dim; A.v_ld = M.vdim; A.v_in_k = 0;
-            A.gate_off = (size_t)M.heads * M.dim + (size_t)M.kv_heads * (M.dim + M.vdim); A.gate_ld = M.vdim; A.gate_step = 1;
+            A.gate_off = (size_t)attn_qkv_rows(M); A.gate_ld = M.vdim; A.gate_step = 1;
             A.has_gate = M.no_gate ? 0 : 1;
             A.q_norm = M.q_norm; A.k_norm = M.k_norm; A.r1 = M.dist_r1; A.r2 = M.dist_r2; A.sink = M.sink;
             A.slope = M.dist_slope; A.window = M.window; A.softcap = M.softcap; A.two_over_cap = M.softcap > 0.0f ? 2.0f / M.softcap : 0.0f;
             A.out_ld = out_ld_now; A.out_scale = M.mix_scale;
             A.temp_coef = M.q_temp_coef; A.temp_every = M.q_temp_every;
+            A.maps = maps_of(M); A.diff_lambda = M.diff_lambda; A.diff_scale = M.diff_scale; A.own_kv = M.kv_from == 0;
             if (M.norm_whole) {
-                attn_prep_whole_kernel<T><<<Tn, Tn > 64 ? 128 : 256, 0, st>>>(A, qbuf, pool);      // few tokens: more loads in flight per token
+                const int threads = Tn > 64 ? 128 : 256;      // few tokens: more loads in flight per token
+                A.rot_pairs = M.rot_dims / 2; A.rot_half = M.rot_half; A.rot_mult = M.rot_mult != 0.0f ? M.rot_mult : 1.0f;
+                A.freq = reinterpret_cast<const float*>(m->ws + m->o_freq) + Ri.freq_off;
+                if (A.rot_pairs > 0) attn_prep_whole_kernel<T, true><<<Tn, threads, 0, st>>>(A, qbuf, pool);
+                else attn_prep_whole_kernel<T, false><<<Tn, threads, 0, st>>>(A, qbuf, pool);
             } else {
-                const int units = Tn * (M.heads + 2 * M.kv_heads);
+                const int units = Tn * (M.heads * A.maps + (A.own_kv ? M.kv_heads * (A.maps + 1) : 0));
                 attn_prep_kernel<T><<<(units + 3) / 4, 128, 0, st>>>(A, qbuf, pool);
             }
             m->launches += 1;
             const bool flash = sizeof(T) == 2 && std::max(M.dim, M.vdim) <= 128;
-            if (M.vdim <= 256) launch_attention<T, 8>(m, s, A, flash, qbuf, pool, mix_at, st);
-            else launch_attention<T, 16>(m, s, A, flash, qbuf, pool, mix_at, st);
+            if (A.maps == 2) {
+                if (M.vdim <= 256) launch_attention<T, 8, 2>(m, s, A, flash, qbuf, pool, mix_at, st);
+                else launch_attention<T, 16, 2>(m, s, A, flash, qbuf, pool, mix_at, st);
+            } else if (M.vdim <= 256) launch_attention<T, 8, 1>(m, s, A, flash, qbuf, pool, mix_at, st);
+            else launch_attention<T, 16, 1>(m, s, A, flash, qbuf, pool, mix_at, st);
             return SMOL_OK;
         };
         // State-space recurrence: convolution and per-head step / decay, the scan over the slot's state, then skip, gate and the
@@ -2438,12 +2665,60 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             m->launches += 3;
             return SMOL_OK;
         };
+        // Gated delta rule: convolutions, unit vectors, decay and step; the scan over the slot's state; norm per head, silu gate.
+        auto gated_delta = [&](const SmolLmLayer& M, const RunInfo& Ri, const float* pj, T* mix_at, int ld) -> int {
+            const int hv = M.heads * M.vdim, ch = 2 * M.kv_heads * M.dim + hv;
+            GatedDeltaArgs P;
+            P.proj = pj; P.n_in = n_in; P.H = M.heads; P.G = M.kv_heads; P.d = M.dim; P.dv = M.vdim; P.n_tokens = Tn;
+            P.q_scale = M.score_scale; P.unit_eps = M.unit_eps; P.a_log = M.a_log; P.dt_bias = M.dt_bias;
+            P.tok_seq = s->tok_seq; P.state_off = Ri.state_off; P.err = err;
+            P.conv = ConvIo{pj, nullptr, n_in, ch, M.conv_taps, M.conv_w, nullptr, s->seq_start, s->seq_pos0, s->seq_slot, m->slot_floats, Ri.conv_off, m->n_slots};
+            const int warps = M.kv_heads + (hv + kGatedDeltaCols - 1) / kGatedDeltaCols;
+            gated_delta_prep_kernel<<<dim3(Tn, (warps + 3) / 4), 128, 0, st>>>(P, m->slots, conv, head);
+            if (M.dim <= 16) CU(launch_gated_delta<16>(P, s->n_seqs, conv, head, m->slots, oraw, st));
+            else if (M.dim <= 32) CU(launch_gated_delta<32>(P, s->n_seqs, conv, head, m->slots, oraw, st));
+            else if (M.dim <= 64) CU(launch_gated_delta<64>(P, s->n_seqs, conv, head, m->slots, oraw, st));
+            else if (M.dim <= 128) CU(launch_gated_delta<128>(P, s->n_seqs, conv, head, m->slots, oraw, st));
+            else CU(launch_gated_delta<256>(P, s->n_seqs, conv, head, m->slots, oraw, st));
+            GlaArgs A = scan_args(M, Ri, pj);
+            A.out_norm = M.out_norm; A.gate_off = ch; A.out_ld = ld; A.out_scale = M.mix_scale;
+            gla_out_kernel<T><<<(Tn * M.heads + 3) / 4, 128, 0, st>>>(A, oraw, mix_at);
+            m->launches += 3;
+            return SMOL_OK;
+        };
+        // mLSTM: gates and running maximum, the scan with the unit column (the key sum's product with the query), then the
+        // denominator, norm per head and sigmoid gate.
+        auto mlstm = [&](const SmolLmLayer& M, const RunInfo& Ri, const float* pj, T* mix_at, int ld) -> int {
+            const int hd = M.heads * M.dim, hv = M.heads * M.vdim;
+            const size_t TH = (size_t)Tn * M.heads;
+            MlstmArgs P;
+            P.proj = pj; P.n_in = n_in; P.H = M.heads; P.n_tokens = Tn; P.gate_off = (size_t)2 * hd + 2 * hv; P.cap = M.gate_cap;
+            P.i_bias = M.rate_bias; P.f_bias = M.decay_bias;
+            P.seq_start = s->seq_start; P.seq_pos0 = s->seq_pos0; P.seq_slot = s->seq_slot;
+            P.slot_floats = m->slot_floats; P.m_off = Ri.m_off; P.n_slots = m->n_slots; P.err = err;
+            const int max_n = s->max_seq_tokens > 0 ? s->max_seq_tokens : Tn;
+            mlstm_gate_kernel<<<s->n_seqs * M.heads, std::min(kMlstmTile, (max_n + 31) / 32 * 32), 0, st>>>(P, m->slots, head);
+            GlaArgs A = scan_args(M, Ri, pj);
+            A.q_src = pj; A.k_src = pj + hd; A.v_src = pj + 2 * hd;
+            A.q_ld = A.k_ld = A.v_ld = n_in;
+            A.q_scale = M.score_scale;
+            A.head_decay = head; A.head_step = head + TH;
+            A.unit_out = head + 3 * TH; A.unit_off = Ri.unit_off;
+            CU(launch_gla_scan_any(A, s->n_seqs, nullptr, m->slots, oraw, st));
+            A.unit_floor = head + 2 * TH; A.den_eps = M.den_eps;
+            A.out_norm = M.out_norm; A.norm_own = 1; A.gate_sigmoid = 1; A.out_ld = ld; A.out_scale = M.mix_scale;
+            gla_out_kernel<T><<<(Tn * M.heads + 3) / 4, 128, 0, st>>>(A, oraw, mix_at);
+            m->launches += 3;
+            return SMOL_OK;
+        };
         auto run_mixer = [&](const SmolLmLayer& M, const RunInfo& Ri, const float* pj, const float* bias, T* mix_at, int ld) -> int {
             out_ld_now = ld;
             if (M.mixer == SMOL_LM_MIX_SINK_ATTENTION) return attention(M, Ri, pj, bias, mix_at);
             if (M.mixer == SMOL_LM_MIX_STATE_SPACE) return state_space(M, Ri, pj, bias, mix_at);
             if (M.mixer == SMOL_LM_MIX_SIGMOID_ATTENTION) return sigmoid_attention(M, Ri, pj, bias, mix_at, ld);
             if (M.mixer == SMOL_LM_MIX_RETENTION) return retention(M, Ri, pj, mix_at, ld);
+            if (M.mixer == SMOL_LM_MIX_GATED_DELTA) return gated_delta(M, Ri, pj, mix_at, ld);
+            if (M.mixer == SMOL_LM_MIX_MLSTM) return mlstm(M, Ri, pj, mix_at, ld);
             return lightning(M, Ri, pj, mix_at, ld);
         };
         // the feed-forward reads hn and leaves its output in y, routed experts theirs in `routed` for the kernel that follows
@@ -2642,8 +2917,8 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
                 A.gate_off = (size_t)L.q_rank + dk; A.gate_ld = 1; A.gate_step = 0;
                 A.q_norm = A.k_norm = A.r1 = A.r2 = A.sink = nullptr;
                 const bool flash = sizeof(T) == 2 && dk <= 192;          // larger latents take the warp-per-row form for prompt portions
-                if (L.kv_rank <= 256) launch_attention<T, 8>(m, s, A, flash, qbuf, pool, mix, st);
-                else launch_attention<T, 16>(m, s, A, flash, qbuf, pool, mix, st);
+                if (L.kv_rank <= 256) launch_attention<T, 8, 1>(m, s, A, flash, qbuf, pool, mix, st);
+                else launch_attention<T, 16, 1>(m, s, A, flash, qbuf, pool, mix, st);
                 // per head: the attended latent [Tn, kv_rank] times the value expansion [vdim, kv_rank]^T
                 GemmIo iv = plain_io(L.kv_rank, L.vdim);
                 iv.lda = L.heads * L.kv_rank; iv.ldy = L.heads * L.vdim;
@@ -2704,6 +2979,27 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             Ra.next = (Ln && !merge) ? norm_of(Ln->norm1, Ln->norm1_shift, Ln->norm1_alpha) : no_norm;
             launch_residual_norm<T>(Ra, Tn, nthr, hn, st);
             m->launches += 1;
+        } else if (outnorm) {
+            // x += r(mixer + bias) * norm1, x += r(feed-forward) * norm2; each kernel leaves the new stream in T for the next sublayer
+            const bool has_ff = L.mlp != SMOL_LM_MLP_NONE;
+            float* tr_row = s->trace ? s->trace + n * (size_t)Tn * D : nullptr;
+            ResidualArgs Ra;
+            Ra.x = x; Ra.D = D; Ra.eps = c.norm_eps;
+            Ra.y = y; Ra.y_w = L.norm1; Ra.y_b = L.out_bias; Ra.sy = 1.0f;
+            Ra.y2 = Ra.y2_w = nullptr; Ra.sy2 = 0.0f;
+            Ra.rs = no_sum; Ra.s_routed = 1.0f; Ra.x0 = nullptr; Ra.cat = nullptr;
+            Ra.trace = has_ff ? nullptr : tr_row;
+            Ra.next = has_ff || !last ? copy_row : no_norm;
+            launch_residual_norm<T>(Ra, Tn, nthr, hn, st);
+            m->launches += 1;
+            if (has_ff) {
+                const int rc = feed_forward(st);
+                if (rc != SMOL_OK) return rc;
+                Ra.y_w = L.norm2; Ra.y_b = nullptr; Ra.trace = tr_row;
+                Ra.next = last ? no_norm : copy_row;
+                launch_residual_norm<T>(Ra, Tn, nthr, hn, st);
+                m->launches += 1;
+            }
         } else if (prenorm) {
             // x += mixer (mixers with their own projections: each normed over the width first); x += feed-forward.  The kernel
             // that ends the layer also leaves the traced row, restarts the stream where the next run asks for it and applies
@@ -2757,12 +3053,12 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             add_norm_kernel<T><<<Tn, nthr, D * sizeof(float), st>>>(x, y, L.norm1b, L.ls1, next_norm1, c.norm_eps, D, hn, woff, L.out_bias, no_sum, hn);
             m->launches += 1;
         }
-        if (s->trace && !prenorm && !parallel) CU(cudaMemcpyAsync(s->trace + n * (size_t)Tn * D, x, (size_t)Tn * D * 4, cudaMemcpyDeviceToDevice, st));
+        if (s->trace && !prenorm && !parallel && !outnorm) CU(cudaMemcpyAsync(s->trace + n * (size_t)Tn * D, x, (size_t)Tn * D * 4, cudaMemcpyDeviceToDevice, st));
     }
     if (s->n_want > 0) {
         if (postnorm) post_norm_kernel<T><<<s->n_want, nthr, 2 * D * sizeof(float), st>>>(x, nullptr, c.logit_scale, m->g.final_norm, c.norm_eps, D, nullptr, 0, 0,
                                                                                       nullptr, s->want_rows, hw, RoutedSum{nullptr, nullptr, nullptr, 0});
-        else if (prenorm || parallel) prenorm_rows_kernel<T><<<s->n_want, nthr, 0, st>>>(x, s->want_rows, norm_of(m->g.final_norm, m->g.final_norm_shift, m->g.final_norm_alpha), D, hw);
+        else if (prenorm || parallel || outnorm) prenorm_rows_kernel<T><<<s->n_want, nthr, 0, st>>>(x, s->want_rows, norm_of(m->g.final_norm, m->g.final_norm_shift, m->g.final_norm_alpha), D, hw);
         else norm_rows_kernel<T><<<s->n_want, nthr, 0, st>>>(x, s->want_rows, m->g.final_norm, c.norm_eps, D, hw, woff);
         m->launches++;
         CU(linear<T>(m, hw, static_cast<const T*>(m->g.head), s->logits, s->n_want, c.vocab, D, st));

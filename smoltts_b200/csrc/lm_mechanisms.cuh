@@ -323,6 +323,16 @@ struct GlaArgs {
     int head_ld;
     int out_ld;                                        // row stride of the finished mixer output
     float out_scale;
+    // A further state column per head whose value is 1 for every token (the running sum of the written keys): its rows live at
+    // unit_off inside the slot ([H][d]), its product with the query goes to unit_out[t * H + h].  nullptr: none.
+    float* unit_out = nullptr;
+    size_t unit_off = 0;
+    // Back end: where the gate rows start in proj (negative: behind q, k and v), sigmoid or silu, the norm weight shared by the heads
+    // ([dv]) or their own ([H * dv]); with unit_out the head's o is first divided by max(|unit_out|, unit_floor[t * H + h]) + den_eps.
+    long long gate_off = -1;
+    int gate_sigmoid = 0, norm_own = 0;
+    const float* unit_floor = nullptr;
+    float den_eps = 0.0f;
 };
 __host__ __device__ inline void gla_sources_from_proj(GlaArgs& A) {
     A.q_src = A.proj; A.k_src = A.proj + A.H * A.d; A.v_src = A.proj + 2 * A.H * A.d;
@@ -397,11 +407,11 @@ __global__ void __launch_bounds__(gla_block_cols(DK) * gla_lanes(DK)) gla_scan_k
     constexpr int kBuf = gla_buf_floats(DK);
     static_assert(DK % (4 * L) == 0, "every lane owns whole 16-byte pieces");
     extern __shared__ __align__(16) float sh[];
-    const int d = A.d, dv = A.dv, NS = (dv + CB - 1) / CB;
+    const int d = A.d, dv = A.dv, dvs = dv + (SCALAR && A.unit_out ? 1 : 0), NS = (dvs + CB - 1) / CB;      // dvs: state columns
     const int group = blockIdx.x % NS, sh_id = blockIdx.x / NS;
     const int seq = sh_id / A.H, h = sh_id % A.H;
     const int j0 = group * CB;
-    const int nc = min(CB, dv - j0);
+    const int nc = max(0, min(CB, dv - j0));
     const int col = threadIdx.x / L, q = threadIdx.x % L, j = j0 + col;
     const int t0 = A.seq_start[seq], t1 = A.seq_start[seq + 1];
     const int slot = A.seq_slot[seq];
@@ -413,11 +423,18 @@ __global__ void __launch_bounds__(gla_block_cols(DK) * gla_lanes(DK)) gla_scan_k
     const bool vec = (d % 4 == 0) && (dv % 4 == 0) && (A.q_ld % 4 == 0) && (A.k_ld % 4 == 0) && (A.v_ld % 4 == 0) &&
                      ((reinterpret_cast<uintptr_t>(A.q_src) | reinterpret_cast<uintptr_t>(A.k_src) | reinterpret_cast<uintptr_t>(A.v_src)) % 16 == 0);
     for (int i = threadIdx.x; i < 2 * kBuf; i += blockDim.x) sh[i] = 0.0f;      // padded channels and columns stay zero for good
+    if (SCALAR && dvs > dv && dv >= j0 && dv < j0 + CB) {                      // ... and the unit column one
+        __syncthreads();
+        for (int i = threadIdx.x; i < 2 * kDeltaChunk; i += blockDim.x) sh[(i / kDeltaChunk) * kBuf + 3 * PL + (i % kDeltaChunk) * CB + dv - j0] = 1.0f;
+    }
     __syncthreads();
     if (vec) gla_stage<DK, 4, SCALAR>(A, sh, t0, min(kDeltaChunk, t1 - t0), h, j0, nc, decay);
     else gla_stage<DK, 1, SCALAR>(A, sh, t0, min(kDeltaChunk, t1 - t0), h, j0, nc, decay);
     cp_async_commit();
-    float* st = state_pool + (size_t)slot * A.slot_floats + A.state_off + (size_t)h * d * dv;
+    // element i of this thread's column: st[i * st_ld]
+    const bool unit = SCALAR && j == dv && dvs > dv;
+    float* st = state_pool + (size_t)slot * A.slot_floats + (unit ? A.unit_off + (size_t)h * d : A.state_off + (size_t)h * d * dv + j);
+    const int st_ld = unit ? 1 : dv;
     float S[RV][4];
     const bool fresh = A.seq_pos0[seq] == 0;
 #pragma unroll
@@ -425,7 +442,7 @@ __global__ void __launch_bounds__(gla_block_cols(DK) * gla_lanes(DK)) gla_scan_k
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
             const int i = 4 * (e * L + q) + x;
-            S[e][x] = (!fresh && i < d && j < dv) ? st[(size_t)i * dv + j] : 0.0f;
+            S[e][x] = (!fresh && i < d && j < dvs) ? st[(size_t)i * st_ld] : 0.0f;
         }
     int cur = 0;
     for (int c0 = t0; c0 < t1; c0 += kDeltaChunk, cur ^= 1) {
@@ -474,10 +491,12 @@ __global__ void __launch_bounds__(gla_block_cols(DK) * gla_lanes(DK)) gla_scan_k
             for (int s = 1; s < L; s <<= 1)
 #pragma unroll
                 for (int u = 0; u < 4; ++u) po[u] += __shfl_xor_sync(0xffffffffu, po[u], s);
-            if (q == 0 && j < dv) {
+            if (q == 0 && j < dvs) {
+                float* dst = unit ? A.unit_out + (size_t)(c0 + tt) * A.H + h : o_raw + (size_t)(c0 + tt) * A.H * dv + h * dv + j;
+                const int ld = unit ? A.H : A.H * dv;
 #pragma unroll
                 for (int u = 0; u < 4; ++u)
-                    if (FULL || tt + u < n) o_raw[(size_t)(c0 + tt + u) * A.H * dv + h * dv + j] = po[u] * A.q_scale;
+                    if (FULL || tt + u < n) dst[(size_t)u * ld] = po[u] * A.q_scale;
             }
         };
         if (n == kDeltaChunk) {
@@ -493,12 +512,13 @@ __global__ void __launch_bounds__(gla_block_cols(DK) * gla_lanes(DK)) gla_scan_k
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
             const int i = 4 * (e * L + q) + x;
-            if (i < d && j < dv) st[(size_t)i * dv + j] = S[e][x];
+            if (i < d && j < dvs) st[(size_t)i * st_ld] = S[e][x];
         }
 }
 
-// End of the mixer: each head's o divided by its root mean square over dv, times the plain weight [dv] (shared by the
-// heads; nullptr: none), times silu(gate), written in T.  One warp per (token, head).
+// End of the mixer: each head's o (divided by its unit column's product first, where there is one) divided by its root mean square
+// over dv, times the plain weight (shared by the heads or their own; nullptr: none), times silu or sigmoid of the gate, written in
+// T.  One warp per (token, head).
 template <class T>
 __global__ void gla_out_kernel(const GlaArgs A, const float* __restrict__ o_raw, T* __restrict__ out) {
     const int lane = threadIdx.x & 31;
@@ -506,19 +526,100 @@ __global__ void gla_out_kernel(const GlaArgs A, const float* __restrict__ o_raw,
     if (unit >= A.n_tokens * A.H) return;
     const int t = unit / A.H, h = unit % A.H, dv = A.dv, HV = A.H * dv;
     const float* o = o_raw + (size_t)t * HV + h * dv;
-    const float* gate = A.proj + (size_t)t * A.n_in + 2 * A.H * A.d + HV + h * dv;
+    const float* gate = A.proj + (size_t)t * A.n_in + (A.gate_off >= 0 ? (size_t)A.gate_off : (size_t)2 * A.H * A.d + HV) + h * dv;
+    const float* weight = A.out_norm ? A.out_norm + (A.norm_own ? h * dv : 0) : nullptr;
+    float inv = 1.0f;
+    if (A.unit_out) inv = 1.0f / (fmaxf(fabsf(A.unit_out[(size_t)t * A.H + h]), A.unit_floor[(size_t)t * A.H + h]) + A.den_eps);
+    auto finish = [&](float v, float rs, float w, float g) { return from_f<T>(v * rs * w * (A.gate_sigmoid ? sigmoidf_(g) : silu_(g)) * A.out_scale); };
+    constexpr int R = 4;                 // up to 128 columns in registers: every load goes out before the reduction
+    if (dv <= 32 * R) {
+        float v[R], w[R], g[R];
+        float ss = 0.0f;
+#pragma unroll
+        for (int e = 0; e < R; ++e) {
+            const int c = lane + 32 * e;
+            const bool in = c < dv;
+            v[e] = in ? o[c] : 0.0f;
+            w[e] = in && weight ? weight[c] : 1.0f;
+            g[e] = in ? gate[c] : 0.0f;
+        }
+#pragma unroll
+        for (int e = 0; e < R; ++e) {
+            v[e] *= inv;
+            ss = fmaf(v[e], v[e], ss);
+        }
+        ss = warp_sum(ss);
+        const float rs = 1.0f / sqrtf(ss / (float)dv + A.eps);
+#pragma unroll
+        for (int e = 0; e < R; ++e) {
+            const int c = lane + 32 * e;
+            if (c < dv) out[(size_t)t * A.out_ld + h * dv + c] = finish(v[e], rs, w[e], g[e]);
+        }
+        return;
+    }
     float ss = 0.0f;
-    for (int c = lane; c < dv; c += 32) ss = fmaf(o[c], o[c], ss);
+    for (int c = lane; c < dv; c += 32) { const float v = o[c] * inv; ss = fmaf(v, v, ss); }
     ss = warp_sum(ss);
     const float rs = 1.0f / sqrtf(ss / (float)dv + A.eps);
-    for (int c = lane; c < dv; c += 32) out[(size_t)t * A.out_ld + h * dv + c] = from_f<T>(o[c] * rs * (A.out_norm ? A.out_norm[c] : 1.0f) * silu_(gate[c]) * A.out_scale);
+    for (int c = lane; c < dv; c += 32) out[(size_t)t * A.out_ld + h * dv + c] = finish(o[c] * inv, rs, weight ? weight[c] : 1.0f, gate[c]);
+}
+
+// ---------------------------------------------------------------------------------------------------------------------
+// Short causal convolution over a sequence's positions: channel c of a token is silu(b[c] + sum_k w[c][k] * input at k - (taps - 1)
+// positions from it), zeros before position 0; the inputs are columns of the fused projection.  The last taps - 1 inputs live
+// in the sequence's slot.
+constexpr int kMaxTaps = 16;
+struct ConvIo {
+    const float* src;         // first channel of row 0; row stride ld
+    const float* bias;        // of the projection's rows, or nullptr
+    int ld, ch, taps;
+    const float *w, *b;       // [ch][taps], [ch] (nullptr: none)
+    const int32_t *seq_start, *seq_pos0, *seq_slot;
+    size_t slot_floats, conv_off;      // float offset of this run's inputs inside a slot: [taps - 1][ch]
+    int n_slots;
+};
+// channel c of token t, the r-th of its sequence's portion; before: the slot's inputs of positions pos0 - (taps - 1) .. pos0 - 1
+__device__ __forceinline__ float conv_channel(const ConvIo& C, const float* __restrict__ before, int t, int r, int pos0, int c) {
+    float acc = C.b ? C.b[c] : 0.0f;
+    const float bc = C.bias ? C.bias[c] : 0.0f;
+#pragma unroll 4
+    for (int k = 0; k < C.taps; ++k) {
+        const int back = C.taps - 1 - k;       // how many positions before the token
+        float v = 0.0f;
+        if (back <= r) v = C.src[(size_t)(t - back) * C.ld + c] + bc;
+        else if (pos0 + r - back >= 0) v = before[(size_t)(C.taps - 1 - (back - r)) * C.ch + c];
+        acc = fmaf(C.w[(size_t)c * C.taps + k], v, acc);
+    }
+    return silu_(acc);
+}
+// After a step the slot keeps the last taps - 1 inputs of every sequence: channel c of sequence s.  A thread reads all it needs
+// of the old inputs before it writes; every reader of the old inputs has to be done.
+__device__ __forceinline__ void conv_state_update(const ConvIo& C, float* __restrict__ slots, int s, int c) {
+    const int keep = C.taps - 1;
+    const int t0 = C.seq_start[s], n = C.seq_start[s + 1] - t0, pos0 = C.seq_pos0[s];
+    const int slot = C.seq_slot[s];
+    if (slot < 0 || slot >= C.n_slots) return;
+    float* st = slots + (size_t)slot * C.slot_floats + C.conv_off;
+    const float bc = C.bias ? C.bias[c] : 0.0f;
+    float nv[kMaxTaps];
+#pragma unroll
+    for (int k = 0; k < kMaxTaps; ++k) {
+        if (k >= keep) break;
+        const int back = keep - k;                 // new entry k is the input `back` positions before the next token
+        if (back <= n) nv[k] = C.src[(size_t)(t0 + n - back) * C.ld + c] + bc;
+        else nv[k] = (pos0 + n - back >= 0) ? st[(size_t)(keep - (back - n)) * C.ch + c] : 0.0f;
+    }
+#pragma unroll
+    for (int k = 0; k < kMaxTaps; ++k) {
+        if (k >= keep) break;
+        st[(size_t)k * C.ch + c] = nv[k];
+    }
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
 // State-space recurrence.  proj row layout: gate z [H*dv] | x [H*dv] | B [G*N] | C [G*N] | dt [H]; N = d of the scan's
-// arguments (the state of a head is [N, dv]), G groups of H / G heads share B and C.  The x | B | C channels pass a causal
-// convolution over the sequence's positions (taps inputs, the last tap on the current token, zeros before position 0)
-// and silu.  The convolution's last taps - 1 inputs live in the sequence's slot behind the states.
+// arguments (the state of a head is [N, dv]), G groups of H / G heads share B and C.  The x | B | C channels pass the short
+// convolution; its inputs live in the sequence's slot behind the states.
 struct SsdArgs {
     const float* proj;        // this mixer's rows of the fused projection
     const float* bias;        // of those rows, or nullptr
@@ -533,8 +634,13 @@ struct SsdArgs {
     float out_scale;
 };
 
-// Blocks (token, slice of channels): conv[t][c] = silu(b[c] + sum_k w[c][k] * in[pos - (taps-1) + k][c]); an input of an
-// earlier step comes from the slot, one before the sequence's start is zero.  The block of a token's first slice also
+__device__ __forceinline__ ConvIo conv_of(const SsdArgs& A) {
+    const int inner = A.H * A.dv;
+    return ConvIo{A.proj + inner, A.bias ? A.bias + inner : nullptr, A.n_in, inner + 2 * A.G * A.N, A.taps, A.conv_w, A.conv_b,
+                  A.seq_start, A.seq_pos0, A.seq_slot, A.slot_floats, A.conv_off, A.n_slots};
+}
+
+// Blocks (token, slice of channels): the convolved channels.  The block of a token's first slice also
 // leaves the heads' step dt = softplus(dt + bias) and decay exp(-exp(a_log) * dt) in `head` ([T][H] decay, then [T][H] step).
 __global__ void ssd_conv_kernel(const SsdArgs A, const float* __restrict__ slots, float* __restrict__ conv, float* __restrict__ head) {
     const int t = blockIdx.x, inner = A.H * A.dv, ch = inner + 2 * A.G * A.N;
@@ -547,49 +653,12 @@ __global__ void ssd_conv_kernel(const SsdArgs A, const float* __restrict__ slots
     }
     const float* before = slots + (size_t)slot * A.slot_floats + A.conv_off;      // inputs of positions pos0 - (taps-1) .. pos0 - 1
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
-    if (c < ch) {
-        float acc = A.conv_b[c];
-        const float bc = A.bias ? A.bias[inner + c] : 0.0f;
-        for (int k = 0; k < A.taps; ++k) {
-            const int back = A.taps - 1 - k;       // how many positions before the token
-            float v = 0.0f;
-            if (back <= r) v = A.proj[(size_t)(t - back) * A.n_in + inner + c] + bc;
-            else if (pos0 + r - back >= 0) v = before[(size_t)(A.taps - 1 - (back - r)) * ch + c];
-            acc = fmaf(A.conv_w[(size_t)c * A.taps + k], v, acc);
-        }
-        conv[(size_t)t * ch + c] = silu_(acc);
-    }
+    if (c < ch) conv[(size_t)t * ch + c] = conv_channel(conv_of(A), before, t, r, pos0, c);
     for (int h = threadIdx.x; blockIdx.y == 0 && h < A.H; h += blockDim.x) {
         const float raw = A.proj[(size_t)t * A.n_in + inner + ch + h] + (A.bias ? A.bias[inner + ch + h] : 0.0f);
         const float dt = softplus_(raw + A.dt_bias[h]);
         head[(size_t)t * A.H + h] = expf(-expf(A.a_log[h]) * dt);
         head[(size_t)(A.n_tokens + t) * A.H + h] = dt;
-    }
-}
-
-// After the convolution of a step the slot keeps the last taps - 1 inputs of every sequence: channel c of sequence s.  A
-// thread reads all it needs of the old inputs before it writes.  (Runs inside ssd_out_kernel, after every reader of the
-// old inputs.)
-constexpr int kMaxTaps = 16;
-__device__ __forceinline__ void ssd_conv_state_update(const SsdArgs& A, float* __restrict__ slots, int s, int c) {
-    const int inner = A.H * A.dv, ch = inner + 2 * A.G * A.N, keep = A.taps - 1;
-    const int t0 = A.seq_start[s], n = A.seq_start[s + 1] - t0, pos0 = A.seq_pos0[s];
-    const int slot = A.seq_slot[s];
-    if (slot < 0 || slot >= A.n_slots) return;
-    float* st = slots + (size_t)slot * A.slot_floats + A.conv_off;
-    const float bc = A.bias ? A.bias[inner + c] : 0.0f;
-    float nv[kMaxTaps];
-#pragma unroll
-    for (int k = 0; k < kMaxTaps; ++k) {
-        if (k >= keep) break;
-        const int back = keep - k;                 // new entry k is the input `back` positions before the next token
-        if (back <= n) nv[k] = A.proj[(size_t)(t0 + n - back) * A.n_in + inner + c] + bc;
-        else nv[k] = (pos0 + n - back >= 0) ? st[(size_t)(keep - (back - n)) * ch + c] : 0.0f;
-    }
-#pragma unroll
-    for (int k = 0; k < kMaxTaps; ++k) {
-        if (k >= keep) break;
-        st[(size_t)k * ch + c] = nv[k];
     }
 }
 
@@ -645,7 +714,7 @@ __global__ void ssd_out_kernel(const SsdArgs A, const float* __restrict__ o_raw,
         for (int c = c0 + threadIdx.x; c < c0 + len; c += blockDim.x) out[(size_t)t * A.out_ld + c] = from_f<T>(value(c) * r * A.out_norm[c]);
     }
     if ((int)blockIdx.x < A.n_seqs && A.taps > 1)          // the parts' blocks share a sequence's channels
-        for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < ch; c += gridDim.y * blockDim.x) ssd_conv_state_update(A, slots, blockIdx.x, c);
+        for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < ch; c += gridDim.y * blockDim.x) conv_state_update(conv_of(A), slots, blockIdx.x, c);
 }
 
 // ---------------------------------------------------------------------------------------------------------------------

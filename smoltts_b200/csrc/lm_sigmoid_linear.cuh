@@ -22,6 +22,7 @@ struct NormSpec {
     const float *w, *shift, *alpha;   // w == nullptr: no norm follows
     float eps;
 };
+constexpr int kNormCopy = -1;         // a kind of its own: the row itself goes on in T (the output-norm block's sublayers read the stream)
 __device__ __forceinline__ float dyt_(const NormSpec& n, float alpha, float v, int c) { return fmaf(tanhf(alpha * v), n.w[c], n.shift[c]); }
 
 // A row of D <= 8 blockDim elements in registers, 8 per thread: VEC (D % 4 == 0, rows 16-byte aligned) two 16-byte pieces of
@@ -130,6 +131,7 @@ __global__ void embed_prenorm_kernel(const int32_t* __restrict__ tokens, const T
         if (x0) x0[o + c] = v;
         if (cat) cat[2 * o + c] = cat[2 * o + D + c] = from_f<T>(v);
         if (nm.kind == SMOL_LM_NORM_DYT) hn[o + c] = from_f<T>(dyt_(nm, alpha, v, c));
+        if (nm.kind == kNormCopy) hn[o + c] = from_f<T>(v);
         ss += v * v;
     }
     if (nm.kind == SMOL_LM_NORM_DYT || !nm.w) return;
@@ -167,7 +169,8 @@ __global__ void prenorm_rows_kernel(const float* __restrict__ x, const int32_t* 
 // End of a sublayer of the pre-norm block or of a layer of the parallel block, fused with the norm in front of the next one.
 // One block per row:
 //   x <- x + sy * f(y) + sy2 * f2(y2) + s_routed * (the routed experts' weighted sum)
-// where f(y) = y, or y / rms(y) * y_w when y_w is set (mixers side by side: each projected result is normed over the width).
+// where f(y) = y, or y / rms(y) * y_w when y_w is set (mixers side by side: each projected result is normed over the width; the
+// output-norm block: the sublayer's result, to which y_b, when set, is added first: the output projection's bias).
 // `trace` then takes the row (the stream after the sublayer); x0, when set, joins x after that (the next run restarts from
 // stream + embedding output); hn <- next(x).  Routed experts: every choice has a row (no identity outputs here).  `cat`, when set, takes x in T as the first half of the row a merging run
 // multiplies (no norm follows here then).
@@ -183,6 +186,7 @@ struct ResidualArgs {
     const float* x0;
     void* cat;                            // T [rows][2 * D]
     NormSpec next;
+    const float* y_b = nullptr;           // added to y [D]
 };
 
 template <class T, bool VEC>
@@ -209,6 +213,11 @@ __global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn) {
         float xv[kRowRegs], yv[kRowRegs], nw[kRowRegs], nb[kRowRegs];
         row_load<VEC>(A.x + o, D, 0.0f, xv);
         if (A.y) row_load<VEC>(A.y + o, D, 0.0f, yv);
+        if (A.y_b) {
+            row_load<VEC>(A.y_b, D, 0.0f, nb);
+#pragma unroll
+            for (int i = 0; i < kRowRegs; ++i) yv[i] += nb[i];
+        }
         if (A.next.w) row_load<VEC>(A.next.w, D, 0.0f, nw);
         if (dyt_r || layer_r) row_load<VEC>(A.next.shift, D, 0.0f, nb);
         auto add_routed = [&](int slot, float wk) {
@@ -257,6 +266,7 @@ __global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn) {
         }
         row_store<VEC, float>(A.x + o, D, xv);
         if (A.cat) row_store<VEC, T>(static_cast<T*>(A.cat) + 2 * o, D, xv);
+        if (A.next.kind == kNormCopy) row_store<VEC, T>(hn + o, D, xv);
         if (!A.next.w) return;
         if (dyt_r) {
 #pragma unroll
@@ -282,7 +292,7 @@ __global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn) {
     if (A.y_w || A.y2_w) {
         float s1 = 0.0f, s2 = 0.0f, s3 = 0.0f;
         for (int c = threadIdx.x; c < D; c += blockDim.x) {
-            const float a = A.y[o + c], b = A.y2 ? A.y2[o + c] : 0.0f;
+            const float a = A.y[o + c] + (A.y_b ? A.y_b[c] : 0.0f), b = A.y2 ? A.y2[o + c] : 0.0f;
             s1 = fmaf(a, a, s1);
             s2 = fmaf(b, b, s2);
         }
@@ -296,7 +306,7 @@ __global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn) {
     float ss = 0.0f;
     for (int c = threadIdx.x; c < D; c += blockDim.x) {
         float v = A.x[o + c];
-        if (A.y) v = fmaf(r1 * (A.y_w ? A.y_w[c] : 1.0f), A.y[o + c], v);
+        if (A.y) v = fmaf(r1 * (A.y_w ? A.y_w[c] : 1.0f), A.y[o + c] + (A.y_b ? A.y_b[c] : 0.0f), v);
         if (A.y2) v = fmaf(r2 * (A.y2_w ? A.y2_w[c] : 1.0f), A.y2[o + c], v);
         if (A.rs.yp) {
             float acc = 0.0f;
@@ -311,6 +321,7 @@ __global__ void residual_norm_kernel(const ResidualArgs A, T* __restrict__ hn) {
         A.x[o + c] = v;
         if (A.cat) static_cast<T*>(A.cat)[2 * o + c] = from_f<T>(v);
         if (dyt) hn[o + c] = from_f<T>(dyt_(A.next, alpha, v, c));
+        else if (A.next.kind == kNormCopy) hn[o + c] = from_f<T>(v);
         else row[c] = v;
         ss = fmaf(v, v, ss);
     }

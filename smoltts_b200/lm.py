@@ -18,6 +18,9 @@ HGRN2; feed-forwards are gated or routed squared-relu experts with a shared expe
 stream), a looped span whose passes start from a matrix applied to [stream; embedding output]; softmax attention with a
 query temperature and soft-capped scores (keys and values in the paged pool) or retention (state in the slot); routed
 gated experts beside a shared expert with one gate per token; soft-capped logits.
+``VirusunLM`` serves the Virusun design: layers that norm only their sublayers' outputs; differential attention (keys of two
+maps and values in the paged pool, some layers reading an earlier layer's), the gated delta rule (state and convolution
+inputs in the slot), or rotary attention beside an mLSTM (state, key sum and running maximum in the slot); gated feed-forwards.
 
 The engine owns two pools -- key/value pages (``PagePool``) and state slots (``SlotPool``) -- and one step function,
 ``forward``: any number of sequences, each with its next tokens (a portion of a prompt or a single decoded token).
@@ -29,6 +32,7 @@ from __future__ import annotations
 
 import ctypes as C
 import json
+import math
 import os
 import struct
 from pathlib import Path
@@ -38,9 +42,9 @@ import torch
 
 from . import _capi_lm
 from ._errors import SMOL_ERR_CAPACITY, SmolError
-from .lm_config import (ACT_CLAMPED, ACT_GELU_TANH, ACT_RELU_SQUARED, ACT_SILU, BLOCK_PARALLEL, BLOCK_POSTNORM, BLOCK_PRENORM, BLOCK_SANDWICH,
+from .lm_config import (ACT_CLAMPED, ACT_GELU_TANH, ACT_RELU_SQUARED, ACT_SILU, BLOCK_OUTNORM, BLOCK_PARALLEL, BLOCK_POSTNORM, BLOCK_PRENORM, BLOCK_SANDWICH,
                         MAFERAX_MLP_KINDS, MIXER_KINDS, MLP_KINDS, NORM_DYT, NORM_LAYER, ROUTE_CHOSEN, ROUTE_SIGMOID, RUN_ADD_EMBED, RUN_MERGE_EMBED,
-                        BizulixConfig, GuniraxConfig, MaferaxConfig, PamasunConfig, SunutarConfig)
+                        BizulixConfig, GuniraxConfig, MaferaxConfig, PamasunConfig, SunutarConfig, VirusunConfig)
 from .pool import PagePool, SlotPool
 
 _ST_DTYPES = {"BF16": torch.bfloat16, "F16": torch.float16, "F32": torch.float32, "I32": torch.int32, "I64": torch.int64}
@@ -611,3 +615,75 @@ class BizulixLM(HybridLM):
             g["w_merge"] = mat("loop.in")
         return {"config": {"block": BLOCK_PARALLEL, "norm_kind": NORM_LAYER, "residual_mult": cfg.residual_mult, "logit_softcap": cfg.logit_softcap},
                 "run_flags": [RUN_MERGE_EMBED * f for f in cfg.run_merges()], "globals": g}
+
+
+class VirusunLM(HybridLM):
+    """B200 engine of one Virusun checkpoint."""
+
+    architecture = "Virusun"
+    config_class = VirusunConfig
+
+    def _shapes(self, sd):
+        return self.config.tensor_shapes()
+
+    def _describe(self, sd, layers, mat, vec):
+        cfg, D = self.config, self.config.width
+        self._sides = []                                   # the side mixers' structs live as long as the engine's create call needs them
+
+        def dot(a, b):
+            return float((sd[a].double() * sd[b].double()).sum())
+
+        for i, L in enumerate(cfg.layers):
+            p, q, c = f"l{i}.", f"l{i}.mix.", layers[i]
+            c.norm1 = vec(p + "norm1").data_ptr()
+            if L.kind == "attention":
+                m = L.mixer
+                c.mixer, c.heads, c.kv_heads, c.dim, c.vdim = MIXER_KINDS["attention"], m.heads, m.kv_heads, m.dim, m.vdim
+                c.score_scale, c.n_maps, c.diff_scale = m.scale, m.maps, 1.0 - m.diff
+                c.diff_lambda = math.exp(dot(q + "lq1", q + "lk1")) - math.exp(dot(q + "lq2", q + "lk2")) + m.diff
+                own = m.kv_from is None
+                rows = [q + "q"] + ([q + "k", q + "v"] if own else [])
+                c.kv_from = 0 if own else m.kv_from + 1
+                c.q_norm = vec(q + "q.norm").data_ptr()
+                c.k_norm = vec(q + "k.norm").data_ptr() if own else c.q_norm      # without own keys nothing is normed by it
+                bias, out = [sd[r + ".b"].float() for r in rows], [sd[q + "o"].float()]
+                rows.append(q + "g")
+                c.out_bias = vec(q + "o.b").data_ptr()
+            elif L.kind == "delta":
+                m = L.mixer
+                c.mixer, c.heads, c.kv_heads, c.dim, c.vdim = MIXER_KINDS["gated_delta"], m.heads, m.kv_heads, m.dim, m.vdim
+                c.score_scale, c.unit_eps, c.conv_taps = m.dim ** -0.5, m.unit_eps, m.conv
+                c.conv_w = vec(torch.cat([sd[q + nm + ".conv"].float() for nm in ("q", "k", "v")], 0)).data_ptr()
+                c.a_log, c.dt_bias, c.out_norm = vec(q + "A_log").data_ptr(), vec(q + "dt_bias").data_ptr(), vec(q + "norm").data_ptr()
+                rows, bias, out = [q + nm for nm in ("q", "k", "v", "g", "b", "a")], [], [sd[q + "o"].float()]
+            else:
+                # the attention is the layer's own mixer, the matrix memory its side mixer: one input product, one output product
+                a, r, lq, t = L.left, L.right, q + "left.", q + "right."
+                c.mixer, c.heads, c.kv_heads, c.dim, c.vdim = MIXER_KINDS["attention"], a.heads, a.kv_heads, a.dim, a.vdim
+                c.score_scale, c.norm_whole, c.no_gate, c.mix_scale = a.scale, 1, 1, L.left_scale
+                c.q_norm, c.k_norm = vec(lq + "q.norm").data_ptr(), vec(lq + "k.norm").data_ptr()
+                c.rot_dims, c.rot_base, c.rot_half, c.rot_mult = a.rot.dims, a.rot.base, 1, a.rot.mult
+                c.rot_yarn, c.rot_original, c.rot_fast, c.rot_slow = a.rot.factor, a.rot.original, a.rot.fast, a.rot.slow
+                side = _capi_lm.SmolLmLayer()
+                side.mixer, side.heads, side.kv_heads, side.dim, side.vdim = MIXER_KINDS["mlstm"], r.heads, r.heads, r.dim, r.vdim
+                side.mix_scale, side.score_scale, side.gate_cap, side.den_eps = L.right_scale, r.dim ** -0.5, r.gate_cap, r.den_eps
+                side.rate_bias, side.decay_bias, side.out_norm = vec(t + "i.b").data_ptr(), vec(t + "f.b").data_ptr(), vec(t + "norm").data_ptr()
+                self._sides.append(side)
+                c.side = C.pointer(side)
+                rows, bias = [lq + "q", lq + "k", lq + "v"], [sd[lq + nm + ".b"].float() for nm in ("q", "k", "v")]
+                rows += [t + nm for nm in ("q", "k", "v", "g", "i", "f")]
+                out = [sd[lq + "o"].float(), sd[t + "o"].float()]
+                c.out_bias = vec(sd[lq + "o.b"].float() * L.left_scale).data_ptr()
+            n_in = sum(int(sd[x].shape[0]) for x in rows)
+            if n_in % 8:
+                rows.append(torch.zeros(8 - n_in % 8, D))
+            if bias:
+                bias = torch.cat(bias)
+                c.in_bias = vec(torch.cat([bias, torch.zeros((n_in + 7) // 8 * 8 - bias.numel())])).data_ptr()
+            c.w_in, c.w_out = mat(*rows).data_ptr(), mat(torch.cat(out, 1)).data_ptr()
+            c.mlp = MAFERAX_MLP_KINDS["dense" if L.ff else None]
+            if L.ff:
+                c.ff, c.mlp_act, c.norm2 = L.ff, ACT_SILU, vec(p + "norm2").data_ptr()
+                c.w_up, c.w_down = mat(p + "mlp.gate", p + "mlp.up").data_ptr(), mat(p + "mlp.down").data_ptr()
+        return {"config": {"block": BLOCK_OUTNORM},
+                "globals": {"embed": mat("embed"), "head": mat("head"), "final_norm": vec("final.norm")}}

@@ -15,13 +15,13 @@ from typing import Any, Dict, List, Optional
 
 # values of SMOL_LM_MIX_* (include/smoltts_b200_lm.h)
 MIXER_KINDS = {"attention": 0, "general_delta": 1, "latent_attention": 2, "gla": 3, "state_space": 4, "sigmoid_attention": 5,
-               "lightning": 6, "hgrn2": 7, "retention": 8}
+               "lightning": 6, "hgrn2": 7, "retention": 8, "gated_delta": 9, "mlstm": 10}
 MLP_KINDS = {None: 0, "dense": 1}                        # SMOL_LM_MLP_* of Pamasun: "dense" = up, PolyNorm, down
 # SMOL_LM_MLP_* of Maferax: "dense" = gated (tanh-form gelu), "moe" = routed mixture of gated (silu) experts
 MAFERAX_MLP_KINDS = {None: 0, "dense": 2, "moe": 3}
 ACT_GELU_TANH, ACT_SILU, ACT_CLAMPED, ACT_RELU_SQUARED = 0, 1, 2, 3      # SMOL_LM_ACT_*
 ROUTE_SOFTMAX, ROUTE_SIGMOID, ROUTE_CHOSEN = 0, 1, 2     # SMOL_LM_ROUTE_*
-BLOCK_SANDWICH, BLOCK_POSTNORM, BLOCK_PRENORM, BLOCK_PARALLEL = 0, 1, 2, 3   # SMOL_LM_BLOCK_*
+BLOCK_SANDWICH, BLOCK_POSTNORM, BLOCK_PRENORM, BLOCK_PARALLEL, BLOCK_OUTNORM = 0, 1, 2, 3, 4   # SMOL_LM_BLOCK_*
 NORM_RMS, NORM_DYT, NORM_LAYER = 0, 1, 2                 # SMOL_LM_NORM_*
 RUN_ADD_EMBED, RUN_MERGE_EMBED = 1, 2                    # SMOL_LM_RUN_*
 
@@ -1055,3 +1055,266 @@ class BizulixConfig:
     def matmul_flops_per_token(self) -> int:
         per = self._elements_by_part(True)
         return int(2 * (sum(per.get(i, 0.0) for i in self.layer_runs()) + sum(self.run_merges()) * per.get("loop.in", 0.0) + per["head"]))
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Virusun: layers that norm only what their sublayers return.  Mixers: differential attention (two softmax maps per head over
+# the same values, one subtracted from the other; some layers read an earlier layer's keys and values), the gated delta rule
+# behind short convolutions, or a pair on the same input -- rotary softmax attention beside an mLSTM -- summed with two scales.
+# Feed-forwards: gated (silu) or none.
+
+
+@dataclass
+class RampRotarySpec:
+    """Rotation of halves (coordinate i with i + dims / 2), its frequencies interpolated along a ramp (factor 0: not)."""
+    base: float = 10000.0
+    dims: int = 0
+    factor: float = 0.0
+    original: float = 0.0
+    fast: float = 32.0
+    slow: float = 1.0
+
+    @classmethod
+    def from_dict(cls, d: Optional[Dict[str, Any]]) -> "RampRotarySpec":
+        if not d:
+            return cls()
+        sc = d.get("scaling") or {}
+        spec = cls(float(d["base"]), int(d["dims"]))
+        if sc:
+            spec.factor, spec.original, spec.fast, spec.slow = float(sc["factor"]), float(sc["original"]), float(sc["fast"]), float(sc["slow"])
+        if spec.dims % 2 or spec.dims < 0 or spec.base <= 0 or (sc and (spec.factor <= 0 or spec.original <= 0 or spec.fast <= 0 or spec.slow <= 0)):
+            raise ValueError("rotary: dims must be even, base and the scaling's numbers positive")
+        return spec
+
+    def to_dict(self) -> Dict[str, Any]:
+        d: Dict[str, Any] = {"base": self.base, "dims": self.dims}
+        if self.factor:
+            d["scaling"] = {"factor": self.factor, "original": self.original, "fast": self.fast, "slow": self.slow}
+        return d
+
+    @property
+    def mult(self) -> float:
+        """Multiplies cosine and sine."""
+        return 0.1 * math.log(self.factor) + 1.0 if self.factor else 1.0
+
+
+@dataclass
+class DiffAttentionSpec:
+    kind = "attention"
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    diff: float                     # constant part of the second map's weight
+    kv_from: Optional[int] = None   # layer whose keys and values are read (None: own)
+    maps = 2                        # fixed by the design
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "DiffAttentionSpec":
+        src = d.get("kv_from")
+        spec = cls(int(d["heads"]), int(d.get("kv_heads", d["heads"])), int(d["dim"]), int(d.get("vdim", d["dim"])), float(d["scale"]), float(d["diff"]),
+                   None if src is None else int(src))
+        if spec.kv_heads < 1 or spec.heads % spec.kv_heads:
+            raise ValueError("attention: heads must be a multiple of kv_heads")
+        return spec
+
+    def to_dict(self) -> Dict[str, Any]:
+        d = {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale, "diff": self.diff}
+        if self.kv_from is not None:
+            d["kv_from"] = self.kv_from
+        return d
+
+
+@dataclass
+class GatedDeltaSpec:
+    kind = "gated_delta"
+    heads: int                      # value heads; each reads key head floor(h / (heads / kv_heads))
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int                       # taps of the convolutions
+    unit_eps = 1e-6                 # fixed by the design: unit vectors are x / sqrt(sum x^2 + unit_eps)
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "GatedDeltaSpec":
+        spec = cls(int(d["heads"]), int(d.get("kv_heads", d["heads"])), int(d["dim"]), int(d.get("vdim", d["dim"])), int(d["conv"]))
+        if spec.kv_heads < 1 or spec.heads % spec.kv_heads or spec.conv < 1:
+            raise ValueError("delta: heads must be a multiple of kv_heads, conv at least 1")
+        return spec
+
+    def to_dict(self) -> Dict[str, Any]:
+        return {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "conv": self.conv}
+
+    @property
+    def channels(self) -> int:
+        """Channels that pass the convolutions: q | k | v."""
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+
+@dataclass
+class RotaryAttentionSpec:
+    kind = "attention"
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: RampRotarySpec
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "RotaryAttentionSpec":
+        spec = cls(int(d["heads"]), int(d.get("kv_heads", d["heads"])), int(d["dim"]), int(d.get("vdim", d["dim"])), float(d["scale"]),
+                   RampRotarySpec.from_dict(d.get("rot")))
+        if spec.kv_heads < 1 or spec.heads % spec.kv_heads or spec.rot.dims > spec.dim:
+            raise ValueError("attention: heads must be a multiple of kv_heads, rot.dims at most dim")
+        return spec
+
+    def to_dict(self) -> Dict[str, Any]:
+        return {"heads": self.heads, "kv_heads": self.kv_heads, "dim": self.dim, "vdim": self.vdim, "scale": self.scale, "rot": self.rot.to_dict()}
+
+
+@dataclass
+class MlstmSpec:
+    kind = "mlstm"
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+    den_eps = 1e-6                  # fixed by the design: added to the denominator
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "MlstmSpec":
+        spec = cls(int(d["heads"]), int(d["dim"]), int(d.get("vdim", d["dim"])), float(d["gate_cap"]))
+        if spec.gate_cap <= 0:
+            raise ValueError("mLSTM: gate_cap must be positive")
+        return spec
+
+    def to_dict(self) -> Dict[str, Any]:
+        return {"heads": self.heads, "dim": self.dim, "vdim": self.vdim, "gate_cap": self.gate_cap}
+
+
+@dataclass
+class VirusunLayer:
+    kind: str                                # "attention" | "delta" | "parallel"
+    mixer: Any = None                        # DiffAttentionSpec | GatedDeltaSpec
+    left: Optional[RotaryAttentionSpec] = None
+    right: Optional[MlstmSpec] = None
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+    ff: int = 0                              # feed-forward size (0: none)
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "VirusunLayer":
+        m = d["mixer"]
+        if d["type"] == "attention":
+            L = cls("attention", DiffAttentionSpec.from_dict(m))
+        elif d["type"] == "delta":
+            L = cls("delta", GatedDeltaSpec.from_dict(m))
+        elif d["type"] == "parallel":
+            L = cls("parallel", None, RotaryAttentionSpec.from_dict(m["left"]), MlstmSpec.from_dict(m["right"]), float(m["left_scale"]), float(m["right_scale"]))
+        else:
+            raise ValueError(f"unknown mixer type {d['type']!r}; have ['attention', 'delta', 'parallel']")
+        mlp = d.get("mlp")
+        if mlp:
+            if mlp["kind"] != "dense":
+                raise ValueError(f"unknown feed-forward kind {mlp['kind']!r}")
+            L.ff = int(mlp["ff"])
+            if L.ff < 1:
+                raise ValueError("feed-forward: ff must be positive")
+        return L
+
+    def to_dict(self) -> Dict[str, Any]:
+        mixer = self.mixer.to_dict() if self.mixer is not None else {"left": self.left.to_dict(), "right": self.right.to_dict(),
+                                                                     "left_scale": self.left_scale, "right_scale": self.right_scale}
+        return {"type": self.kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": self.ff} if self.ff else None}
+
+
+@dataclass
+class VirusunConfig:
+    architecture: str = "Virusun"
+    vocab: int = 0
+    width: int = 0
+    norm_eps: float = 1e-6
+    layers: List[VirusunLayer] = field(default_factory=list)
+    extra: Dict[str, Any] = field(default_factory=dict, repr=False)
+
+    @classmethod
+    def from_dict(cls, d: Dict[str, Any]) -> "VirusunConfig":
+        known = {"architecture", "vocab", "width", "norm", "layers"}
+        cfg = cls(architecture=d.get("architecture", "Virusun"), vocab=int(d["vocab"]), width=int(d["width"]), norm_eps=float(d["norm"]["eps"]),
+                  layers=[VirusunLayer.from_dict(x) for x in d["layers"]], extra={k: v for k, v in d.items() if k not in known})
+        for i, L in enumerate(cfg.layers):
+            if L.kind != "attention" or L.mixer.kv_from is None:
+                continue
+            j, m = L.mixer.kv_from, L.mixer
+            o = cfg.layers[j].mixer if 0 <= j < i and cfg.layers[j].kind == "attention" else None
+            if o is None or o.kv_from is not None or (o.kv_heads, o.dim, o.vdim) != (m.kv_heads, m.dim, m.vdim):
+                raise ValueError(f"layer {i}: kv_from must name an earlier attention layer with own keys and values of the same sizes")
+        return cfg
+
+    @classmethod
+    def from_pretrained(cls, pathname: str) -> "VirusunConfig":
+        path = Path(pathname)
+        if path.is_dir():
+            path = path / "config.json"
+        with open(path, "r", encoding="utf-8") as f:
+            return cls.from_dict(json.load(f))
+
+    def to_dict(self) -> Dict[str, Any]:
+        d = dict(self.extra)
+        d.update(architecture=self.architecture, vocab=self.vocab, width=self.width, norm={"eps": self.norm_eps}, layers=[x.to_dict() for x in self.layers])
+        return d
+
+    def save(self, path: str) -> None:
+        with open(path, "w") as f:
+            json.dump(self.to_dict(), f, indent=1, sort_keys=True)
+
+    def layer_runs(self) -> List[int]:
+        return list(range(len(self.layers)))
+
+    def tensor_shapes(self) -> Dict[str, tuple]:
+        """Checkpoint tensor names and shapes."""
+        D, V = self.width, self.vocab
+        out: Dict[str, tuple] = {"embed": (V, D), "head": (V, D), "final.norm": (D,)}
+
+        def attention(q, a, maps, own):
+            nq, nk, nv = a.heads * maps * a.dim, a.kv_heads * maps * a.dim, a.kv_heads * a.vdim
+            for nm, rows in (("q", nq),) + ((("k", nk), ("v", nv)) if own else ()):
+                out.update({q + nm: (rows, D), q + nm + ".b": (rows,)})
+            out.update({q + "o": (D, a.heads * a.vdim), q + "o.b": (D,)})
+            return nq, nk
+
+        for i, L in enumerate(self.layers):
+            p, q = f"l{i}.", f"l{i}.mix."
+            out[p + "norm1"] = (D,)
+            if L.kind == "attention":
+                m = L.mixer
+                own = m.kv_from is None
+                attention(q, m, m.maps, own)
+                out.update({q + nm: (m.dim,) for nm in ("q.norm", "lq1", "lk1", "lq2", "lk2") + (("k.norm",) if own else ())})
+                out[q + "g"] = (m.heads * m.vdim, D)
+            elif L.kind == "delta":
+                m = L.mixer
+                for nm, rows in (("q", m.kv_heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.heads * m.vdim)):
+                    out.update({q + nm: (rows, D), q + nm + ".conv": (rows, m.conv)})
+                out.update({q + "b": (m.heads, D), q + "a": (m.heads, D), q + "A_log": (m.heads,), q + "dt_bias": (m.heads,), q + "norm": (m.vdim,),
+                            q + "g": (m.heads * m.vdim, D), q + "o": (D, m.heads * m.vdim)})
+            else:
+                nq, nk = attention(q + "left.", L.left, 1, True)
+                out.update({q + "left.q.norm": (nq,), q + "left.k.norm": (nk,)})
+                t, r = q + "right.", L.right
+                hd, hv = r.heads * r.dim, r.heads * r.vdim
+                out.update({t + "q": (hd, D), t + "k": (hd, D), t + "v": (hv, D), t + "g": (hv, D), t + "o": (D, hv), t + "norm": (hv,),
+                            t + "i": (r.heads, D), t + "i.b": (r.heads,), t + "f": (r.heads, D), t + "f.b": (r.heads,)})
+            if L.ff:
+                out.update({p + "norm2": (D,), p + "mlp.gate": (L.ff, D), p + "mlp.up": (L.ff, D), p + "mlp.down": (D, L.ff)})
+        return out
+
+    # ---- accounting used by the benchmark ----
+    def weight_elements(self) -> int:
+        """Matrix elements one token touches (without the embedding table)."""
+        return sum(s[0] * s[1] for k, s in self.tensor_shapes().items() if len(s) == 2 and k != "embed" and not k.endswith(".conv"))
+
+    def matmul_flops_per_token(self) -> int:
+        return 2 * self.weight_elements()

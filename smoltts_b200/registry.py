@@ -24,6 +24,7 @@ register_model("Maferax", "smoltts_b200.lm", "MaferaxLM")
 register_model("Sunutar", "smoltts_b200.lm", "SunutarLM")
 register_model("Gunirax", "smoltts_b200.lm", "GuniraxLM")
 register_model("Bizulix", "smoltts_b200.lm", "BizulixLM")
+register_model("Virusun", "smoltts_b200.lm", "VirusunLM")
 
 
 def registered() -> Dict[str, Tuple[str, str]]:
