@@ -134,6 +134,11 @@ def rotary_attention(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, m: dic
     return out.reshape(n, H * dv) @ w[p + "o"].T + w[p + "o.b"]
 
 
+def memory_denominator(dot: torch.Tensor, m: torch.Tensor) -> torch.Tensor:
+    """dot: key sum . query, m: running maximum (the memory holds everything times e^-m)."""
+    return torch.maximum(dot.abs(), torch.exp(-m)) + DEN_EPS
+
+
 def mlstm(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, m: dict, eps: float, past: Optional[dict] = None) -> torch.Tensor:
     """h [n, width] -> [n, width].  ``past``: {"S": [heads, d, dv], "n": [heads, d], "m": [heads]}, updated in place."""
     H, d, dv, cap = m["heads"], m["dim"], m["vdim"], m["gate_cap"]
@@ -154,8 +159,7 @@ def mlstm(h: torch.Tensor, w: Dict[str, torch.Tensor], p: str, m: dict, eps: flo
         S = keep[:, None, None] * S + write[:, None, None] * k[t][:, :, None] * v[t][:, None, :]
         nn = keep[:, None] * nn + write[:, None] * k[t]
         mx = new
-        den = torch.maximum((nn * q[t]).sum(-1).abs(), torch.exp(-mx)) + DEN_EPS
-        o[t] = (S * q[t][:, :, None]).sum(1) / den[:, None]
+        o[t] = (S * q[t][:, :, None]).sum(1) / memory_denominator((nn * q[t]).sum(-1), mx)[:, None]
     if past is not None:
         past["S"], past["n"], past["m"] = S, nn, mx
     y = rms_divide(o, eps).reshape(n, H * dv) * w[p + "norm"] * torch.sigmoid(h @ w[p + "g"].T)
