@@ -1,7 +1,8 @@
 """Prefill and decode throughput of the hybrid language-model engine at layer sizes that resemble a real model's:
 the Pamasun design beside the DualAR slow transformer (the package's closest model: attention + gated MLP layers), and the
 Maferax and Sunutar designs beside Pamasun at equal width, depth and head count (``--lm-design maferax`` / ``sunutar``),
-the Gunirax design beside Sunutar (``--lm-design gunirax``), and the Bizulix design beside Maferax (``--lm-design bizulix``).
+the Gunirax design beside Sunutar (``--lm-design gunirax``), the Bizulix design beside Maferax (``--lm-design bizulix``), and the Virusun design
+beside Pamasun (``--lm-design virusun``).
 
 ``python bench.py --lm`` prints one JSON line: for every size, tokens/s of a whole-prompt prefill and of single-token
 decode steps against a filled cache, each with its distance from the roofline (matrix-product + attention flops over the
@@ -471,6 +472,120 @@ def bench_bizulix(name: str, prompt: int, batch: int, decode_steps: int, warmup:
             "gpu_launches": int(launches)}
 
 
+VIRUSUN_SIZES = {
+    # layers after Pamasun's pattern (d = gated delta rule, heads x (dim keys, dim values) over kv_heads key heads; a = differential
+    # attention, heads / 2 heads of two maps x dim with values of 2 dim over kv_heads / 2, so that a cached position takes what
+    # Pamasun's takes; b = the same reading the keys and values of the last "a"; p = rotary attention heads x dim over kv_heads beside
+    # an mLSTM heads x (dim, dim)); dense gated feed-forward with as many elements as Pamasun's two-matrix one
+    "w768": dict(width=768, layers=10, heads=12, kv_heads=4, dim=64, ff=3072, vocab=2368, pattern="daa"),
+    "w768mix": dict(width=768, layers=10, heads=12, kv_heads=4, dim=64, ff=3072, vocab=2368, pattern="adbp"),
+    "w1536": dict(width=1536, layers=12, heads=12, kv_heads=4, dim=128, ff=4096, vocab=8192, pattern="adbp"),
+}
+
+
+def virusun_config(width, layers, heads, kv_heads, dim, ff, vocab, pattern) -> dict:
+    ls, last = [], 0
+    for i in range(layers):
+        mlp, kind = {"kind": "dense", "ff": ff}, pattern[i % len(pattern)]
+        if kind in "ab":
+            # a head size of 128 would need values of 256: the maps then take half of it
+            d, h = (dim, heads // 2) if dim <= 64 else (dim // 2, heads)
+            m = {"heads": h, "kv_heads": kv_heads // (heads // h), "dim": d, "vdim": 2 * d, "scale": d ** -0.5, "diff": 0.5}
+            if kind == "b":
+                m["kv_from"] = last
+            else:
+                last = i
+            ls.append({"type": "attention", "mixer": m, "mlp": mlp})
+        elif kind == "d":
+            ls.append({"type": "delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "conv": 4}, "mlp": mlp})
+        else:
+            ls.append({"type": "parallel", "mlp": mlp,
+                       "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                                          "rot": {"base": 10000.0, "dims": dim, "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}},
+                                 "right": {"heads": heads, "dim": dim, "vdim": dim, "gate_cap": 15.0}, "left_scale": 1.0, "right_scale": 1.0}})
+    return {"architecture": "Virusun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": ls}
+
+
+def virusun_state_dict(cfg, seed: int = 0) -> Dict[str, torch.Tensor]:
+    g = torch.Generator().manual_seed(seed)
+    sd = {}
+    for k, s in cfg.tensor_shapes().items():
+        if len(s) == 2:
+            sd[k] = (torch.randn(*s, generator=g) * (s[1] ** -0.5)).bfloat16()
+        elif k.endswith((".norm", "norm1", "norm2")):
+            sd[k] = torch.full(s, 0.5 if k.endswith(("norm1", "norm2")) else 1.0).bfloat16()
+        elif k.endswith(("A_log", "dt_bias", "f.b")):
+            sd[k] = torch.full(s, {"A_log": -1.0, "dt_bias": -1.0}.get(k.rsplit(".", 1)[1], 4.0)).bfloat16()
+        else:
+            sd[k] = (torch.randn(*s, generator=g) * 0.05).bfloat16()
+    sd["embed"] = torch.randn(*sd["embed"].shape, generator=g).bfloat16()
+    return sd
+
+
+def bench_virusun(name: str, prompt: int, batch: int, decode_steps: int, warmup: int, steps: int, peaks) -> dict:
+    """Like bench_pamasun.  Prefill flops: matrix products, attention (per visible key and score map 2 dim + 2 vdim flops), delta rule
+    (8 dim vdim per head and token: two reads, decay and write) and mLSTM (6 dim vdim); decode bytes: the weights, the keys and values
+    every attention layer reads, and the states (read and written)."""
+    from .lm import VirusunLM
+    from .lm_config import VirusunConfig
+
+    hbm, tflops, _ = peaks
+    spec = VIRUSUN_SIZES[name]
+    cfg = VirusunConfig.from_dict(virusun_config(**spec))
+    model = VirusunLM(cfg, dtype=torch.bfloat16, max_tokens=batch * (prompt + 64 + decode_steps), max_seqs=batch, page_size=64,
+                      max_step_tokens=2048, max_want=batch)
+    model.load_state_dict(virusun_state_dict(cfg, 0))
+    g = torch.Generator().manual_seed(1)
+    toks = torch.randint(0, cfg.vocab, (batch, prompt + decode_steps), generator=g).tolist()
+    pair_flops = kv_elems = rec_flops = st_elems = 0                  # per visible key; per cached position; per token; per sequence
+    for L in cfg.layers:
+        a = L.mixer if L.kind == "attention" else L.left
+        if a is not None:
+            maps = L.mixer.maps if L.kind == "attention" else 1
+            pair_flops += a.heads * maps * (2 * a.dim + 2 * a.vdim)
+            kv_elems += a.kv_heads * (maps * a.dim + a.vdim)
+        r = L.mixer if L.kind == "delta" else L.right
+        if r is not None:
+            rec_flops += (8 if L.kind == "delta" else 6) * r.heads * r.dim * r.vdim
+            st_elems += r.heads * r.dim * r.vdim
+
+    def prefill():
+        seq = model.open_sequence()
+        for lo in range(0, prompt, model.max_step_tokens):
+            part = toks[0][lo:min(prompt, lo + model.max_step_tokens)]
+            model.forward([(seq, part, [len(part) - 1] if lo + len(part) == prompt else [])])
+        model.close_sequence(seq)
+
+    l0 = model.launch_count
+    ms_p = _timed(prefill, warmup, steps)
+    launches = model.launch_count - l0
+    flops_p = prompt * (cfg.matmul_flops_per_token() - 2 * cfg.vocab * cfg.width + rec_flops) + pair_flops * prompt * (prompt + 1) / 2
+    seqs = [model.open_sequence() for _ in range(batch)]
+    for b, s in enumerate(seqs):
+        for lo in range(0, prompt, model.max_step_tokens):
+            model.forward([(s, toks[b][lo:min(prompt, lo + model.max_step_tokens)], [])])
+
+    def decode():
+        for i in range(decode_steps):
+            model.forward([(s, [toks[b][prompt + i]], [0]) for b, s in enumerate(seqs)])
+        for s in seqs:
+            s.length = prompt
+
+    l0 = model.launch_count
+    ms_d = _timed(decode, 2, steps) / decode_steps
+    launches += model.launch_count - l0
+    bytes_d = 2 * cfg.weight_elements() + batch * (kv_elems * 2 * (prompt + decode_steps / 2) + st_elems * 2 * 4)
+    model.check_device_errors()
+    for s in seqs:
+        model.close_sequence(s)
+    return {"model": f"Virusun {name}", "spec": spec, "parameters_m": round(cfg.weight_elements() / 1e6, 1),
+            "prefill": {"prompt": prompt, "tokens_per_s": prompt / ms_p * 1e3, "ms": ms_p, "tflops": flops_p / ms_p / 1e9,
+                        "of_peak": flops_p / ms_p / 1e9 / tflops},
+            "decode": {"batch": batch, "context": prompt, "tokens_per_s": batch / ms_d * 1e3, "ms_per_step": ms_d,
+                       "gbs": bytes_d / ms_d / 1e6, "of_peak": bytes_d / ms_d / 1e6 / hbm},
+            "gpu_launches": int(launches)}
+
+
 def pamasun_config(width, layers, heads, kv_heads, dim, ff, vocab, pattern) -> dict:
     ls = []
     for i in range(layers):
@@ -642,7 +757,17 @@ def run(args, root: str) -> None:
     peaks = _peaks(root)
     t0 = time.time()
     entries: List[dict] = []
-    if getattr(args, "lm_design", "pamasun") == "bizulix":
+    if getattr(args, "lm_design", "pamasun") == "virusun":
+        # Virusun beside Pamasun (the engine's closest design: attention and a delta rule, dense feed-forwards) at equal width, depth,
+        # state sizes, cached bytes per attention layer and feed-forward elements
+        names = [n for n in (args.lm_sizes.split(",") if args.lm_sizes else ["w768", "w768mix", "w1536"])]
+        for n in names:
+            for batch in (1, 4):
+                entries.append(bench_virusun(n, args.lm_prompt, batch, 16, args.warmup, args.steps, peaks))
+        for n in sorted({"w1536" if n == "w1536" else "w768" for n in names}):
+            for batch in (1, 4):
+                entries.append(bench_pamasun(n, args.lm_prompt, batch, 16, args.warmup, args.steps, peaks))
+    elif getattr(args, "lm_design", "pamasun") == "bizulix":
         # Bizulix beside Maferax (the engine's closest design: every layer either an attention over the paged pool or a linear recurrence
         # on the shared scan, routed silu experts) at equal width, depth, heads, state sizes and active feed-forward size
         names = [n for n in (args.lm_sizes.split(",") if args.lm_sizes else ["w768", "w768loop", "w1536"])]
