@@ -919,35 +919,45 @@ __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
 __device__ __forceinline__ void cp_async_commit_group() { asm volatile("cp.async.commit_group;" ::); }
 template <int N> __device__ __forceinline__ void cp_async_wait_group() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// q (fp32, shared memory) . k (one cached key row), 16-byte loads where the row allows them
+// q (fp32, shared memory) . k (one cached key row), 16-byte loads where both rows allow them
 template <class T> __device__ __forceinline__ float key_dot(const float* qs, const T* k, int d);
 template <> __device__ __forceinline__ float key_dot<float>(const float* qs, const float* k, int d) {
-    float dot = 0.0f;
-    if (d % 4 == 0 && reinterpret_cast<uintptr_t>(k) % 16 == 0) {
+    float a0 = 0.0f, a1 = 0.0f, a2 = 0.0f, a3 = 0.0f;
+    if (d % 4 == 0 && (reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(qs)) % 16 == 0) {
         for (int c = 0; c < d; c += 4) {
-            const float4 v = *reinterpret_cast<const float4*>(k + c);
-            dot = fmaf(qs[c], v.x, dot); dot = fmaf(qs[c + 1], v.y, dot); dot = fmaf(qs[c + 2], v.z, dot); dot = fmaf(qs[c + 3], v.w, dot);
+            const float4 v = *reinterpret_cast<const float4*>(k + c), x = *reinterpret_cast<const float4*>(qs + c);
+            a0 = fmaf(x.x, v.x, a0); a1 = fmaf(x.y, v.y, a1); a2 = fmaf(x.z, v.z, a2); a3 = fmaf(x.w, v.w, a3);
         }
     } else {
-        for (int c = 0; c < d; ++c) dot = fmaf(qs[c], k[c], dot);
+        for (int c = 0; c < d; ++c) a0 = fmaf(qs[c], k[c], a0);
     }
-    return dot;
+    return (a0 + a1) + (a2 + a3);
 }
 template <> __device__ __forceinline__ float key_dot<bf16>(const float* qs, const bf16* k, int d) {
-    float dot = 0.0f;
-    if (d % 8 == 0 && reinterpret_cast<uintptr_t>(k) % 16 == 0) {
+    float a0 = 0.0f, a1 = 0.0f, a2 = 0.0f, a3 = 0.0f;
+    if (d % 8 == 0 && (reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(qs)) % 16 == 0) {
         for (int c = 0; c < d; c += 8) {
-            const uint4 v = ldg_v4(k + c);
-            dot = fmaf(qs[c], bf_lo(v.x), dot); dot = fmaf(qs[c + 1], bf_hi(v.x), dot);
-            dot = fmaf(qs[c + 2], bf_lo(v.y), dot); dot = fmaf(qs[c + 3], bf_hi(v.y), dot);
-            dot = fmaf(qs[c + 4], bf_lo(v.z), dot); dot = fmaf(qs[c + 5], bf_hi(v.z), dot);
-            dot = fmaf(qs[c + 6], bf_lo(v.w), dot); dot = fmaf(qs[c + 7], bf_hi(v.w), dot);
+            const uint4 v = *reinterpret_cast<const uint4*>(k + c);
+            const float4 x = *reinterpret_cast<const float4*>(qs + c), y = *reinterpret_cast<const float4*>(qs + c + 4);
+            a0 = fmaf(x.x, bf_lo(v.x), a0); a1 = fmaf(x.y, bf_hi(v.x), a1);
+            a2 = fmaf(x.z, bf_lo(v.y), a2); a3 = fmaf(x.w, bf_hi(v.y), a3);
+            a0 = fmaf(y.x, bf_lo(v.z), a0); a1 = fmaf(y.y, bf_hi(v.z), a1);
+            a2 = fmaf(y.z, bf_lo(v.w), a2); a3 = fmaf(y.w, bf_hi(v.w), a3);
         }
     } else {
-        for (int c = 0; c < d; ++c) dot = fmaf(qs[c], __bfloat162float(k[c]), dot);
+        for (int c = 0; c < d; ++c) a0 = fmaf(qs[c], __bfloat162float(k[c]), a0);
     }
-    return dot;
+    return (a0 + a1) + (a2 + a3);
 }
+
+// two neighbouring elements (the address is a multiple of their size)
+__device__ __forceinline__ float2 load_pair(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 load_pair(const bf16* p) {
+    const uint32_t v = *reinterpret_cast<const uint32_t*>(p);
+    return make_float2(bf_lo(v), bf_hi(v));
+}
+// row stride of the staged values: an even number of elements
+template <class T> __host__ __device__ constexpr int split_value_ld(int dv) { return (dv + 16 / (int)sizeof(T) + 1) / 2 * 2; }
 
 template <class T, int MAXV>
 __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const T* __restrict__ qbuf, const T* __restrict__ pool) {
@@ -973,7 +983,7 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bool active = hq < Gq;
     const int h = g * Gq + (active ? hq : 0), map = h % A.maps, head = h / A.maps;      // h: query row
-    const int ldk = A.d + kPad, ldv = A.v_in_k ? ldk : A.dv + kPad;
+    const int ldk = A.v_in_k ? (A.d + kPad + 1) / 2 * 2 : A.d + kPad, ldv = A.v_in_k ? ldk : split_value_ld<T>(A.dv);
     float* qs = reinterpret_cast<float*>(sm_raw) + warp * A.d;
     float* ps = reinterpret_cast<float*>(sm_raw) + nwarp * A.d + warp * 32;
     T* Ks = reinterpret_cast<T*>(sm_raw + (((size_t)nwarp * (A.d + 32) * 4 + 15) / 16) * 16);
@@ -982,7 +992,7 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
     for (int c = lane; c < A.d; c += 32) qs[c] = to_f<T>(qbuf[((size_t)t * A.H * A.maps + h) * A.d + c]);
     const float r1 = A.r1 ? A.r1[head] : 0.0f, r2 = A.r1 ? A.r2[head] : 0.0f, slope = A.slope ? A.slope[head] : 0.0f;
     float m = -INFINITY, l = 0.0f;
-    float o[MAXV];
+    float o[MAXV];                       // columns 2 lane + 64 (e / 2) + e % 2
 #pragma unroll
     for (int e = 0; e < MAXV; ++e) o[e] = 0.0f;
     // whole 16-byte pieces when every cached row starts on a 16-byte boundary (pages are 16-byte aligned)
@@ -992,22 +1002,23 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
     for (int j0 = j_lo; j0 <= j_hi; j0 += 32) {
         const int cnt = min(32, j_hi - j0 + 1);
         __syncthreads();
-        for (int idx = threadIdx.x; idx < cnt * (kchunks + vchunks); idx += blockDim.x) {
-            const int row = idx / (kchunks + vchunks), c = idx % (kchunks + vchunks);
-            const int j = j0 + row;
-            const T* base = pool + (size_t)bt[j / A.page_size] * A.page_elems;
-            const int in_pg = j % A.page_size;
-            if (c < kchunks) {
-                const int km = c / kchunk1, ck = c - km * kchunk1;
-                const T* src = base + A.k_off + ((size_t)(g * A.maps + km) * A.page_size + in_pg) * A.k_ld;
-                T* dst = Ks + (km * 32 + row) * ldk;
-                if (kvec) cp_async16(dst + ck * kPad, src + ck * kPad);
-                else dst[ck] = src[ck];
-            } else {
-                const int cv = c - kchunks;
-                const T* src = base + A.v_off + ((size_t)g * A.page_size + in_pg) * A.v_ld;
-                if (vvec) cp_async16(Vs + row * ldv + cv * kPad, src + cv * kPad);
-                else Vs[row * ldv + cv] = src[cv];
+        // a warp per cached row, its lanes side by side over the row's pieces
+        for (int row = warp; row < cnt; row += nwarp) {
+            const int jr = j0 + row, pg = jr / A.page_size, in_pg = jr - pg * A.page_size;
+            const T* base = pool + (size_t)bt[pg] * A.page_elems;
+            for (int c = lane; c < kchunks + vchunks; c += 32) {
+                if (c < kchunks) {
+                    const int km = A.maps > 1 ? c / kchunk1 : 0, ck = c - km * kchunk1;
+                    const T* src = base + A.k_off + ((size_t)(g * A.maps + km) * A.page_size + in_pg) * A.k_ld;
+                    T* dst = Ks + (km * 32 + row) * ldk;
+                    if (kvec) cp_async16(dst + ck * kPad, src + ck * kPad);
+                    else dst[ck] = src[ck];
+                } else {
+                    const int cv = c - kchunks;
+                    const T* src = base + A.v_off + ((size_t)g * A.page_size + in_pg) * A.v_ld;
+                    if (vvec) cp_async16(Vs + row * ldv + cv * kPad, src + cv * kPad);
+                    else Vs[row * ldv + cv] = src[cv];
+                }
             }
         }
         cp_async_commit_group();
@@ -1031,9 +1042,13 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
         for (int jj = 0; jj < cnt; ++jj) {
             const float pj = ps[jj];
 #pragma unroll
-            for (int e = 0; e < MAXV; ++e) {
-                const int c = lane + e * 32;
-                if (c < A.dv) o[e] = fmaf(pj, to_f<T>(Vs[jj * ldv + c]), o[e]);
+            for (int e = 0; e < MAXV; e += 2) {
+                const int c = 2 * lane + e * 32;
+                if (c < A.dv) {               // an odd last column's neighbour is padding and is not stored
+                    const float2 v = load_pair(Vs + jj * ldv + c);
+                    o[e] = fmaf(pj, v.x, o[e]);
+                    o[e + 1] = fmaf(pj, v.y, o[e + 1]);
+                }
             }
         }
         __syncwarp();
@@ -1043,60 +1058,84 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
     if (lane == 0) { dst[0] = m; dst[1] = l; }
 #pragma unroll
     for (int e = 0; e < MAXV; ++e) {
-        const int c = lane + e * 32;
+        const int c = 2 * lane + e / 2 * 64 + e % 2;
         if (c < A.dv) dst[2 + c] = o[e];
     }
 }
 
-// One warp per (row, query head): merges the ranges of every map and joins the maps; the sink enters here, once, with no value.
+// One block per (row, query head): merges the ranges of every map and joins the maps; the sink enters here, once, with no value.
+// The ranges are dealt out to the block's warps (those of a map in turn), so that a row with many of them waits for global memory a
+// few times only; the warps' shares are added in warp order.
+constexpr int kMergeWarps = 8;
 template <class T, int MAXV, int MAPS>
-__global__ void __launch_bounds__(128) attn_merge_kernel(const AttnArgs A, T* __restrict__ out) {
-    const int lane = threadIdx.x & 31;
-    const int unit = blockIdx.x * 4 + (threadIdx.x >> 5);
-    if (unit >= A.short_rows * A.H) return;
-    const int x = unit / A.H, h = unit % A.H;
+__global__ void __launch_bounds__(kMergeWarps * 32) attn_merge_kernel(const AttnArgs A, T* __restrict__ out) {
+    extern __shared__ float share[];                    // [kMergeWarps][dv], then [kMergeWarps] denominators
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int x = blockIdx.x / A.H, h = blockIdx.x % A.H;
     const int s = x / kShortSeq, r = x % kShortSeq;
     const int t0 = A.seq_start[s], n = A.seq_start[s + 1] - t0;
     if (n > kShortSeq || r >= n) return;
     const int t = t0 + r, pos = A.tok_pos[t];
     const int ns = pos / A.split_len - attn_first_key(A, pos) / A.split_len + 1;
+    constexpr int PER = kMergeWarps / MAPS;             // warps per map
+    const int map = warp / PER, w0 = warp % PER;
+    const float* src = A.part + (((size_t)x * A.H + h) * MAPS + map) * A.n_splits * (A.dv + 2);
     const float sink = A.sink ? A.sink[h] : -INFINITY;
-    float sum[MAXV];                    // the maps' joined result
+    float M = sink;
+    for (int z = lane; z < ns; z += 32) M = fmaxf(M, src[(size_t)z * (A.dv + 2)]);
+    M = warp_max(M);
+    float l = 0.0f;
+    float o[MAXV];
 #pragma unroll
-    for (int map = 0; map < MAPS; ++map) {
-        const float* src = A.part + (((size_t)x * A.H + h) * MAPS + map) * A.n_splits * (A.dv + 2);
-        // lanes take the ranges' maxima and weights side by side; the value columns are then summed range by range with the
-        // weights handed on by shuffles, so that no load waits for an earlier one
-        float M = sink;
-        for (int z = lane; z < ns; z += 32) M = fmaxf(M, src[(size_t)z * (A.dv + 2)]);
-        M = warp_max(M);
-        float l = 0.0f;
-        float o[MAXV];
-#pragma unroll
-        for (int e = 0; e < MAXV; ++e) o[e] = 0.0f;
-        for (int z0 = 0; z0 < ns; z0 += 32) {
-            const int z = z0 + lane, cnt = min(32, ns - z0);
-            float wz = 0.0f;
-            if (z < ns) {
-                const float* p = src + (size_t)z * (A.dv + 2);
-                wz = expf(p[0] - M);
-                l = fmaf(p[1], wz, l);
-            }
+    for (int e = 0; e < MAXV; ++e) o[e] = 0.0f;
+    // lane i holds the weight of this warp's range number i
+    for (int z0 = w0; z0 < ns; z0 += 32 * PER) {
+        const int z = z0 + lane * PER, cnt = min(32, (ns - z0 + PER - 1) / PER);
+        float wz = 0.0f;
+        if (z < ns) {
+            const float* p = src + (size_t)z * (A.dv + 2);
+            wz = expf(p[0] - M);
+            l = fmaf(p[1], wz, l);
+        }
 #pragma unroll 4
-            for (int i = 0; i < cnt; ++i) {
-                const float w = __shfl_sync(0xffffffffu, wz, i);
-                const float* p = src + (size_t)(z0 + i) * (A.dv + 2) + 2;
+        for (int i = 0; i < cnt; ++i) {
+            const float w = __shfl_sync(0xffffffffu, wz, i);
+            const float* p = src + (size_t)(z0 + i * PER) * (A.dv + 2) + 2;
 #pragma unroll
-                for (int e = 0; e < MAXV; ++e) {
-                    const int c = lane + e * 32;
-                    if (c < A.dv) o[e] = fmaf(p[c], w, o[e]);
-                }
+            for (int e = 0; e < MAXV; ++e) {
+                const int c = lane + e * 32;
+                if (c < A.dv) o[e] = fmaf(p[c], w, o[e]);
             }
         }
-        l = warp_sum(l) + expf(sink - M);
-        const float inv = 1.0f / l;
+    }
+    l = warp_sum(l);
+    if (lane == 0) share[kMergeWarps * A.dv + warp] = l + (w0 == 0 ? expf(sink - M) : 0.0f);
 #pragma unroll
-        for (int e = 0; e < MAXV; ++e) sum[e] = map == 0 ? o[e] * inv : fmaf(-A.diff_lambda, o[e] * inv, sum[e]);
+    for (int e = 0; e < MAXV; ++e) {
+        const int c = lane + e * 32;
+        if (c < A.dv) share[warp * A.dv + c] = o[e];
+    }
+    __syncthreads();
+    if (warp > 0) return;
+    float sum[MAXV];                    // the maps' joined result
+#pragma unroll
+    for (int e = 0; e < MAXV; ++e) sum[e] = 0.0f;
+#pragma unroll
+    for (int mp = 0; mp < MAPS; ++mp) {
+        float den = 0.0f;
+#pragma unroll
+        for (int w = 0; w < PER; ++w) den += share[kMergeWarps * A.dv + mp * PER + w];
+        const float inv = (mp == 0 ? 1.0f : -A.diff_lambda) / den;
+#pragma unroll
+        for (int e = 0; e < MAXV; ++e) {
+            const int c = lane + e * 32;
+            if (c < A.dv) {
+                float v = 0.0f;
+#pragma unroll
+                for (int w = 0; w < PER; ++w) v += share[(mp * PER + w) * A.dv + c];
+                sum[e] = fmaf(v, inv, sum[e]);
+            }
+        }
     }
     attn_finish<T, MAXV, MAPS>(A, t, h, lane, sum, out);
 }
@@ -1636,6 +1675,8 @@ struct SmolLm {
     std::vector<RunInfo> side_runs;       // the cache / state placement of a run's side mixer
     size_t o_conv = 0, o_head = 0;        // state-space: convolved channels [T][channels], per-head decay and step [2][T][heads]
     int max_conv = 0, max_ssd_heads = 0;
+    size_t o_pairs = 0;                   // four-token scan: products between a group's queries and keys
+    int max_pair_heads = 0;
     SmolLmGlobals g{};
     size_t page_elems = 0, slot_floats = 0, esize = 2;
     int max_in = 0, max_mix = 0, max_ff = 0, max_hd = 0, max_q = 0;
@@ -1778,7 +1819,7 @@ extern "C" int smol_lm_create(const SmolLmConfig* cfg, const SmolLmLayer* layers
             if (L.rot_dims < 0 || L.rot_dims > L.dim || L.rot_dims % 2) return fail(SMOL_ERR_INVALID, "attention: rot_dims even and at most dim");
             if (L.rot_dims > 0 && (!L.norm_whole || L.rot_dims > 2 * kMaxRotPairs)) return fail(SMOL_ERR_UNSUPPORTED, "attention: rotation needs norm_whole and at most 512 coordinates");
             const size_t split_smem = ((size_t)std::min(L.heads / L.kv_heads * maps, 8) * (L.dim + 32) * 4 + 15) / 16 * 16 +
-                                      (size_t)32 * (maps * (L.dim + 16 / m->esize) + L.vdim + 16 / m->esize) * m->esize;
+                                      (size_t)32 * (maps * (L.dim + 16 / m->esize + 1) + L.vdim + 16 / m->esize + 1) * m->esize;
             if (split_smem > (size_t)kAttnSplitSmemMax) return fail(SMOL_ERR_UNSUPPORTED, "attention: key and value sizes need more shared memory than an SM has");
             if (L.kv_from > 0) {
                 // another layer's cache, as its latest run leaves it
@@ -1815,7 +1856,8 @@ extern "C" int smol_lm_create(const SmolLmConfig* cfg, const SmolLmLayer* layers
             m->max_hd = std::max(m->max_hd, L.heads * L.vdim);
             m->max_mix = std::max(m->max_mix, L.heads * L.vdim);
             m->max_conv = std::max(m->max_conv, ch);
-            m->max_ssd_heads = std::max(m->max_ssd_heads, (2 * L.heads + L.kv_heads + 1) / 2);        // decay, step, k.q
+            m->max_ssd_heads = std::max(m->max_ssd_heads, L.heads);        // decay and step
+            m->max_pair_heads = std::max(m->max_pair_heads, L.kv_heads);
         } else if (L.mixer == SMOL_LM_MIX_MLSTM) {
             if (L.dim > 256) return fail(SMOL_ERR_UNSUPPORTED, "recurrent mixer: key size above 256");
             if (L.vdim < 1 || !(L.gate_cap > 0.0f) || !L.rate_bias || !L.decay_bias || !L.out_norm)
@@ -1830,7 +1872,8 @@ extern "C" int smol_lm_create(const SmolLmConfig* cfg, const SmolLmLayer* layers
             m->max_hd = std::max(m->max_hd, L.heads * L.vdim);
             m->max_mix = std::max(m->max_mix, L.heads * L.vdim);
             m->max_conv = std::max(m->max_conv, 1);
-            m->max_ssd_heads = std::max(m->max_ssd_heads, 2 * L.heads);        // decay, write weight, floor, key sum . query
+            m->max_ssd_heads = std::max(m->max_ssd_heads, 2 * L.heads);        // decay and write weight, floor, key sum . query
+            m->max_pair_heads = std::max(m->max_pair_heads, L.heads);
         } else if (L.mixer == SMOL_LM_MIX_STATE_SPACE) {
             if (L.vdim < 1 || L.n_state < 1 || L.bc_groups < 1 || L.heads % L.bc_groups != 0 || L.conv_taps < 1 || L.norm_parts < 1 ||
                 (L.heads * L.vdim) % L.norm_parts != 0)
@@ -2032,6 +2075,7 @@ extern "C" int smol_lm_create(const SmolLmConfig* cfg, const SmolLmLayer* layers
         m->o_conv = carve(T * (size_t)m->max_conv * 4);
         m->o_head = carve(2 * T * (size_t)m->max_ssd_heads * 4);
     }
+    if (m->max_pair_heads > 0) m->o_pairs = carve(T * (size_t)m->max_pair_heads * kPairFloats * 4);
     if (m->max_top > 0) {
         const size_t pairs = T * (size_t)m->max_top;
         m->o_sel_id = carve(pairs * 4);
@@ -2070,7 +2114,8 @@ template <int DK>
 static cudaError_t scan_attribute() {
     cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(2 * delta_buf_floats(DK) * sizeof(float)));
     if (e == cudaSuccess) e = cudaFuncSetAttribute(gla_scan_kernel<DK, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, std::max(kScanSpread, (int)(2 * gla_buf_floats(DK) * sizeof(float))));
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(gated_delta_scan_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, std::max(kScanSpread, (int)(2 * gated_delta_buf_floats(DK) * sizeof(float))));
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(group_scan_kernel<DK, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, std::max(kScanSpread, (int)(2 * group_scan_buf_floats(DK) * sizeof(float))));
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(group_scan_kernel<DK, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, std::max(kScanSpread, (int)(2 * group_scan_buf_floats(DK) * sizeof(float))));
     if (e == cudaSuccess) e = cudaFuncSetAttribute(gla_scan_kernel<DK, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, std::max(kScanSpread, (int)(2 * gla_buf_floats(DK) * sizeof(float))));
     return e;
 }
@@ -2287,7 +2332,7 @@ static cudaError_t launch_scan(const DeltaArgs& A, int n_seqs, const float* dec,
 template <int DK>
 static cudaError_t launch_gla_scan(const GlaArgs& A, int n_seqs, const float* dec, float* pool, float* o_raw, cudaStream_t st, size_t min_smem) {
     constexpr int CB = gla_block_cols(DK), threads = CB * gla_lanes(DK);
-    const int groups = (A.dv + (A.unit_out ? 1 : 0) + CB - 1) / CB;
+    const int groups = (A.dv + CB - 1) / CB;
     const size_t smem = std::max(2 * gla_buf_floats(DK) * sizeof(float), min_smem);
     if (A.head_decay) gla_scan_kernel<DK, true><<<n_seqs * A.H * groups, threads, smem, st>>>(A, dec, pool, o_raw);
     else gla_scan_kernel<DK, false><<<n_seqs * A.H * groups, threads, smem, st>>>(A, dec, pool, o_raw);
@@ -2303,12 +2348,27 @@ static cudaError_t launch_gla_scan_any(const GlaArgs& A, int n_seqs, const float
     return launch_gla_scan<256>(A, n_seqs, dec, pool, o_raw, st, min_smem);
 }
 
-template <int DK>
-static cudaError_t launch_gated_delta(const GatedDeltaArgs& A, int n_seqs, const float* qkv, const float* head, float* pool, float* o_raw, cudaStream_t st) {
+template <int DK, bool DELTA>
+static cudaError_t launch_group_scan(const GroupScanArgs& A, int n_seqs, float* pool, float* o_raw, cudaStream_t st, size_t min_smem) {
     constexpr int CB = gla_block_cols(DK), threads = CB * gla_lanes(DK);
-    const int groups = (A.dv + CB - 1) / CB;
-    gated_delta_scan_kernel<DK><<<n_seqs * A.H * groups, threads, 2 * gated_delta_buf_floats(DK) * sizeof(float), st>>>(A, qkv, head, pool, o_raw);
+    const int parts = (A.dv + (A.unit_out ? 1 : 0) + CB - 1) / CB;
+    group_scan_kernel<DK, DELTA><<<n_seqs * A.H * parts, threads, std::max(2 * group_scan_buf_floats(DK) * sizeof(float), min_smem), st>>>(A, pool, o_raw);
     return cudaGetLastError();
+}
+// The four-token scan: the group's products (not needed where every sequence brings one token), then the recurrence itself.
+template <bool DELTA>
+static cudaError_t launch_group_scan_any(SmolLm* m, const GroupScanArgs& A, float* pairs, int n_seqs, int max_n, float* pool, float* o_raw, cudaStream_t st,
+                                         size_t min_smem = 0) {
+    if (max_n > 1) {
+        scan_pairs_kernel<DELTA><<<dim3((max_n + kScanGroup - 1) / kScanGroup, n_seqs, (A.G + 3) / 4), 128, 0, st>>>(A, pairs);
+        m->launches++;
+    }
+    m->launches++;
+    if (A.d <= 16) return launch_group_scan<16, DELTA>(A, n_seqs, pool, o_raw, st, min_smem);
+    if (A.d <= 32) return launch_group_scan<32, DELTA>(A, n_seqs, pool, o_raw, st, min_smem);
+    if (A.d <= 64) return launch_group_scan<64, DELTA>(A, n_seqs, pool, o_raw, st, min_smem);
+    if (A.d <= 128) return launch_group_scan<128, DELTA>(A, n_seqs, pool, o_raw, st, min_smem);
+    return launch_group_scan<256, DELTA>(A, n_seqs, pool, o_raw, st, min_smem);
 }
 
 // The attention kernels over the rows of a step: prompt portions on the tensor-core form (bf16, `flash`) or the
@@ -2359,10 +2419,10 @@ static void launch_attention(SmolLm* m, const SmolLmStep* s, AttnArgs& A, bool f
     if (min_n <= kShortSeq && (flash || max_n <= kShortSeq)) {
         const int Gq = A.H / A.G * MAPS, nwarp = std::min(Gq, 8), groups = (Gq + nwarp - 1) / nwarp;
         const int pad = 16 / (int)sizeof(T);
-        const size_t smem = ((size_t)nwarp * (A.d + 32) * 4 + 15) / 16 * 16 + (size_t)32 * (MAPS * (A.d + pad) + (A.v_in_k ? 0 : A.dv + pad)) * sizeof(T);
+        const size_t smem = ((size_t)nwarp * (A.d + 32) * 4 + 15) / 16 * 16 + (size_t)32 * (MAPS * (A.d + pad + 1) + (A.v_in_k ? 0 : split_value_ld<T>(A.dv))) * sizeof(T);
         dim3 grid(A.short_rows, A.G * groups, A.n_splits);
         attn_split_kernel<T, MAXV><<<grid, nwarp * 32, smem, st>>>(A, qbuf, pool);
-        attn_merge_kernel<T, MAXV, MAPS><<<(A.short_rows * A.H + 3) / 4, 128, 0, st>>>(A, mix);
+        attn_merge_kernel<T, MAXV, MAPS><<<A.short_rows * A.H, kMergeWarps * 32, kMergeWarps * (A.dv + 1) * sizeof(float), st>>>(A, mix);
         m->launches += 2;
     }
 }
@@ -2665,25 +2725,38 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             m->launches += 3;
             return SMOL_OK;
         };
+        // The four-token scan's arguments for a state [dim, vdim] per head in the slot.
+        const int max_n = s->max_seq_tokens > 0 ? s->max_seq_tokens : Tn;
+        float* pairs = reinterpret_cast<float*>(m->ws + m->o_pairs);
+        auto group_args = [&](const SmolLmLayer& M, const RunInfo& Ri, int G) {
+            GroupScanArgs A;
+            A.H = M.heads; A.G = G; A.d = M.dim; A.dv = M.vdim; A.q_scale = 1.0f;
+            A.head = head; A.pairs = pairs;
+            A.seq_start = s->seq_start; A.seq_pos0 = s->seq_pos0; A.seq_slot = s->seq_slot;
+            A.slot_floats = m->slot_floats; A.state_off = Ri.state_off; A.n_slots = m->n_slots; A.err = err;
+            A.unit_out = nullptr; A.unit_off = 0;
+            A.conv = ConvIo{};
+            return A;
+        };
         // Gated delta rule: convolutions, unit vectors, decay and step; the scan over the slot's state; norm per head, silu gate.
         auto gated_delta = [&](const SmolLmLayer& M, const RunInfo& Ri, const float* pj, T* mix_at, int ld) -> int {
-            const int hv = M.heads * M.vdim, ch = 2 * M.kv_heads * M.dim + hv;
+            const int hv = M.heads * M.vdim, gd = M.kv_heads * M.dim, ch = 2 * gd + hv;
             GatedDeltaArgs P;
             P.proj = pj; P.n_in = n_in; P.H = M.heads; P.G = M.kv_heads; P.d = M.dim; P.dv = M.vdim; P.n_tokens = Tn;
             P.q_scale = M.score_scale; P.unit_eps = M.unit_eps; P.a_log = M.a_log; P.dt_bias = M.dt_bias;
-            P.tok_seq = s->tok_seq; P.state_off = Ri.state_off; P.err = err;
+            P.tok_seq = s->tok_seq; P.err = err;
             P.conv = ConvIo{pj, nullptr, n_in, ch, M.conv_taps, M.conv_w, nullptr, s->seq_start, s->seq_pos0, s->seq_slot, m->slot_floats, Ri.conv_off, m->n_slots};
             const int warps = M.kv_heads + (hv + kGatedDeltaCols - 1) / kGatedDeltaCols;
-            gated_delta_prep_kernel<<<dim3(Tn, (warps + 3) / 4), 128, 0, st>>>(P, m->slots, conv, head);
-            if (M.dim <= 16) CU(launch_gated_delta<16>(P, s->n_seqs, conv, head, m->slots, oraw, st));
-            else if (M.dim <= 32) CU(launch_gated_delta<32>(P, s->n_seqs, conv, head, m->slots, oraw, st));
-            else if (M.dim <= 64) CU(launch_gated_delta<64>(P, s->n_seqs, conv, head, m->slots, oraw, st));
-            else if (M.dim <= 128) CU(launch_gated_delta<128>(P, s->n_seqs, conv, head, m->slots, oraw, st));
-            else CU(launch_gated_delta<256>(P, s->n_seqs, conv, head, m->slots, oraw, st));
+            gated_delta_prep_kernel<<<dim3(Tn, (warps + 3) / 4), 128, 0, st>>>(P, m->slots, conv, head, pairs);
+            GroupScanArgs S = group_args(M, Ri, M.kv_heads);
+            S.q_src = conv; S.k_src = conv + gd; S.v_src = conv + 2 * gd;
+            S.q_ld = S.k_ld = S.v_ld = ch;
+            S.conv = P.conv;
+            CU(launch_group_scan_any<true>(m, S, pairs, s->n_seqs, max_n, m->slots, oraw, st));
             GlaArgs A = scan_args(M, Ri, pj);
             A.out_norm = M.out_norm; A.gate_off = ch; A.out_ld = ld; A.out_scale = M.mix_scale;
             gla_out_kernel<T><<<(Tn * M.heads + 3) / 4, 128, 0, st>>>(A, oraw, mix_at);
-            m->launches += 3;
+            m->launches += 2;
             return SMOL_OK;
         };
         // mLSTM: gates and running maximum, the scan with the unit column (the key sum's product with the query), then the
@@ -2691,24 +2764,24 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
         auto mlstm = [&](const SmolLmLayer& M, const RunInfo& Ri, const float* pj, T* mix_at, int ld) -> int {
             const int hd = M.heads * M.dim, hv = M.heads * M.vdim;
             const size_t TH = (size_t)Tn * M.heads;
+            float *floor_at = head + 2 * TH, *den = head + 3 * TH;
             MlstmArgs P;
-            P.proj = pj; P.n_in = n_in; P.H = M.heads; P.n_tokens = Tn; P.gate_off = (size_t)2 * hd + 2 * hv; P.cap = M.gate_cap;
+            P.proj = pj; P.n_in = n_in; P.H = M.heads; P.d = M.dim; P.n_tokens = Tn; P.gate_off = (size_t)2 * hd + 2 * hv; P.cap = M.gate_cap;
             P.i_bias = M.rate_bias; P.f_bias = M.decay_bias;
             P.seq_start = s->seq_start; P.seq_pos0 = s->seq_pos0; P.seq_slot = s->seq_slot;
             P.slot_floats = m->slot_floats; P.m_off = Ri.m_off; P.n_slots = m->n_slots; P.err = err;
-            const int max_n = s->max_seq_tokens > 0 ? s->max_seq_tokens : Tn;
-            mlstm_gate_kernel<<<s->n_seqs * M.heads, std::min(kMlstmTile, (max_n + 31) / 32 * 32), 0, st>>>(P, m->slots, head);
+            mlstm_gate_kernel<<<s->n_seqs * M.heads, std::min(kMlstmTile, (max_n + 31) / 32 * 32), 0, st>>>(P, m->slots, head, floor_at, pairs);
+            GroupScanArgs S = group_args(M, Ri, M.heads);
+            S.q_src = pj; S.k_src = pj + hd; S.v_src = pj + 2 * hd;
+            S.q_ld = S.k_ld = S.v_ld = n_in;
+            S.q_scale = M.score_scale;
+            S.unit_out = den; S.unit_off = Ri.unit_off;
+            CU(launch_group_scan_any<false>(m, S, pairs, s->n_seqs, max_n, m->slots, oraw, st));
             GlaArgs A = scan_args(M, Ri, pj);
-            A.q_src = pj; A.k_src = pj + hd; A.v_src = pj + 2 * hd;
-            A.q_ld = A.k_ld = A.v_ld = n_in;
-            A.q_scale = M.score_scale;
-            A.head_decay = head; A.head_step = head + TH;
-            A.unit_out = head + 3 * TH; A.unit_off = Ri.unit_off;
-            CU(launch_gla_scan_any(A, s->n_seqs, nullptr, m->slots, oraw, st));
-            A.unit_floor = head + 2 * TH; A.den_eps = M.den_eps;
+            A.den = den; A.den_floor = floor_at; A.den_eps = M.den_eps;
             A.out_norm = M.out_norm; A.norm_own = 1; A.gate_sigmoid = 1; A.out_ld = ld; A.out_scale = M.mix_scale;
             gla_out_kernel<T><<<(Tn * M.heads + 3) / 4, 128, 0, st>>>(A, oraw, mix_at);
-            m->launches += 3;
+            m->launches += 2;
             return SMOL_OK;
         };
         auto run_mixer = [&](const SmolLmLayer& M, const RunInfo& Ri, const float* pj, const float* bias, T* mix_at, int ld) -> int {

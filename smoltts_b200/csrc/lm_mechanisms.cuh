@@ -323,15 +323,11 @@ struct GlaArgs {
     int head_ld;
     int out_ld;                                        // row stride of the finished mixer output
     float out_scale;
-    // A further state column per head whose value is 1 for every token (the running sum of the written keys): its rows live at
-    // unit_off inside the slot ([H][d]), its product with the query goes to unit_out[t * H + h].  nullptr: none.
-    float* unit_out = nullptr;
-    size_t unit_off = 0;
     // Back end: where the gate rows start in proj (negative: behind q, k and v), sigmoid or silu, the norm weight shared by the heads
-    // ([dv]) or their own ([H * dv]); with unit_out the head's o is first divided by max(|unit_out|, unit_floor[t * H + h]) + den_eps.
+    // ([dv]) or their own ([H * dv]); with `den` ([T][H]) a head's o is first divided by max(|den|, den_floor) + den_eps.
     long long gate_off = -1;
     int gate_sigmoid = 0, norm_own = 0;
-    const float* unit_floor = nullptr;
+    const float *den = nullptr, *den_floor = nullptr;
     float den_eps = 0.0f;
 };
 __host__ __device__ inline void gla_sources_from_proj(GlaArgs& A) {
@@ -407,11 +403,11 @@ __global__ void __launch_bounds__(gla_block_cols(DK) * gla_lanes(DK)) gla_scan_k
     constexpr int kBuf = gla_buf_floats(DK);
     static_assert(DK % (4 * L) == 0, "every lane owns whole 16-byte pieces");
     extern __shared__ __align__(16) float sh[];
-    const int d = A.d, dv = A.dv, dvs = dv + (SCALAR && A.unit_out ? 1 : 0), NS = (dvs + CB - 1) / CB;      // dvs: state columns
+    const int d = A.d, dv = A.dv, NS = (dv + CB - 1) / CB;
     const int group = blockIdx.x % NS, sh_id = blockIdx.x / NS;
     const int seq = sh_id / A.H, h = sh_id % A.H;
     const int j0 = group * CB;
-    const int nc = max(0, min(CB, dv - j0));
+    const int nc = min(CB, dv - j0);
     const int col = threadIdx.x / L, q = threadIdx.x % L, j = j0 + col;
     const int t0 = A.seq_start[seq], t1 = A.seq_start[seq + 1];
     const int slot = A.seq_slot[seq];
@@ -423,18 +419,11 @@ __global__ void __launch_bounds__(gla_block_cols(DK) * gla_lanes(DK)) gla_scan_k
     const bool vec = (d % 4 == 0) && (dv % 4 == 0) && (A.q_ld % 4 == 0) && (A.k_ld % 4 == 0) && (A.v_ld % 4 == 0) &&
                      ((reinterpret_cast<uintptr_t>(A.q_src) | reinterpret_cast<uintptr_t>(A.k_src) | reinterpret_cast<uintptr_t>(A.v_src)) % 16 == 0);
     for (int i = threadIdx.x; i < 2 * kBuf; i += blockDim.x) sh[i] = 0.0f;      // padded channels and columns stay zero for good
-    if (SCALAR && dvs > dv && dv >= j0 && dv < j0 + CB) {                      // ... and the unit column one
-        __syncthreads();
-        for (int i = threadIdx.x; i < 2 * kDeltaChunk; i += blockDim.x) sh[(i / kDeltaChunk) * kBuf + 3 * PL + (i % kDeltaChunk) * CB + dv - j0] = 1.0f;
-    }
     __syncthreads();
     if (vec) gla_stage<DK, 4, SCALAR>(A, sh, t0, min(kDeltaChunk, t1 - t0), h, j0, nc, decay);
     else gla_stage<DK, 1, SCALAR>(A, sh, t0, min(kDeltaChunk, t1 - t0), h, j0, nc, decay);
     cp_async_commit();
-    // element i of this thread's column: st[i * st_ld]
-    const bool unit = SCALAR && j == dv && dvs > dv;
-    float* st = state_pool + (size_t)slot * A.slot_floats + (unit ? A.unit_off + (size_t)h * d : A.state_off + (size_t)h * d * dv + j);
-    const int st_ld = unit ? 1 : dv;
+    float* st = state_pool + (size_t)slot * A.slot_floats + A.state_off + (size_t)h * d * dv;
     float S[RV][4];
     const bool fresh = A.seq_pos0[seq] == 0;
 #pragma unroll
@@ -442,7 +431,7 @@ __global__ void __launch_bounds__(gla_block_cols(DK) * gla_lanes(DK)) gla_scan_k
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
             const int i = 4 * (e * L + q) + x;
-            S[e][x] = (!fresh && i < d && j < dvs) ? st[(size_t)i * st_ld] : 0.0f;
+            S[e][x] = (!fresh && i < d && j < dv) ? st[(size_t)i * dv + j] : 0.0f;
         }
     int cur = 0;
     for (int c0 = t0; c0 < t1; c0 += kDeltaChunk, cur ^= 1) {
@@ -491,12 +480,10 @@ __global__ void __launch_bounds__(gla_block_cols(DK) * gla_lanes(DK)) gla_scan_k
             for (int s = 1; s < L; s <<= 1)
 #pragma unroll
                 for (int u = 0; u < 4; ++u) po[u] += __shfl_xor_sync(0xffffffffu, po[u], s);
-            if (q == 0 && j < dvs) {
-                float* dst = unit ? A.unit_out + (size_t)(c0 + tt) * A.H + h : o_raw + (size_t)(c0 + tt) * A.H * dv + h * dv + j;
-                const int ld = unit ? A.H : A.H * dv;
+            if (q == 0 && j < dv) {
 #pragma unroll
                 for (int u = 0; u < 4; ++u)
-                    if (FULL || tt + u < n) dst[(size_t)u * ld] = po[u] * A.q_scale;
+                    if (FULL || tt + u < n) o_raw[(size_t)(c0 + tt + u) * A.H * dv + h * dv + j] = po[u] * A.q_scale;
             }
         };
         if (n == kDeltaChunk) {
@@ -512,11 +499,11 @@ __global__ void __launch_bounds__(gla_block_cols(DK) * gla_lanes(DK)) gla_scan_k
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
             const int i = 4 * (e * L + q) + x;
-            if (i < d && j < dvs) st[(size_t)i * st_ld] = S[e][x];
+            if (i < d && j < dv) st[(size_t)i * dv + j] = S[e][x];
         }
 }
 
-// End of the mixer: each head's o (divided by its unit column's product first, where there is one) divided by its root mean square
+// End of the mixer: each head's o (divided by its denominator first, where there is one) divided by its root mean square
 // over dv, times the plain weight (shared by the heads or their own; nullptr: none), times silu or sigmoid of the gate, written in
 // T.  One warp per (token, head).
 template <class T>
@@ -529,7 +516,7 @@ __global__ void gla_out_kernel(const GlaArgs A, const float* __restrict__ o_raw,
     const float* gate = A.proj + (size_t)t * A.n_in + (A.gate_off >= 0 ? (size_t)A.gate_off : (size_t)2 * A.H * A.d + HV) + h * dv;
     const float* weight = A.out_norm ? A.out_norm + (A.norm_own ? h * dv : 0) : nullptr;
     float inv = 1.0f;
-    if (A.unit_out) inv = 1.0f / (fmaxf(fabsf(A.unit_out[(size_t)t * A.H + h]), A.unit_floor[(size_t)t * A.H + h]) + A.den_eps);
+    if (A.den) inv = 1.0f / (fmaxf(fabsf(A.den[(size_t)t * A.H + h]), A.den_floor[(size_t)t * A.H + h]) + A.den_eps);
     auto finish = [&](float v, float rs, float w, float g) { return from_f<T>(v * rs * w * (A.gate_sigmoid ? sigmoidf_(g) : silu_(g)) * A.out_scale); };
     constexpr int R = 4;                 // up to 128 columns in registers: every load goes out before the reduction
     if (dv <= 32 * R) {
