@@ -924,6 +924,7 @@ template <class T> __device__ __forceinline__ float key_dot(const float* qs, con
 template <> __device__ __forceinline__ float key_dot<float>(const float* qs, const float* k, int d) {
     float a0 = 0.0f, a1 = 0.0f, a2 = 0.0f, a3 = 0.0f;
     if (d % 4 == 0 && (reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(qs)) % 16 == 0) {
+#pragma unroll 4
         for (int c = 0; c < d; c += 4) {
             const float4 v = *reinterpret_cast<const float4*>(k + c), x = *reinterpret_cast<const float4*>(qs + c);
             a0 = fmaf(x.x, v.x, a0); a1 = fmaf(x.y, v.y, a1); a2 = fmaf(x.z, v.z, a2); a3 = fmaf(x.w, v.w, a3);
@@ -936,6 +937,7 @@ template <> __device__ __forceinline__ float key_dot<float>(const float* qs, con
 template <> __device__ __forceinline__ float key_dot<bf16>(const float* qs, const bf16* k, int d) {
     float a0 = 0.0f, a1 = 0.0f, a2 = 0.0f, a3 = 0.0f;
     if (d % 8 == 0 && (reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(qs)) % 16 == 0) {
+#pragma unroll 4
         for (int c = 0; c < d; c += 8) {
             const uint4 v = *reinterpret_cast<const uint4*>(k + c);
             const float4 x = *reinterpret_cast<const float4*>(qs + c), y = *reinterpret_cast<const float4*>(qs + c + 4);
@@ -959,14 +961,14 @@ __device__ __forceinline__ float2 load_pair(const bf16* p) {
 // row stride of the staged values: an even number of elements
 template <class T> __host__ __device__ constexpr int split_value_ld(int dv) { return (dv + 16 / (int)sizeof(T) + 1) / 2 * 2; }
 
-template <class T, int MAXV>
+template <class T, int MAXV, int KPL>
 __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const T* __restrict__ qbuf, const T* __restrict__ pool) {
     // One block per (row, key/value head x group of up to 8 of its query rows, key range); one warp per query row (a query
     // head, or one of its maps: the block then stages every map's keys beside the values they share).
-    // 32 keys and values at a time are staged in shared memory (rows padded by 16 bytes: conflict-free row-per-lane
-    // reads), so that no global load sits inside the softmax / value loops.
+    // 32 * KPL keys and values at a time (KPL keys per lane) are staged in shared memory (rows padded by 16 bytes: conflict-free
+    // row-per-lane reads), so that no global load sits inside the softmax / value loops.
     extern __shared__ __align__(16) unsigned char sm_raw[];
-    constexpr int kPad = 16 / (int)sizeof(T);
+    constexpr int kPad = 16 / (int)sizeof(T), KEYS = 32 * KPL;
     const int s = blockIdx.x / kShortSeq, r = blockIdx.x % kShortSeq;
     const int t0 = A.seq_start[s], n = A.seq_start[s + 1] - t0;
     if (n > kShortSeq || r >= n) return;
@@ -985,9 +987,9 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
     const int h = g * Gq + (active ? hq : 0), map = h % A.maps, head = h / A.maps;      // h: query row
     const int ldk = A.v_in_k ? (A.d + kPad + 1) / 2 * 2 : A.d + kPad, ldv = A.v_in_k ? ldk : split_value_ld<T>(A.dv);
     float* qs = reinterpret_cast<float*>(sm_raw) + warp * A.d;
-    float* ps = reinterpret_cast<float*>(sm_raw) + nwarp * A.d + warp * 32;
-    T* Ks = reinterpret_cast<T*>(sm_raw + (((size_t)nwarp * (A.d + 32) * 4 + 15) / 16) * 16);
-    T* Vs = A.v_in_k ? Ks : Ks + 32 * ldk * A.maps;
+    float* ps = reinterpret_cast<float*>(sm_raw) + nwarp * A.d + warp * KEYS;
+    T* Ks = reinterpret_cast<T*>(sm_raw + (((size_t)nwarp * (A.d + KEYS) * 4 + 15) / 16) * 16);
+    T* Vs = A.v_in_k ? Ks : Ks + KEYS * ldk * A.maps;
     const int32_t* bt = A.block_table + (size_t)s * A.max_pages;
     for (int c = lane; c < A.d; c += 32) qs[c] = to_f<T>(qbuf[((size_t)t * A.H * A.maps + h) * A.d + c]);
     const float r1 = A.r1 ? A.r1[head] : 0.0f, r2 = A.r1 ? A.r2[head] : 0.0f, slope = A.slope ? A.slope[head] : 0.0f;
@@ -999,47 +1001,62 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
     const bool kvec = (A.d * sizeof(T)) % 16 == 0 && (A.k_ld * sizeof(T)) % 16 == 0 && (A.k_off * sizeof(T)) % 16 == 0;
     const bool vvec = (A.dv * sizeof(T)) % 16 == 0 && (A.v_ld * sizeof(T)) % 16 == 0 && (A.v_off * sizeof(T)) % 16 == 0;
     const int kchunk1 = kvec ? A.d / kPad : A.d, kchunks = kchunk1 * A.maps, vchunks = A.v_in_k ? 0 : (vvec ? A.dv / kPad : A.dv);
-    for (int j0 = j_lo; j0 <= j_hi; j0 += 32) {
-        const int cnt = min(32, j_hi - j0 + 1);
+    for (int j0 = j_lo; j0 <= j_hi; j0 += KEYS) {
+        const int cnt = min(KEYS, j_hi - j0 + 1);
         __syncthreads();
-        // a warp per cached row, its lanes side by side over the row's pieces
-        for (int row = warp; row < cnt; row += nwarp) {
-            const int jr = j0 + row, pg = jr / A.page_size, in_pg = jr - pg * A.page_size;
-            const T* base = pool + (size_t)bt[pg] * A.page_elems;
-            for (int c = lane; c < kchunks + vchunks; c += 32) {
-                if (c < kchunks) {
-                    const int km = A.maps > 1 ? c / kchunk1 : 0, ck = c - km * kchunk1;
-                    const T* src = base + A.k_off + ((size_t)(g * A.maps + km) * A.page_size + in_pg) * A.k_ld;
-                    T* dst = Ks + (km * 32 + row) * ldk;
-                    if (kvec) cp_async16(dst + ck * kPad, src + ck * kPad);
-                    else dst[ck] = src[ck];
-                } else {
-                    const int cv = c - kchunks;
-                    const T* src = base + A.v_off + ((size_t)g * A.page_size + in_pg) * A.v_ld;
-                    if (vvec) cp_async16(Vs + row * ldv + cv * kPad, src + cv * kPad);
-                    else Vs[row * ldv + cv] = src[cv];
+        // Where the round's rows are cached: lane r looks rows r, r + 32 up.  Then a warp per row, its lanes side by side over the
+        // row's pieces (a lane keeps its piece over the rows, so that nothing is divided inside the loop).
+        int page[KPL], place[KPL];
+#pragma unroll
+        for (int x = 0; x < KPL; ++x) {
+            const int jr = min(j0 + lane + 32 * x, j_hi), pg = jr / A.page_size;
+            place[x] = jr - pg * A.page_size;
+            page[x] = bt[pg];
+        }
+        for (int c = lane; c - lane < kchunks + vchunks; c += 32) {
+            const bool key = c < kchunks, mine = c < kchunks + vchunks;
+            const int km = key && A.maps > 1 ? c / kchunk1 : 0, piece = key ? c - km * kchunk1 : c - kchunks;
+            const int step = (key ? kvec : vvec) ? kPad : 1, ld = key ? A.k_ld : A.v_ld;
+            const T* src0 = pool + (key ? A.k_off + (size_t)(g * A.maps + km) * A.page_size * ld : A.v_off + (size_t)g * A.page_size * ld) + piece * step;
+            T* dst0 = (key ? Ks + km * KEYS * ldk : Vs) + piece * step;
+            const int dst_ld = key ? ldk : ldv;
+#pragma unroll
+            for (int x = 0; x < KPL; ++x)
+#pragma unroll 4
+                for (int r = warp; r < min(32, cnt - 32 * x); r += nwarp) {
+                    const int pg = __shfl_sync(0xffffffffu, page[x], r), in_pg = __shfl_sync(0xffffffffu, place[x], r);
+                    const T* src = src0 + (size_t)pg * A.page_elems + (size_t)in_pg * ld;
+                    T* dst = dst0 + (r + 32 * x) * dst_ld;
+                    if (!mine) continue;
+                    if (step == kPad) cp_async16(dst, src);
+                    else *dst = *src;
                 }
-            }
         }
         cp_async_commit_group();
         cp_async_wait_group<0>();
         __syncthreads();
         if (!active) continue;
-        const int j = j0 + lane;
-        float sc = -INFINITY;
-        if (lane < cnt) {
-            sc = attn_score<false>(A, key_dot<T>(qs, Ks + (map * 32 + lane) * ldk, A.d), pos - j, r1, r2, slope);
+        float sc[KPL], mx = -INFINITY, pl = 0.0f;
+#pragma unroll
+        for (int x = 0; x < KPL; ++x) {
+            const int row = lane + 32 * x;
+            sc[x] = row < cnt ? attn_score<false>(A, key_dot<T>(qs, Ks + (map * KEYS + row) * ldk, A.d), pos - (j0 + row), r1, r2, slope) : -INFINITY;
+            mx = fmaxf(mx, sc[x]);
         }
-        const float mn = fmaxf(m, warp_max(sc));          // finite: lane 0 of every round holds a valid key
-        const float p = lane < cnt ? expf(sc - mn) : 0.0f;
+        const float mn = fmaxf(m, warp_max(mx));          // finite: lane 0 of every round holds a valid key
         const float corr = expf(m - mn);
-        l = l * corr + warp_sum(p);
+#pragma unroll
+        for (int x = 0; x < KPL; ++x) {
+            const float p = lane + 32 * x < cnt ? expf(sc[x] - mn) : 0.0f;
+            ps[lane + 32 * x] = p;
+            pl += p;
+        }
+        l = l * corr + warp_sum(pl);
         m = mn;
-        ps[lane] = p;
         __syncwarp();
 #pragma unroll
         for (int e = 0; e < MAXV; ++e) o[e] *= corr;
-        for (int jj = 0; jj < cnt; ++jj) {
+        auto add_value = [&](int jj) {
             const float pj = ps[jj];
 #pragma unroll
             for (int e = 0; e < MAXV; e += 2) {
@@ -1050,7 +1067,13 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
                     o[e + 1] = fmaf(pj, v.y, o[e + 1]);
                 }
             }
+        };
+        int jj = 0;
+        for (; jj + 8 <= cnt; jj += 8) {
+#pragma unroll
+            for (int x = 0; x < 8; ++x) add_value(jj + x);      // the next keys' loads go out under the current products
         }
+        for (; jj < cnt; ++jj) add_value(jj);
         __syncwarp();
     }
     if (!active) return;
@@ -1237,11 +1260,17 @@ __global__ void __launch_bounds__(128 * MAPS) attn_flash_kernel(const AttnArgs A
     for (int nt = 0; nt < DV / 8; ++nt)
 #pragma unroll
         for (int e = 0; e < 4; ++e) o[nt][e] = 0.0f;
+    const bool one_page = A.page_size % 64 == 0;
     // the next tile of keys and values is on its way (cp.async) while the current one is multiplied
     auto stage_tile = [&](int j0, int buf) {
+        // a tile within one page is looked up once, else every row for itself
+        const int pg0 = j0 / A.page_size;
+        const bf16* base0 = pool + (size_t)bt[pg0] * A.page_elems;
+        const int in0 = j0 - pg0 * A.page_size;
         auto row_of = [&](int row, size_t off, int width, int in_head) -> const bf16* {
             const int j = j0 + row;
             if (j > last_pos) return nullptr;
+            if (one_page) return base0 + off + ((size_t)in_head * A.page_size + in0 + row) * width;
             return pool + (size_t)bt[j / A.page_size] * A.page_elems + off + ((size_t)in_head * A.page_size + j % A.page_size) * width;
         };
 #pragma unroll
@@ -1717,6 +1746,7 @@ struct SmolLm {
 };
 
 constexpr int kAttnSplitSmemMax = 200 * 1024;      // shared memory the few-token attention may ask for
+constexpr int kAttnSplitWideSmem = 64 * 1024;      // ... and up to which it takes 64 keys at a time instead of 32
 
 static size_t al256(size_t v) { return (v + 255) / 256 * 256; }
 
@@ -2135,8 +2165,9 @@ static cudaError_t set_kernel_attributes() {
     if (e == cudaSuccess) e = scan_attribute<64>();
     if (e == cudaSuccess) e = scan_attribute<128>();
     if (e == cudaSuccess) e = scan_attribute<256>();
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_split_kernel<T, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, kAttnSplitSmemMax);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_split_kernel<T, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, kAttnSplitSmemMax);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_split_kernel<T, 8, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kAttnSplitSmemMax);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_split_kernel<T, 8, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, kAttnSplitWideSmem);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(attn_split_kernel<T, 16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kAttnSplitSmemMax);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(sigmoid_attn_kernel<T, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(sigmoid_attn_kernel<T, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(sigmoid_split_kernel<T, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSigmoidSmemMax);
@@ -2419,9 +2450,16 @@ static void launch_attention(SmolLm* m, const SmolLmStep* s, AttnArgs& A, bool f
     if (min_n <= kShortSeq && (flash || max_n <= kShortSeq)) {
         const int Gq = A.H / A.G * MAPS, nwarp = std::min(Gq, 8), groups = (Gq + nwarp - 1) / nwarp;
         const int pad = 16 / (int)sizeof(T);
-        const size_t smem = ((size_t)nwarp * (A.d + 32) * 4 + 15) / 16 * 16 + (size_t)32 * (MAPS * (A.d + pad + 1) + (A.v_in_k ? 0 : split_value_ld<T>(A.dv))) * sizeof(T);
+        auto smem_of = [&](int keys) {
+            return ((size_t)nwarp * (A.d + keys) * 4 + 15) / 16 * 16 + (size_t)keys * (MAPS * (A.d + pad + 1) + (A.v_in_k ? 0 : split_value_ld<T>(A.dv))) * sizeof(T);
+        };
         dim3 grid(A.short_rows, A.G * groups, A.n_splits);
-        attn_split_kernel<T, MAXV><<<grid, nwarp * 32, smem, st>>>(A, qbuf, pool);
+        bool wide = false;
+        if constexpr (MAXV == 8) {
+            wide = smem_of(64) <= (size_t)kAttnSplitWideSmem;
+            if (wide) attn_split_kernel<T, MAXV, 2><<<grid, nwarp * 32, smem_of(64), st>>>(A, qbuf, pool);
+        }
+        if (!wide) attn_split_kernel<T, MAXV, 1><<<grid, nwarp * 32, smem_of(32), st>>>(A, qbuf, pool);
         attn_merge_kernel<T, MAXV, MAPS><<<A.short_rows * A.H, kMergeWarps * 32, kMergeWarps * (A.dv + 1) * sizeof(float), st>>>(A, mix);
         m->launches += 2;
     }
