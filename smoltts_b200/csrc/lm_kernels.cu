@@ -1089,10 +1089,11 @@ __global__ void __launch_bounds__(256) attn_split_kernel(const AttnArgs A, const
 // One block per (row, query head): merges the ranges of every map and joins the maps; the sink enters here, once, with no value.
 // The ranges are dealt out to the block's warps (those of a map in turn), so that a row with many of them waits for global memory a
 // few times only; the warps' shares are added in warp order.
-constexpr int kMergeWarps = 8;
+constexpr int kMergeWarps = 8;      // per map
 template <class T, int MAXV, int MAPS>
-__global__ void __launch_bounds__(kMergeWarps * 32) attn_merge_kernel(const AttnArgs A, T* __restrict__ out) {
-    extern __shared__ float share[];                    // [kMergeWarps][dv], then [kMergeWarps] denominators
+__global__ void __launch_bounds__(kMergeWarps * MAPS * 32) attn_merge_kernel(const AttnArgs A, T* __restrict__ out) {
+    constexpr int PER = kMergeWarps, ALL = PER * MAPS;   // warps per map, of the block
+    extern __shared__ float share[];                    // [ALL][dv], then [ALL] denominators
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int x = blockIdx.x / A.H, h = blockIdx.x % A.H;
     const int s = x / kShortSeq, r = x % kShortSeq;
@@ -1100,7 +1101,6 @@ __global__ void __launch_bounds__(kMergeWarps * 32) attn_merge_kernel(const Attn
     if (n > kShortSeq || r >= n) return;
     const int t = t0 + r, pos = A.tok_pos[t];
     const int ns = pos / A.split_len - attn_first_key(A, pos) / A.split_len + 1;
-    constexpr int PER = kMergeWarps / MAPS;             // warps per map
     const int map = warp / PER, w0 = warp % PER;
     const float* src = A.part + (((size_t)x * A.H + h) * MAPS + map) * A.n_splits * (A.dv + 2);
     const float sink = A.sink ? A.sink[h] : -INFINITY;
@@ -1132,7 +1132,7 @@ __global__ void __launch_bounds__(kMergeWarps * 32) attn_merge_kernel(const Attn
         }
     }
     l = warp_sum(l);
-    if (lane == 0) share[kMergeWarps * A.dv + warp] = l + (w0 == 0 ? expf(sink - M) : 0.0f);
+    if (lane == 0) share[ALL * A.dv + warp] = l + (w0 == 0 ? expf(sink - M) : 0.0f);
 #pragma unroll
     for (int e = 0; e < MAXV; ++e) {
         const int c = lane + e * 32;
@@ -1147,7 +1147,7 @@ __global__ void __launch_bounds__(kMergeWarps * 32) attn_merge_kernel(const Attn
     for (int mp = 0; mp < MAPS; ++mp) {
         float den = 0.0f;
 #pragma unroll
-        for (int w = 0; w < PER; ++w) den += share[kMergeWarps * A.dv + mp * PER + w];
+        for (int w = 0; w < PER; ++w) den += share[ALL * A.dv + mp * PER + w];
         const float inv = (mp == 0 ? 1.0f : -A.diff_lambda) / den;
 #pragma unroll
         for (int e = 0; e < MAXV; ++e) {
@@ -1174,7 +1174,21 @@ __device__ __forceinline__ void ldmatrix_x2_trans(uint32_t& r0, uint32_t& r1, co
     const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
     asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(a));
 }
-
+// four 8 x 8 blocks at once (lane l gives the address of row l % 8 of block l / 8)
+__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* p) {
+    const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], const void* p) {
+    const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
+}
+// 2^x by the hardware instruction (relative error about 2^-22)
+__device__ __forceinline__ float exp2_fast(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 
 // 64 rows of `cols` bf16 into a [64][DP + 8] tile; src(row) is the row's address or nullptr (zero row).  ASYNC: whole
 // 16-byte pieces of aligned rows go by cp.async (the caller commits and waits); everything else is stored directly.
@@ -1261,6 +1275,8 @@ __global__ void __launch_bounds__(128 * MAPS) attn_flash_kernel(const AttnArgs A
 #pragma unroll
         for (int e = 0; e < 4; ++e) o[nt][e] = 0.0f;
     const bool one_page = A.page_size % 64 == 0;
+    // the score is the scaled product alone
+    const bool plain = !penalty && !A.slope && A.softcap == 0.0f && A.window == 0 && A.scale > 0.0f;
     // the next tile of keys and values is on its way (cp.async) while the current one is multiplied
     auto stage_tile = [&](int j0, int buf) {
         // a tile within one page is looked up once, else every row for itself
@@ -1300,55 +1316,77 @@ __global__ void __launch_bounds__(128 * MAPS) attn_flash_kernel(const AttnArgs A
 #pragma unroll
             for (int kk = 0; kk < DK / 16; ++kk)
 #pragma unroll
-                for (int nt = 0; nt < 8; ++nt) {
-                    const bf16* p = Kt + (nt * 8 + gq) * LD + kk * 16 + tq * 2;
-                    mma_bf16_16816(S[nt], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], *reinterpret_cast<const uint32_t*>(p),
-                                   *reinterpret_cast<const uint32_t*>(p + 8));
+                for (int nt = 0; nt < 8; nt += 4) {
+                    uint32_t k0[4], k1[4];          // two 8-key blocks each, their 16 coordinates in two halves
+                    const bf16* p = Kt + (nt * 8 + (lane & 7) + (lane >> 4) * 8) * LD + kk * 16 + ((lane >> 3) & 1) * 8;
+                    ldmatrix_x4(k0, p);
+                    ldmatrix_x4(k1, p + 16 * LD);
+                    mma_bf16_16816(S[nt], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], k0[0], k0[1]);
+                    mma_bf16_16816(S[nt + 1], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], k0[2], k0[3]);
+                    mma_bf16_16816(S[nt + 2], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], k1[0], k1[1]);
+                    mma_bf16_16816(S[nt + 3], qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], k1[2], k1[3]);
                 }
+            // scores: scaled, capped, penalised and masked -- or, in a tile that every row of the warp sees whole and where the score
+            // is the scaled product alone, left as they are with the scale inside the exponent
+            const bool direct = plain && j0 + 63 <= pos0 + tile * 64 + warp * 16;
             float mx_a = -INFINITY, mx_b = -INFINITY;
+            if (!direct) {
 #pragma unroll
-            for (int nt = 0; nt < 8; ++nt)
+                for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int j = j0 + nt * 8 + tq * 2 + (e & 1);
-                    const int i = e < 2 ? i_a : i_b;
-                    const float v = (j <= i && i - j < win) ? attn_score<true>(A, S[nt][e], i - j, r1, r2, slope) : -INFINITY;
-                    S[nt][e] = v;
-                    if (e < 2) mx_a = fmaxf(mx_a, v); else mx_b = fmaxf(mx_b, v);
-                }
+                    for (int e = 0; e < 4; ++e) {
+                        const int j = j0 + nt * 8 + tq * 2 + (e & 1);
+                        const int i = e < 2 ? i_a : i_b;
+                        S[nt][e] = (j <= i && i - j < win) ? attn_score<true>(A, S[nt][e], i - j, r1, r2, slope) : -INFINITY;
+                    }
+            }
+#pragma unroll
+            for (int nt = 0; nt < 8; ++nt) {
+                mx_a = fmaxf(mx_a, fmaxf(S[nt][0], S[nt][1]));
+                mx_b = fmaxf(mx_b, fmaxf(S[nt][2], S[nt][3]));
+            }
             mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 1));
             mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 2));
             mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 1));
             mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 2));
+            const float mul = direct ? A.scale : 1.0f;
             // without a sink a row of the tile's padding (beyond the sequence's rows) sees no key at all: keep its maximum finite
-            const float mn_a = fmaxf(fmaxf(m_a, mx_a), -1e30f), mn_b = fmaxf(fmaxf(m_b, mx_b), -1e30f);
-            const float ca = __expf(m_a - mn_a), cb = __expf(m_b - mn_b);
+            const float mn_a = fmaxf(fmaxf(m_a, mx_a * mul), -1e30f), mn_b = fmaxf(fmaxf(m_b, mx_b * mul), -1e30f);
+            constexpr float kLog2e = 1.4426950408889634f;
+            const float ca = exp2_fast((m_a - mn_a) * kLog2e), cb = exp2_fast((m_b - mn_b) * kLog2e);
             m_a = mn_a; m_b = mn_b;
             l_a *= ca; l_b *= cb;
 #pragma unroll
             for (int nt = 0; nt < DV / 8; ++nt) { o[nt][0] *= ca; o[nt][1] *= ca; o[nt][2] *= cb; o[nt][3] *= cb; }
+            const float mul2 = mul * kLog2e, na = -mn_a * kLog2e, nb = -mn_b * kLog2e;
             uint32_t hi[8][2], lo[8][2];
 #pragma unroll
             for (int nt = 0; nt < 8; ++nt) {
-                float p[4];
-#pragma unroll
-                for (int e = 0; e < 4; ++e) p[e] = __expf(S[nt][e] - (e < 2 ? mn_a : mn_b));
-                l_a += p[0] + p[1];
-                l_b += p[2] + p[3];
-                float ph[4];
-#pragma unroll
-                for (int e = 0; e < 4; ++e) ph[e] = bf16_round(p[e]);
-                hi[nt][0] = pack_bf16(ph[0], ph[1]); hi[nt][1] = pack_bf16(ph[2], ph[3]);
-                lo[nt][0] = pack_bf16(p[0] - ph[0], p[1] - ph[1]); lo[nt][1] = pack_bf16(p[2] - ph[2], p[3] - ph[3]);
+                const float p0 = exp2_fast(fmaf(S[nt][0], mul2, na)), p1 = exp2_fast(fmaf(S[nt][1], mul2, na));
+                const float p2 = exp2_fast(fmaf(S[nt][2], mul2, nb)), p3 = exp2_fast(fmaf(S[nt][3], mul2, nb));
+                l_a += p0 + p1;
+                l_b += p2 + p3;
+                hi[nt][0] = pack_bf16(p0, p1);
+                hi[nt][1] = pack_bf16(p2, p3);
+                lo[nt][0] = pack_bf16(p0 - bf_lo(hi[nt][0]), p1 - bf_hi(hi[nt][0]));
+                lo[nt][1] = pack_bf16(p2 - bf_lo(hi[nt][1]), p3 - bf_hi(hi[nt][1]));
             }
 #pragma unroll
             for (int k2 = 0; k2 < 4; ++k2)
 #pragma unroll
-                for (int nt = 0; nt < DV / 8; ++nt) {
-                    uint32_t b0, b1;
-                    ldmatrix_x2_trans(b0, b1, Vt + (k2 * 16 + (lane & 15)) * LDV + nt * 8);
-                    mma_bf16_16816(o[nt], hi[2 * k2][0], hi[2 * k2][1], hi[2 * k2 + 1][0], hi[2 * k2 + 1][1], b0, b1);
-                    mma_bf16_16816(o[nt], lo[2 * k2][0], lo[2 * k2][1], lo[2 * k2 + 1][0], lo[2 * k2 + 1][1], b0, b1);
+                for (int nt = 0; nt < DV / 8; nt += 4) {
+                    uint32_t v0[4], v1[4];          // two 8-column blocks each; all heads of the weights first, then all remainders
+                    const bf16* p = Vt + (k2 * 16 + (lane & 15)) * LDV + nt * 8 + (lane >> 4) * 8;
+                    ldmatrix_x4_trans(v0, p);
+                    ldmatrix_x4_trans(v1, p + 16);
+#pragma unroll
+                    for (int x = 0; x < 2; ++x) {
+                        const uint32_t(&w)[8][2] = x == 0 ? hi : lo;
+                        mma_bf16_16816(o[nt], w[2 * k2][0], w[2 * k2][1], w[2 * k2 + 1][0], w[2 * k2 + 1][1], v0[0], v0[1]);
+                        mma_bf16_16816(o[nt + 1], w[2 * k2][0], w[2 * k2][1], w[2 * k2 + 1][0], w[2 * k2 + 1][1], v0[2], v0[3]);
+                        mma_bf16_16816(o[nt + 2], w[2 * k2][0], w[2 * k2][1], w[2 * k2 + 1][0], w[2 * k2 + 1][1], v1[0], v1[1]);
+                        mma_bf16_16816(o[nt + 3], w[2 * k2][0], w[2 * k2][1], w[2 * k2 + 1][0], w[2 * k2 + 1][1], v1[2], v1[3]);
+                    }
                 }
         }
         __syncthreads();
@@ -1733,7 +1771,8 @@ struct SmolLm {
     struct Captured { SmolLmStep key; cudaGraphExec_t exec; int64_t launches; };
     std::vector<Captured> graphs;
     cudaStream_t cap_stream = nullptr;
-    // parallel block: the feed-forward runs on its own stream beside the mixer, between these two events
+    // parallel block: the feed-forward runs on its own stream beside the mixer, between these two events; output-norm block: a side
+    // mixer beside the layer's own
     cudaStream_t ff_stream = nullptr;
     cudaEvent_t ff_start = nullptr, ff_done = nullptr;
     ~SmolLm() {
@@ -2228,7 +2267,7 @@ extern "C" int smol_lm_bind(SmolLm* m, const SmolLmGlobals* g, void* d_workspace
     if ((m->cfg.block == SMOL_LM_BLOCK_PRENORM || m->cfg.block == SMOL_LM_BLOCK_PARALLEL) && m->cfg.norm_kind == SMOL_LM_NORM_LAYER && !g->final_norm_shift)
         return fail(SMOL_ERR_INVALID, "smol_lm_bind: the final layer norm needs its shift");
     if (m->any_merge && !g->w_merge) return fail(SMOL_ERR_INVALID, "smol_lm_bind: merging runs need w_merge");
-    if (m->cfg.block == SMOL_LM_BLOCK_PARALLEL && !m->ff_stream) {
+    if ((m->cfg.block == SMOL_LM_BLOCK_PARALLEL || m->cfg.block == SMOL_LM_BLOCK_OUTNORM) && !m->ff_stream) {
         CU(cudaStreamCreateWithFlags(&m->ff_stream, cudaStreamNonBlocking));
         CU(cudaEventCreateWithFlags(&m->ff_start, cudaEventDisableTiming));
         CU(cudaEventCreateWithFlags(&m->ff_done, cudaEventDisableTiming));
@@ -2460,7 +2499,7 @@ static void launch_attention(SmolLm* m, const SmolLmStep* s, AttnArgs& A, bool f
             if (wide) attn_split_kernel<T, MAXV, 2><<<grid, nwarp * 32, smem_of(64), st>>>(A, qbuf, pool);
         }
         if (!wide) attn_split_kernel<T, MAXV, 1><<<grid, nwarp * 32, smem_of(32), st>>>(A, qbuf, pool);
-        attn_merge_kernel<T, MAXV, MAPS><<<A.short_rows * A.H, kMergeWarps * 32, kMergeWarps * (A.dv + 1) * sizeof(float), st>>>(A, mix);
+        attn_merge_kernel<T, MAXV, MAPS><<<A.short_rows * A.H, kMergeWarps * MAPS * 32, kMergeWarps * MAPS * (A.dv + 1) * sizeof(float), st>>>(A, mix);
         m->launches += 2;
     }
 }
@@ -2599,6 +2638,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
         int mix_cols;
         int out_ld_now = mix_ld;        // row stride of the buffer the current mixer writes
         const T* mix_in = mix;          // what the output projection reads
+        cudaStream_t ms = st;           // the stream the current mixer runs on
         // Softmax attention over keys and values in the paged pool.  pj / bias: this mixer's rows of the fused projection.
         auto attention = [&](const SmolLmLayer& M, const RunInfo& Ri, const float* pj, const float* bias, T* mix_at) -> int {
             AttnArgs A;
@@ -2621,19 +2661,19 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
                 const int threads = Tn > 64 ? 128 : 256;      // few tokens: more loads in flight per token
                 A.rot_pairs = M.rot_dims / 2; A.rot_half = M.rot_half; A.rot_mult = M.rot_mult != 0.0f ? M.rot_mult : 1.0f;
                 A.freq = reinterpret_cast<const float*>(m->ws + m->o_freq) + Ri.freq_off;
-                if (A.rot_pairs > 0) attn_prep_whole_kernel<T, true><<<Tn, threads, 0, st>>>(A, qbuf, pool);
-                else attn_prep_whole_kernel<T, false><<<Tn, threads, 0, st>>>(A, qbuf, pool);
+                if (A.rot_pairs > 0) attn_prep_whole_kernel<T, true><<<Tn, threads, 0, ms>>>(A, qbuf, pool);
+                else attn_prep_whole_kernel<T, false><<<Tn, threads, 0, ms>>>(A, qbuf, pool);
             } else {
                 const int units = Tn * (M.heads * A.maps + (A.own_kv ? M.kv_heads * (A.maps + 1) : 0));
-                attn_prep_kernel<T><<<(units + 3) / 4, 128, 0, st>>>(A, qbuf, pool);
+                attn_prep_kernel<T><<<(units + 3) / 4, 128, 0, ms>>>(A, qbuf, pool);
             }
             m->launches += 1;
             const bool flash = sizeof(T) == 2 && std::max(M.dim, M.vdim) <= 128;
             if (A.maps == 2) {
-                if (M.vdim <= 256) launch_attention<T, 8, 2>(m, s, A, flash, qbuf, pool, mix_at, st);
-                else launch_attention<T, 16, 2>(m, s, A, flash, qbuf, pool, mix_at, st);
-            } else if (M.vdim <= 256) launch_attention<T, 8, 1>(m, s, A, flash, qbuf, pool, mix_at, st);
-            else launch_attention<T, 16, 1>(m, s, A, flash, qbuf, pool, mix_at, st);
+                if (M.vdim <= 256) launch_attention<T, 8, 2>(m, s, A, flash, qbuf, pool, mix_at, ms);
+                else launch_attention<T, 16, 2>(m, s, A, flash, qbuf, pool, mix_at, ms);
+            } else if (M.vdim <= 256) launch_attention<T, 8, 1>(m, s, A, flash, qbuf, pool, mix_at, ms);
+            else launch_attention<T, 16, 1>(m, s, A, flash, qbuf, pool, mix_at, ms);
             return SMOL_OK;
         };
         // State-space recurrence: convolution and per-head step / decay, the scan over the slot's state, then skip, gate and the
@@ -2648,7 +2688,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             P.slot_floats = m->slot_floats; P.conv_off = Ri.conv_off; P.n_slots = m->n_slots; P.err = err;
             P.out_ld = out_ld_now; P.out_scale = M.mix_scale;
             const dim3 cgrid(Tn, (ch + 127) / 128);
-            ssd_conv_kernel<<<cgrid, 128, 0, st>>>(P, m->slots, conv, head);
+            ssd_conv_kernel<<<cgrid, 128, 0, ms>>>(P, m->slots, conv, head);
             GlaArgs A;
             A.proj = pj; A.n_in = n_in; A.H = M.heads; A.d = M.n_state; A.dv = M.vdim; A.rank = 0; A.n_tokens = Tn;
             A.q_scale = 1.0f; A.tau = 1.0f; A.eps = c.norm_eps;
@@ -2660,8 +2700,8 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             A.qk_share = M.heads / M.bc_groups;
             A.head_decay = head; A.head_step = head + (size_t)Tn * M.heads; A.head_ld = M.heads;
             A.out_ld = out_ld_now; A.out_scale = 1.0f;
-            CU(launch_gla_scan_any(A, s->n_seqs, nullptr, m->slots, oraw, st));
-            ssd_out_kernel<T><<<dim3(Tn, M.norm_parts), 256, 0, st>>>(P, oraw, conv, mix_at, m->slots);
+            CU(launch_gla_scan_any(A, s->n_seqs, nullptr, m->slots, oraw, ms));
+            ssd_out_kernel<T><<<dim3(Tn, M.norm_parts), 256, 0, ms>>>(P, oraw, conv, mix_at, m->slots);
             m->launches += 3;
             return SMOL_OK;
         };
@@ -2687,13 +2727,13 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             S.range_len = 1 << 30; S.n_ranges = 1; S.partial = nullptr;
             S.freq = reinterpret_cast<const float*>(m->ws + m->o_freq) + Ri.freq_off;
             const int units = Tn * (M.heads + M.kv_heads);
-            sigmoid_prep_kernel<T><<<(units + 3) / 4, 128, 0, st>>>(S, qbuf, pool);
+            sigmoid_prep_kernel<T><<<(units + 3) / 4, 128, 0, ms>>>(S, qbuf, pool);
             m->launches += 1;
             const int min_n = s->min_seq_tokens > 0 ? s->min_seq_tokens : 1;
             const int max_n = s->max_seq_tokens > 0 ? s->max_seq_tokens : Tn;
             // sequences that bring more than a few tokens take the tiled tensor-core form (bf16), the others a warp per head
             const bool tiled = max_n > kShortSeq && launch_sigmoid_flash(m, s, S, max_n, reinterpret_cast<const bf16*>(qbuf), reinterpret_cast<const bf16*>(pool),
-                                                                         reinterpret_cast<bf16*>(mix_at), sizeof(T) == 2, st);
+                                                                         reinterpret_cast<bf16*>(mix_at), sizeof(T) == 2, ms);
             // sequences of few tokens (decoding): key ranges over separate blocks, merged afterwards
             const size_t split_smem = sigmoid_split_smem<T>(M.heads, M.kv_heads, M.dim, M.vdim);
             const bool split = min_n <= kShortSeq && split_smem <= (size_t)kSigmoidSmemMax;
@@ -2705,9 +2745,9 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
                 A.n_splits = std::min(m->max_splits, (max_pos / m->split_len + 4) / 4 * 4);
                 if (M.chunk > 0) A.n_splits = std::min(A.n_splits, ((M.chunk - 1) / m->split_len + 2 + 3) / 4 * 4);      // ranges a chunk can touch
                 const dim3 grid(A.short_rows, A.n_splits);
-                if (M.vdim <= 256) sigmoid_split_kernel<T, 8><<<grid, M.heads * 32, split_smem, st>>>(S, qbuf, pool);
-                else sigmoid_split_kernel<T, 16><<<grid, M.heads * 32, split_smem, st>>>(S, qbuf, pool);
-                sigmoid_short_merge_kernel<T><<<A.short_rows, 128, 0, st>>>(S, mix_at);
+                if (M.vdim <= 256) sigmoid_split_kernel<T, 8><<<grid, M.heads * 32, split_smem, ms>>>(S, qbuf, pool);
+                else sigmoid_split_kernel<T, 16><<<grid, M.heads * 32, split_smem, ms>>>(S, qbuf, pool);
+                sigmoid_short_merge_kernel<T><<<A.short_rows, 128, 0, ms>>>(S, mix_at);
                 m->launches += 2;
             }
             const bool long_left = max_n > kShortSeq && !tiled, short_left = min_n <= kShortSeq && !split;
@@ -2715,8 +2755,8 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
                 // the warp-per-head form: every row, or only the rows the other two forms left
                 S.only = (long_left && short_left) ? 0 : long_left ? 1 : 2;
                 const size_t smem = ((size_t)M.heads * (M.dim + 32) + (size_t)M.heads * M.heads) * sizeof(float);
-                if (M.vdim <= 256) sigmoid_attn_kernel<T, 8><<<Tn, M.heads * 32, smem, st>>>(S, qbuf, pool, mix_at);
-                else sigmoid_attn_kernel<T, 16><<<Tn, M.heads * 32, smem, st>>>(S, qbuf, pool, mix_at);
+                if (M.vdim <= 256) sigmoid_attn_kernel<T, 8><<<Tn, M.heads * 32, smem, ms>>>(S, qbuf, pool, mix_at);
+                else sigmoid_attn_kernel<T, 16><<<Tn, M.heads * 32, smem, ms>>>(S, qbuf, pool, mix_at);
                 m->launches += 1;
             }
             return SMOL_OK;
@@ -2737,14 +2777,14 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
         auto lightning = [&](const SmolLmLayer& M, const RunInfo& Ri, const float* pj, T* mix_at, int ld) -> int {
             const int hd = M.heads * M.dim, hv = M.heads * M.vdim, na = 2 * hd + hv;
             LinPrepArgs P{pj, n_in, M.heads, M.dim, M.vdim, Tn, M.head_decay, nullptr, nullptr};
-            lightning_prep_kernel<<<dim3(Tn, (na + 1023) / 1024), 256, 0, st>>>(P, conv, head);
+            lightning_prep_kernel<<<dim3(Tn, (na + 1023) / 1024), 256, 0, ms>>>(P, conv, head);
             GlaArgs A = scan_args(M, Ri, pj);
             A.q_src = conv; A.k_src = conv + hd; A.v_src = conv + 2 * hd;
             A.q_ld = A.k_ld = A.v_ld = na;
             A.head_decay = head; A.head_step = head + (size_t)Tn * M.heads;
-            CU(launch_gla_scan_any(A, s->n_seqs, nullptr, m->slots, oraw, st));
+            CU(launch_gla_scan_any(A, s->n_seqs, nullptr, m->slots, oraw, ms));
             LinOutArgs O{pj, n_in, hv, hv, hv, 1, ld, (size_t)2 * hd + hv, c.norm_eps, 1.0f, M.out_norm};
-            lin_attn_out_kernel<T><<<dim3(Tn, 1), 256, 0, st>>>(O, oraw, mix_at);
+            lin_attn_out_kernel<T><<<dim3(Tn, 1), 256, 0, ms>>>(O, oraw, mix_at);
             m->launches += 3;
             return SMOL_OK;
         };
@@ -2752,14 +2792,14 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
         auto retention = [&](const SmolLmLayer& M, const RunInfo& Ri, const float* pj, T* mix_at, int ld) -> int {
             const int hd = M.heads * M.dim, pairs = M.rot_dims / 2, per = M.heads * (M.dim - pairs);
             RetentionArgs P{pj, n_in, M.heads, M.dim, pairs, M.rot_half, M.score_scale, reinterpret_cast<const float*>(m->ws + m->o_freq) + Ri.freq_off, s->tok_pos};
-            retention_prep_kernel<<<dim3(Tn, (per + 511) / 512), 128, 0, st>>>(P, conv);
+            retention_prep_kernel<<<dim3(Tn, (per + 511) / 512), 128, 0, ms>>>(P, conv);
             GlaArgs A = scan_args(M, Ri, pj);
             A.q_src = conv; A.k_src = conv + hd; A.v_src = pj + 2 * hd;
             A.q_ld = A.k_ld = 2 * hd; A.v_ld = n_in;
             A.head_decay = M.head_decay; A.head_ld = 0;
-            CU(launch_gla_scan_any(A, s->n_seqs, nullptr, m->slots, oraw, st, parallel && Tn > kGraphMaxTokens ? kScanSpread : 0));
+            CU(launch_gla_scan_any(A, s->n_seqs, nullptr, m->slots, oraw, ms, parallel && Tn > kGraphMaxTokens ? kScanSpread : 0));
             A.out_ld = ld; A.out_scale = M.mix_scale;
-            gla_out_kernel<T><<<(Tn * M.heads + 3) / 4, 128, 0, st>>>(A, oraw, mix_at);
+            gla_out_kernel<T><<<(Tn * M.heads + 3) / 4, 128, 0, ms>>>(A, oraw, mix_at);
             m->launches += 3;
             return SMOL_OK;
         };
@@ -2785,15 +2825,15 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             P.tok_seq = s->tok_seq; P.err = err;
             P.conv = ConvIo{pj, nullptr, n_in, ch, M.conv_taps, M.conv_w, nullptr, s->seq_start, s->seq_pos0, s->seq_slot, m->slot_floats, Ri.conv_off, m->n_slots};
             const int warps = M.kv_heads + (hv + kGatedDeltaCols - 1) / kGatedDeltaCols;
-            gated_delta_prep_kernel<<<dim3(Tn, (warps + 3) / 4), 128, 0, st>>>(P, m->slots, conv, head, pairs);
+            gated_delta_prep_kernel<<<dim3(Tn, (warps + 3) / 4), 128, 0, ms>>>(P, m->slots, conv, head, pairs);
             GroupScanArgs S = group_args(M, Ri, M.kv_heads);
             S.q_src = conv; S.k_src = conv + gd; S.v_src = conv + 2 * gd;
             S.q_ld = S.k_ld = S.v_ld = ch;
             S.conv = P.conv;
-            CU(launch_group_scan_any<true>(m, S, pairs, s->n_seqs, max_n, m->slots, oraw, st));
+            CU(launch_group_scan_any<true>(m, S, pairs, s->n_seqs, max_n, m->slots, oraw, ms));
             GlaArgs A = scan_args(M, Ri, pj);
             A.out_norm = M.out_norm; A.gate_off = ch; A.out_ld = ld; A.out_scale = M.mix_scale;
-            gla_out_kernel<T><<<(Tn * M.heads + 3) / 4, 128, 0, st>>>(A, oraw, mix_at);
+            gla_out_kernel<T><<<(Tn * M.heads + 3) / 4, 128, 0, ms>>>(A, oraw, mix_at);
             m->launches += 2;
             return SMOL_OK;
         };
@@ -2808,17 +2848,17 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             P.i_bias = M.rate_bias; P.f_bias = M.decay_bias;
             P.seq_start = s->seq_start; P.seq_pos0 = s->seq_pos0; P.seq_slot = s->seq_slot;
             P.slot_floats = m->slot_floats; P.m_off = Ri.m_off; P.n_slots = m->n_slots; P.err = err;
-            mlstm_gate_kernel<<<s->n_seqs * M.heads, std::min(kMlstmTile, (max_n + 31) / 32 * 32), 0, st>>>(P, m->slots, head, floor_at, pairs);
+            mlstm_gate_kernel<<<s->n_seqs * M.heads, std::min(kMlstmTile, (max_n + 31) / 32 * 32), 0, ms>>>(P, m->slots, head, floor_at, pairs);
             GroupScanArgs S = group_args(M, Ri, M.heads);
             S.q_src = pj; S.k_src = pj + hd; S.v_src = pj + 2 * hd;
             S.q_ld = S.k_ld = S.v_ld = n_in;
             S.q_scale = M.score_scale;
             S.unit_out = den; S.unit_off = Ri.unit_off;
-            CU(launch_group_scan_any<false>(m, S, pairs, s->n_seqs, max_n, m->slots, oraw, st));
+            CU(launch_group_scan_any<false>(m, S, pairs, s->n_seqs, max_n, m->slots, oraw, ms, ms != st && Tn > kGraphMaxTokens ? kScanSpread : 0));
             GlaArgs A = scan_args(M, Ri, pj);
             A.den = den; A.den_floor = floor_at; A.den_eps = M.den_eps;
             A.out_norm = M.out_norm; A.norm_own = 1; A.gate_sigmoid = 1; A.out_ld = ld; A.out_scale = M.mix_scale;
-            gla_out_kernel<T><<<(Tn * M.heads + 3) / 4, 128, 0, st>>>(A, oraw, mix_at);
+            gla_out_kernel<T><<<(Tn * M.heads + 3) / 4, 128, 0, ms>>>(A, oraw, mix_at);
             m->launches += 2;
             return SMOL_OK;
         };
@@ -2970,12 +3010,26 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             if (beside) CU(cudaEventRecord(m->ff_done, m->ff_stream));
         }
         if (pairable(L)) {
-            int rc = run_mixer(L, R, proj, L.in_bias, mix, own_proj ? mix_cols_of(L) : mix_ld);
-            if (rc == SMOL_OK && L.side) {
+            // The pair of the output-norm block shares no buffer but the result, of which each writes its own columns: the side
+            // mixer runs on its own stream beside the layer's.
+            const bool fork = outnorm && L.side;
+            int rc = SMOL_OK;
+            auto run_side = [&]() -> int {
                 const SmolLmLayer& S = *L.side;
                 const float* sb = L.in_bias ? L.in_bias + n_in_main : nullptr;
-                rc = run_mixer(S, m->side_runs[n], proj + n_in_main, sb, own_proj ? mix2 : mix + mix_cols_of(L), own_proj ? mix_cols_of(S) : mix_ld);
+                return run_mixer(S, m->side_runs[n], proj + n_in_main, sb, own_proj ? mix2 : mix + mix_cols_of(L), own_proj ? mix_cols_of(S) : mix_ld);
+            };
+            if (fork) {
+                CU(cudaEventRecord(m->ff_start, st));
+                CU(cudaStreamWaitEvent(m->ff_stream, m->ff_start, 0));
+                ms = m->ff_stream;
+                rc = run_side();
+                CU(cudaEventRecord(m->ff_done, m->ff_stream));
+                ms = st;
             }
+            if (rc == SMOL_OK) rc = run_mixer(L, R, proj, L.in_bias, mix, own_proj ? mix_cols_of(L) : mix_ld);
+            if (rc == SMOL_OK && L.side && !fork) rc = run_side();
+            if (rc == SMOL_OK && fork) CU(cudaStreamWaitEvent(st, m->ff_done, 0));
             if (rc != SMOL_OK) return rc;
             mix_cols = own_proj ? mix_cols_of(L) : mix_ld;
         } else if (L.mixer == SMOL_LM_MIX_HGRN2) {
