@@ -349,7 +349,7 @@ struct MlstmArgs {
     int n_slots;
     int32_t* err;
 };
-constexpr int kMlstmTile = 256;
+constexpr int kMlstmTile = 1024;
 
 // head: (decay, write weight) [T][H]; floor [T][H]
 __global__ void __launch_bounds__(kMlstmTile) mlstm_gate_kernel(const MlstmArgs A, float* __restrict__ slots, float* __restrict__ head, float* __restrict__ floor_,

@@ -1138,29 +1138,48 @@ __global__ void __launch_bounds__(kMergeWarps * MAPS * 32) attn_merge_kernel(con
         const int c = lane + e * 32;
         if (c < A.dv) share[warp * A.dv + c] = o[e];
     }
-    __syncthreads();
-    if (warp > 0) return;
-    float sum[MAXV];                    // the maps' joined result
+    // from here on a thread per column
+    constexpr int COLS = MAXV * 32 / (ALL * 32) > 1 ? MAXV * 32 / (ALL * 32) : 1;
+    float gate[COLS], sum[COLS];
 #pragma unroll
-    for (int e = 0; e < MAXV; ++e) sum[e] = 0.0f;
+    for (int e = 0; e < COLS; ++e) {
+        const int c = threadIdx.x + e * ALL * 32;
+        gate[e] = c < A.dv ? attn_gate(A, t, h, c) : 0.0f;
+    }
+    __syncthreads();
+    float inv[MAPS], ss = 0.0f;
 #pragma unroll
     for (int mp = 0; mp < MAPS; ++mp) {
         float den = 0.0f;
 #pragma unroll
         for (int w = 0; w < PER; ++w) den += share[ALL * A.dv + mp * PER + w];
-        const float inv = (mp == 0 ? 1.0f : -A.diff_lambda) / den;
+        inv[mp] = (mp == 0 ? 1.0f : -A.diff_lambda) / den;
+    }
 #pragma unroll
-        for (int e = 0; e < MAXV; ++e) {
-            const int c = lane + e * 32;
-            if (c < A.dv) {
+    for (int e = 0; e < COLS; ++e) {
+        const int c = threadIdx.x + e * ALL * 32;
+        sum[e] = 0.0f;
+        if (c < A.dv) {
+#pragma unroll
+            for (int mp = 0; mp < MAPS; ++mp) {
                 float v = 0.0f;
 #pragma unroll
                 for (int w = 0; w < PER; ++w) v += share[(mp * PER + w) * A.dv + c];
-                sum[e] = fmaf(v, inv, sum[e]);
+                sum[e] = fmaf(v, inv[mp], sum[e]);
             }
         }
+        ss = fmaf(sum[e], sum[e], ss);
     }
-    attn_finish<T, MAXV, MAPS>(A, t, h, lane, sum, out);
+    float scale = 1.0f;
+    if (MAPS == 2) {
+        __shared__ float red[33];
+        scale = A.diff_scale / sqrtf(block_sum(ss, red) / (float)A.dv + A.eps);
+    }
+#pragma unroll
+    for (int e = 0; e < COLS; ++e) {
+        const int c = threadIdx.x + e * ALL * 32;
+        if (c < A.dv) out[(size_t)t * A.out_ld + h * A.dv + c] = from_f<T>((MAPS == 2 ? sum[e] * scale : sum[e]) * gate[e]);
+    }
 }
 
 // ---------------------------------------------------------------------------------------------------------------------

@@ -355,19 +355,19 @@ def loud_gates(w):
 @both
 def test_mlstm_running_maximum_and_denominator(dtype, monkeypatch):
     """With an eps that does not vanish beside a head's values the denominator shows: an oracle without its floor or without the key
-    sum gives something else.  Gates spread wide move the maximum up and down; the gate kernel's tiles (256 tokens) are crossed by prompts and portions."""
+    sum gives something else.  Gates spread wide move the maximum up and down; the gate kernel's tiles (1024 tokens) are crossed by the whole prompt."""
     from oracle import virusun_oracle as vo
 
     cfg = config([par(left(heads=1, kv_heads=1, dim=4, vdim=4), right(heads=5, dim=8, vdim=12, cap=16.0), 0.1, 1.5)], vocab=43, eps=0.05)
-    model, orc, w = engine_and_oracle(cfg, seed=8, dtype=dtype, edit=loud_gates, max_tokens=768, max_step_tokens=1024)
-    toks = tokens(560, 43, 6)
+    model, orc, w = engine_and_oracle(cfg, seed=8, dtype=dtype, edit=loud_gates, max_tokens=1216, max_step_tokens=2048)
+    toks = tokens(1200, 43, 6)
     want = orc.forward(toks)
     for wrong in (lambda dot, m: dot.abs() + 1e-6, lambda dot, m: torch.exp(-m) + 1e-6):
         with monkeypatch.context() as mp:
             mp.setattr(vo, "memory_denominator", wrong)
             assert rel_err(orc.forward(toks), want) > 100 * TOL[F32]
     assert close_enough(run_whole(model, toks), want, dtype)
-    for sizes in ([255, 2, 256, 2], [300, 1, 1, 200], [33] * 15):
+    for sizes in ([255, 2, 256, 2, 600], [1030, 1, 1, 120], [33] * 33):
         assert close_enough(run_portions(model, toks, sizes), want, dtype), sizes
 
 
