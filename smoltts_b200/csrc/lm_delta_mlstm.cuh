@@ -258,7 +258,7 @@ __global__ void __launch_bounds__(gla_block_cols(DK) * gla_lanes(DK)) group_scan
 //   S <- w S;  u = b (v - S^T k);  S <- S + k u^T;  o = S^T q
 struct GatedDeltaArgs {
     const float* proj;
-    int n_in, H, G, d, dv, n_tokens;
+    int n_in, H, G, d, dv;
     float q_scale, unit_eps;
     const float *a_log, *dt_bias;
     const int32_t* tok_seq;
@@ -339,7 +339,7 @@ __global__ void __launch_bounds__(128) gated_delta_prep_kernel(const GatedDeltaA
 // also gets its k.q here (pairs, see group_scan_kernel).
 struct MlstmArgs {
     const float* proj;
-    int n_in, H, n_tokens;
+    int n_in, H;
     size_t gate_off;                   // column of the input rows; the forget rows follow
     int d;                             // q rows [H*d] first, k rows behind them
     float cap;

@@ -2839,7 +2839,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
         auto gated_delta = [&](const SmolLmLayer& M, const RunInfo& Ri, const float* pj, T* mix_at, int ld) -> int {
             const int hv = M.heads * M.vdim, gd = M.kv_heads * M.dim, ch = 2 * gd + hv;
             GatedDeltaArgs P;
-            P.proj = pj; P.n_in = n_in; P.H = M.heads; P.G = M.kv_heads; P.d = M.dim; P.dv = M.vdim; P.n_tokens = Tn;
+            P.proj = pj; P.n_in = n_in; P.H = M.heads; P.G = M.kv_heads; P.d = M.dim; P.dv = M.vdim;
             P.q_scale = M.score_scale; P.unit_eps = M.unit_eps; P.a_log = M.a_log; P.dt_bias = M.dt_bias;
             P.tok_seq = s->tok_seq; P.err = err;
             P.conv = ConvIo{pj, nullptr, n_in, ch, M.conv_taps, M.conv_w, nullptr, s->seq_start, s->seq_pos0, s->seq_slot, m->slot_floats, Ri.conv_off, m->n_slots};
@@ -2863,7 +2863,7 @@ static int step_impl(SmolLm* m, const SmolLmStep* s, cudaStream_t st) {
             const size_t TH = (size_t)Tn * M.heads;
             float *floor_at = head + 2 * TH, *den = head + 3 * TH;
             MlstmArgs P;
-            P.proj = pj; P.n_in = n_in; P.H = M.heads; P.d = M.dim; P.n_tokens = Tn; P.gate_off = (size_t)2 * hd + 2 * hv; P.cap = M.gate_cap;
+            P.proj = pj; P.n_in = n_in; P.H = M.heads; P.d = M.dim; P.gate_off = (size_t)2 * hd + 2 * hv; P.cap = M.gate_cap;
             P.i_bias = M.rate_bias; P.f_bias = M.decay_bias;
             P.seq_start = s->seq_start; P.seq_pos0 = s->seq_pos0; P.seq_slot = s->seq_slot;
             P.slot_floats = m->slot_floats; P.m_off = Ri.m_off; P.n_slots = m->n_slots; P.err = err;
